@@ -89,6 +89,21 @@ class LatentNeed(PagedCacheNeed):
 
 
 @dataclass(frozen=True)
+class TokenNeed(PagedCacheNeed):
+    """The token ids themselves: ``token`` pages of ``[page_size]`` int32.  ``window = 2`` keeps the token before the
+    next one (for a part that reads pairs of tokens).  Pages rather than a per-request state: a step that is dropped
+    or fails has only written beyond the committed tokens, so nothing has to be taken back."""
+
+    window: int = 0
+    pages_fraction: float = 1.0
+    keep_first: int = 0
+
+    def tensors(self, page_size: int) -> List[PageTensor]:
+        import torch
+        return [("token", (page_size,), torch.int32)]
+
+
+@dataclass(frozen=True)
 class StateNeed:
     """A fixed-size state per request (``shape`` per slot), zeroed when a request starts."""
 

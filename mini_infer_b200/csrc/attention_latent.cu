@@ -7,9 +7,10 @@
 // (attention_mix.cu and attention_mix_tc.cu with a value row stride, attention_prefill_tc.cu with (query, head)
 // pairs as the rows of a query tile); what is left for this file:
 //
-//   latent_store   the cached row of every new token: unit-RMS latent times gain, rotated key part
-//   latent_query   the rotated part of every head's query into its place behind the folded part, and the
-//                  unrotated part in the activation type as the operand of the folding product
+//   latent_rows    (latent_store) the cached row of every new token: unit-RMS latent times gain, rotated key part;
+//                  (latent_query) the rotated part of every head's query into its place behind the folded part, and
+//                  the unrotated part in the activation type as the operand of the folding product; both at once
+//                  when one product of the layer's input holds queries and latent
 //   sigmoid_gate   out[t, h, :] = a[t, h, :] * sigmoid(g[t, h, :]), the gate on the heads' outputs
 //
 // The rotation pairs NEIGHBOURS: dimensions 2i and 2i + 1 turn by the angle position * inv_freq[i].  Angles,
@@ -19,59 +20,98 @@
 
 namespace mi {
 
-// one block per token; src row: `ld` floats, the latent part at column `col0`
+struct LatentStoreArgs {
+    const float* src;           // rows of `ld` floats, latent and rotated key part from column `col0` (null: none)
+    int ld, col0;
+    const float* gain;
+    float eps;
+    const int* slot_mapping;
+    void* cache;                // rows of c + r
+};
+// A query row has H heads of [d unrotated | r rotated] floats.  Unrotated parts go to plain + (t H + h) plain_stride,
+// rotated ones to rot + (t H + h) rot_stride, each followed by zeros up to plain_pad and rot_pad numbers.
+struct LatentQueryArgs {
+    const float* q;             // rows of `ld` floats from column `col0` (null: none)
+    int ld, col0;
+    void *plain, *rot;          // plain null: not wanted
+    int plain_stride, rot_stride, plain_pad, rot_pad;
+};
+
+// grid (tokens, blocks per token): the blocks of a token share its heads, the first one writes the cached row.
+// `magnitude` multiplies cosines and sines.
 template <typename AT>
 __global__ void __launch_bounds__(256)
-latent_store_kernel(const float* __restrict__ src, int ld, int col0, const int* __restrict__ positions,
-                    const float* __restrict__ inv_freq, const float* __restrict__ gain, float eps,
-                    const int* __restrict__ slot_mapping, AT* __restrict__ cache, int c, int r) {
+latent_rows_kernel(LatentStoreArgs st, LatentQueryArgs qa, const int* __restrict__ positions,
+                   const float* __restrict__ inv_freq, float magnitude, int H, int d, int r, int c) {
+    extern __shared__ float trig[];                 // cosines, then sines, of this token's r / 2 angles
     __shared__ float red[32];
     wait_for_earlier_kernels();
     const int t = blockIdx.x;
-    const int slot = slot_mapping[t];
-    if (slot < 0) return;                           // a row of no request: written nowhere
-    const float* row = src + (int64_t)t * ld + col0;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < c; i += blockDim.x) { const float x = row[i]; ss += x * x; }
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)c + eps);
-    AT* out = cache + (int64_t)slot * (c + r);
-    for (int i = threadIdx.x; i < c; i += blockDim.x) out[i] = from_float<AT>(row[i] * inv * gain[i]);
-    const float pos = (float)positions[t];
-    for (int i = threadIdx.x; i < r / 2; i += blockDim.x) {
-        const float ang = pos * inv_freq[i];
-        const float cs = cosf(ang), sn = sinf(ang);
-        const float u = row[c + 2 * i], v = row[c + 2 * i + 1];
-        out[c + 2 * i] = from_float<AT>(u * cs - v * sn);
-        out[c + 2 * i + 1] = from_float<AT>(v * cs + u * sn);
-    }
-}
-
-// one block per token; q row: H heads of [d unrotated | r rotated] floats
-template <typename AT>
-__global__ void __launch_bounds__(256)
-latent_query_kernel(const float* __restrict__ q, const int* __restrict__ positions,
-                    const float* __restrict__ inv_freq, AT* __restrict__ q_plain, AT* __restrict__ q_full, int H,
-                    int d, int r, int c) {
-    wait_for_earlier_kernels();
-    const int t = blockIdx.x;
-    const float* row = q + (int64_t)t * H * (d + r);
-    const float pos = (float)positions[t];
     const int half = r / 2;
-    for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
-        const int h = idx / half, i = idx - h * half;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
         const float ang = pos * inv_freq[i];
-        const float cs = cosf(ang), sn = sinf(ang);
-        const float u = row[h * (d + r) + d + 2 * i], v = row[h * (d + r) + d + 2 * i + 1];
-        AT* out = q_full + ((int64_t)t * H + h) * (c + r) + c;
-        out[2 * i] = from_float<AT>(u * cs - v * sn);
-        out[2 * i + 1] = from_float<AT>(v * cs + u * sn);
+        trig[i] = cosf(ang) * magnitude;
+        trig[half + i] = sinf(ang) * magnitude;
     }
-    if (q_plain)
-        for (int idx = threadIdx.x; idx < H * d; idx += blockDim.x) {
-            const int h = idx / d, i = idx - h * d;
-            q_plain[(int64_t)t * H * d + idx] = from_float<AT>(row[h * (d + r) + i]);
+    __syncthreads();
+    if (st.src && blockIdx.y == 0) {
+        const int slot = st.slot_mapping[t];
+        if (slot >= 0) {                            // else a row of no request: written nowhere
+            const float* row = st.src + (int64_t)t * st.ld + st.col0;
+            float ss = 0.f;
+            for (int i = threadIdx.x; i < c; i += blockDim.x) { const float x = row[i]; ss += x * x; }
+            ss = block_sum(ss, red);
+            const float inv = 1.0f / sqrtf(ss / (float)c + st.eps);
+            AT* out = reinterpret_cast<AT*>(st.cache) + (int64_t)slot * (c + r);
+            for (int i = threadIdx.x; i < c; i += blockDim.x) out[i] = from_float<AT>(row[i] * inv * st.gain[i]);
+            for (int i = threadIdx.x; i < half; i += blockDim.x) {
+                const float u = row[c + 2 * i], v = row[c + 2 * i + 1];
+                out[c + 2 * i] = from_float<AT>(u * trig[i] - v * trig[half + i]);
+                out[c + 2 * i + 1] = from_float<AT>(v * trig[i] + u * trig[half + i]);
+            }
         }
+    }
+    if (!qa.q) return;
+    const float* row = qa.q + (int64_t)t * qa.ld + qa.col0;
+    const int per = (H + gridDim.y - 1) / gridDim.y;
+    const int h_lo = blockIdx.y * per, h_hi = min(H, h_lo + per);
+    const int nh = h_hi - h_lo;
+    if (nh <= 0) return;
+    if (qa.plain) {
+        AT* plain = reinterpret_cast<AT*>(qa.plain) + ((int64_t)t * H + h_lo) * qa.plain_stride;
+        const int pad = qa.plain_pad;
+        if (d % 4 == 0 && pad % 4 == 0 && qa.plain_stride % 4 == 0 && (qa.ld | qa.col0 | r) % 4 == 0 &&
+            ((reinterpret_cast<uintptr_t>(qa.q) | reinterpret_cast<uintptr_t>(qa.plain)) & 15) == 0) {
+            const int pv = pad / 4;
+            for (int idx = threadIdx.x; idx < nh * pv; idx += blockDim.x) {
+                const int h = idx / pv, i = (idx - h * pv) * 4;
+                float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i < d) x = *reinterpret_cast<const float4*>(row + (h_lo + h) * (d + r) + i);
+                store4(plain + (int64_t)h * qa.plain_stride + i, x);
+            }
+        } else {
+            for (int idx = threadIdx.x; idx < nh * pad; idx += blockDim.x) {
+                const int h = idx / pad, i = idx - h * pad;
+                plain[(int64_t)h * qa.plain_stride + i] = from_float<AT>(i < d ? row[(h_lo + h) * (d + r) + i] : 0.f);
+            }
+        }
+    }
+    AT* rot = reinterpret_cast<AT*>(qa.rot) + ((int64_t)t * H + h_lo) * qa.rot_stride;
+    const int hp = (qa.rot_pad > r ? qa.rot_pad : r) / 2;
+    for (int idx = threadIdx.x; idx < nh * hp; idx += blockDim.x) {
+        const int h = idx / hp, i = idx - h * hp;
+        float a = 0.f, b = 0.f;
+        if (i < half) {
+            const float* p = row + (h_lo + h) * (d + r) + d + 2 * i;
+            const float u = p[0], v = p[1];
+            a = u * trig[i] - v * trig[half + i];
+            b = v * trig[i] + u * trig[half + i];
+        }
+        AT* out = rot + (int64_t)h * qa.rot_stride;
+        out[2 * i] = from_float<AT>(a);
+        out[2 * i + 1] = from_float<AT>(b);
+    }
 }
 
 // out[t, h, j] = a[h * a_head + t * a_tok + j] * sigmoid(g[t * ldg + col0 + h * e + j])
@@ -124,31 +164,35 @@ using namespace mi;
 
 extern "C" {
 
-int mi_latent_store(const float* src, int ld, int col0, const int* positions, const float* inv_freq,
-                    const float* gain, float eps, const int* slot_mapping, void* cache, int adtype, int T, int c,
-                    int r, cudaStream_t stream) {
+// `src` null: no cached rows; `q` null: no queries.  q_rot rows (t, h) are rot_stride elements apart, q_plain rows
+// plain_stride (null: not wanted), each written with zeros up to rot_pad and plain_pad numbers.
+int mi_latent_rows(const float* src, int ld, int col0, const float* gain, float eps, const int* slot_mapping,
+                   void* cache, const float* q, int q_ld, int q_col0, void* q_plain, int plain_stride, int plain_pad,
+                   void* q_rot, int rot_stride, int rot_pad, const int* positions, const float* inv_freq,
+                   float magnitude, int adtype, int T, int H, int d, int r, int c, cudaStream_t stream) {
     if (T <= 0) return kOk;
-    if (c < 1 || r < 0 || r % 2 || col0 < 0 || col0 + c + r > ld || (r > 0 && !inv_freq)) {
-        set_last_error("latent_store: latent of %d and rotated part of %d at column %d of rows of %d", c, r, col0, ld);
+    if (c < 1 || r < 0 || r % 2 || (r > 0 && !inv_freq) || (!src && !q)) {
+        set_last_error("latent_rows: latent of %d and rotated part of %d", c, r);
         return kBadShape;
     }
-    MI_DISPATCH_1(adtype, AT,
-        launch_dependent(latent_store_kernel<AT>, dim3(T), dim3(256), 0, stream, src, ld, col0, positions, inv_freq,
-                         gain, eps, slot_mapping, (AT*)cache, c, r));
-    return finish_launch("latent_store");
-}
-
-int mi_latent_query(const float* q, const int* positions, const float* inv_freq, void* q_plain, void* q_full,
-                    int adtype, int T, int H, int d, int r, int c, cudaStream_t stream) {
-    if (T <= 0) return kOk;
-    if (H < 1 || d < 1 || r < 0 || r % 2 || c < 1 || (r > 0 && !inv_freq)) {
-        set_last_error("latent_query: %d heads of %d + %d, latent of %d", H, d, r, c);
+    if (src && (col0 < 0 || col0 + c + r > ld || !gain || !slot_mapping || !cache)) {
+        set_last_error("latent_rows: latent of %d and rotated part of %d at column %d of rows of %d", c, r, col0, ld);
         return kBadShape;
     }
+    if (q && (H < 1 || d < 1 || q_col0 < 0 || q_col0 + H * (d + r) > q_ld || (r > 0 && !q_rot) || rot_pad % 2 ||
+              rot_stride < (rot_pad > r ? rot_pad : r) || (q_plain && (plain_pad < d || plain_stride < plain_pad)))) {
+        set_last_error("latent_rows: %d heads of %d + %d at column %d of rows of %d", H, d, r, q_col0, q_ld);
+        return kBadShape;
+    }
+    const LatentStoreArgs st = {src, ld, col0, gain, eps, slot_mapping, cache};
+    const LatentQueryArgs qa = {q, q_ld, q_col0, q_plain, q_rot, plain_stride, rot_stride, plain_pad, rot_pad};
+    // a step of few tokens spreads a token's heads over several blocks
+    int by = 1;
+    if (q && T <= 32) by = H >= 16 ? 4 : (H >= 4 ? 2 : 1);
     MI_DISPATCH_1(adtype, AT,
-        launch_dependent(latent_query_kernel<AT>, dim3(T), dim3(256), 0, stream, q, positions, inv_freq,
-                         (AT*)q_plain, (AT*)q_full, H, d, r, c));
-    return finish_launch("latent_query");
+        launch_dependent(latent_rows_kernel<AT>, dim3(T, by), dim3(256), sizeof(float) * (r > 0 ? r : 1), stream, st,
+                         qa, positions, inv_freq, magnitude, H, d, r, c));
+    return finish_launch("latent_rows");
 }
 
 int mi_sigmoid_gate(const void* a, int64_t a_head, int64_t a_tok, const float* g, int ldg, int col0, void* out,

@@ -49,7 +49,7 @@ __device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit
 }
 
 // How the two halves of a gated unit meet in a product's epilogue: kind 0 silu(gate) * up, kind 1 the
-// bounded form above.  `row_scale` (or null): one number per row of the product's RESULT that multiplies both
+// bounded form above, kind 2 max(gate, 0) * up.  `row_scale` (or null): one number per row of the product's RESULT that multiplies both
 // halves before they meet, glu(s gate, s up): a product is linear in its input, so this is the gated unit of
 // the row s * x without a scaled copy of x (an expert whose weight multiplies what it reads).
 struct GluForm { int kind; float limit; float slope; const float* row_scale; };
@@ -57,6 +57,7 @@ __device__ __forceinline__ float glu_row_scale(const GluForm& f, int64_t row) {
     return f.row_scale ? __ldg(f.row_scale + row) : 1.0f;
 }
 __device__ __forceinline__ float glu_join(float gate, float up, GluForm f) {
+    if (f.kind == 2) return fmaxf(gate, 0.f) * up;
     return f.kind == 1 ? clamped_glu_f(gate, up, f.limit, f.slope) : gate / (1.0f + expf(-gate)) * up;
 }
 
@@ -67,6 +68,7 @@ __device__ __forceinline__ float glu_join_fast(float gate, float up, GluForm f) 
         const float u = fminf(fmaxf(up, -f.limit), f.limit);
         return __fdividef(g, 1.0f + __expf(-f.slope * g)) * (u + 1.0f);
     }
+    if (f.kind == 2) return fmaxf(gate, 0.f) * up;
     return __fdividef(gate, 1.0f + __expf(-gate)) * up;
 }
 

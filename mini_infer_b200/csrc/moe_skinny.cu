@@ -265,9 +265,9 @@ __device__ __forceinline__ void splitk_tile(const __nv_bfloat16* __restrict__ A,
 template <int MODE, int NT>
 __global__ void __launch_bounds__(256)
 dense_skinny_kernel(const __nv_bfloat16* __restrict__ A, const __nv_bfloat16* __restrict__ W,
-                    const float* __restrict__ bias, void* __restrict__ C, int rows, int Nout, int Kd) {
+                    const float* __restrict__ bias, void* __restrict__ C, int rows, int Nout, int Kd, GluForm glu) {
     wait_for_earlier_kernels();
-    splitk_tile<MODE, NT>(A, nullptr, nullptr, W, bias, C, rows, blockIdx.x * 16, Nout, Kd);
+    splitk_tile<MODE, NT>(A, nullptr, nullptr, W, bias, C, rows, blockIdx.x * 16, Nout, Kd, glu);
 }
 
 // The same with 32 warps to a block, for products with so few output features that their tiles do not
@@ -511,7 +511,7 @@ int mi_grouped_gemm_skinny_pairs(const void* A, const int* topk_idx, const void*
 int mi_dense_skinny_max_rows() { return 32; }
 
 // C = A @ W^T (+ bias) for rows <= 32.  A [rows, Kd], W [Nout (mode 0) or 2*Nout (mode 1), Kd] bfloat16;
-// bias float or null; C float [rows, Nout] (mode 0) or bfloat16 silu(gate)*up (mode 1).
+// bias float or null; C float [rows, Nout] (mode 0), bfloat16 silu(gate)*up (mode 1) or max(gate, 0)*up (mode 2).
 int mi_dense_skinny(const void* A, const void* W, const float* bias, void* C, int rows, int Nout, int Kd,
                     int mode, cudaStream_t stream) {
     if (Kd <= 0 || Kd % 32 != 0) {
@@ -546,8 +546,9 @@ int mi_dense_skinny(const void* A, const void* W, const float* bias, void* C, in
                              c + (int64_t)16 * Nout, rows - 16, Nout, Kd);
         return finish_launch("dense_skinny", rows > 16 ? 2 : 1);
     }
-#define MI_DENSE_SKINNY(MODE, NT) launch_dependent(dense_skinny_kernel<MODE, NT>, grid, block, 0, stream, a, w, bias, C, rows, Nout, Kd)
-    if (mode == 1) {
+#define MI_DENSE_SKINNY(MODE, NT) launch_dependent(dense_skinny_kernel<MODE, NT>, grid, block, 0, stream, a, w, bias, C, rows, Nout, Kd, glu)
+    const GluForm glu = {mode == 2 ? 2 : 0, 0.f, 0.f, nullptr};
+    if (mode >= 1) {
         if (rows <= 8) MI_DENSE_SKINNY(1, 1);
         else if (rows <= 16) MI_DENSE_SKINNY(1, 2);
         else MI_DENSE_SKINNY(1, 4);

@@ -19,7 +19,7 @@ from ..cache.manager import plan_groups
 from ..ops import functional as F
 from ..config.registry import part_class
 from ..config.spec import LayerSpec, ModelSpec, PartSpec
-from ..parts.base import (BuiltLayer, CacheBinding, PagedCacheNeed, Part, Runtime, StateNeed, StepContext,
+from ..parts.base import (BuiltLayer, CacheBinding, Deferred, PagedCacheNeed, Part, Runtime, StateNeed, StepContext,
                           TensorDecl, apply_norm, resolve)
 
 
@@ -58,6 +58,11 @@ class Model:
         # is called after every schedule entry of an eager forward pass (the reference's counterpart is
         # debug_print_tensor, src/model/transformer_model.cpp:24-61)
         self.layer_observer = None
+        streams = getattr(self.embedding, "streams", 1)
+        for layer in self.layers:
+            if getattr(layer.block, "streams", 1) != streams:
+                raise ValueError(f"layer '{layer.name}' works on {getattr(layer.block, 'streams', 1)} residual streams, "
+                                 f"the embedding starts {streams}")
         self._keeps_embedding_output = any(getattr(l.block, "needs_embedding_output", False) for l in self.layers)
         self._plan_caches()
 
@@ -70,6 +75,12 @@ class Model:
         paged: List[Tuple[Tuple[int, str], PagedCacheNeed]] = []
         self.state_needs: List[Tuple[Tuple[int, str], StateNeed]] = []
         needs: List[Dict[str, object]] = []
+        embedding_owner = (-1, "embedding")
+        need = getattr(self.embedding, "cache_need", lambda: None)()
+        if need is not None:
+            if not isinstance(need, PagedCacheNeed):
+                raise TypeError(f"embedding: cache_need() returned {type(need).__name__}; an embedding keeps pages only")
+            paged.append((embedding_owner, need))
         for pos, e in enumerate(self.spec.schedule):
             mine: Dict[str, object] = {}
             for role, part in self.layers[e.layer].parts.items():
@@ -100,6 +111,9 @@ class Model:
                 else:
                     self.state_needs.append(((pos, role), need))
         self.kv_groups, where = plan_groups(paged)
+        self.embedding_binding = None
+        if embedding_owner in where:
+            self.embedding_binding = CacheBinding("kv", *where[embedding_owner], True)
         state_index = {owner: i for i, (owner, _) in enumerate(self.state_needs)}
         self.bindings: List[Dict[str, CacheBinding]] = []
         for pos, e in enumerate(self.spec.schedule):
@@ -182,7 +196,7 @@ class Model:
         return self._forward(ctx, logit_rows)
 
     def _forward(self, ctx: StepContext, logit_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
-        hidden = self.embedding.forward(ctx.token_ids)
+        hidden = self.embedding.forward_step(ctx, self.embedding_binding)
         ctx.carried.clear()
         if self._keeps_embedding_output:
             ctx.embedding_output = hidden.clone()       # the residual stream is updated in place from here on
@@ -202,8 +216,10 @@ class Model:
             pending = layer.block.forward(layer, hidden, pending, ctx, self.bindings[pos])
             if self.layer_observer is not None:
                 # the addition of a part's output is left to the next norm's kernel; form it here
-                left = resolve(pending)
-                self.layer_observer(pos, hidden if left is None else hidden + left)
+                if isinstance(pending, Deferred):
+                    self.layer_observer(pos, pending.residual(hidden))
+                else:
+                    self.layer_observer(pos, hidden if pending is None else hidden + pending)
         if ctx.prefetch is not None:
             ctx.prefetch.join()
         ctx.carried.clear()

@@ -800,12 +800,12 @@ def dense_skinny_takes(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def dense_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                 swiglu_pair: bool = False) -> torch.Tensor:
+                 swiglu_pair: bool = False, activation: str = "silu") -> torch.Tensor:
     """``x @ w.T (+ bias)`` for a step of a few tokens (decode), every weight read once.
 
     ``x`` [T, K] and ``w`` [N, K] bfloat16, ``bias`` float32 [N] or None.  Returns float32
     [T, N]; with ``swiglu_pair`` the rows of ``w`` are N/2 gate rows then N/2 up rows and the
-    result is ``silu(gate) * up`` as bfloat16 [T, N/2].
+    result is ``silu(gate) * up`` (``activation`` ``relu``: ``max(gate, 0) * up``) as bfloat16 [T, N/2].
     """
     _chk(x, "dense_skinny x", BF16)
     T, Kd = x.shape
@@ -818,7 +818,8 @@ def dense_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
         _chk(bias, "dense_skinny bias", F32, (wrows,))
     out = torch.empty(T, nout, dtype=BF16 if swiglu_pair else F32, device=x.device)
     check(library().mi_dense_skinny(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), T, nout, Kd,
-                                    1 if swiglu_pair else 0, _stream()), "dense_skinny")
+                                    {"silu": 1, "relu": 2}[activation] if swiglu_pair else 0, _stream()),
+          "dense_skinny")
     return out
 
 
@@ -1634,42 +1635,78 @@ def dense_f32_heads(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor
     return out
 
 
+def latent_rows(positions: torch.Tensor, inv_freq: Optional[torch.Tensor], rank: int, rot_dim: int, store=None,
+                query=None, magnitude: float = 1.0) -> None:
+    """Row-wise work of attention through a latent, one launch for whichever of the two is given.  ``magnitude``
+    multiplies the cosines and sines of the rotation, which pairs neighbours.
+
+    ``store = (src, col0, gain, eps, slot_mapping, cache)``: columns ``col0 .. col0 + rank`` of the float32 rows
+    ``src`` divided by their root mean square (``eps`` inside the root) times ``gain``, then ``rot_dim`` columns
+    rotated by position, into ``cache [pages, 1, page_size, rank + rot_dim]`` (slot -1: not written).
+
+    ``query = (q, col0, heads, dim, q_plain, plain_pad, q_rot, rot_offset, rot_pad)``: from column ``col0`` of the
+    float32 rows ``q``, ``heads`` queries ``[dim unrotated | rot_dim rotated]``.  The unrotated parts go to the first
+    columns of ``q_plain [T, heads, *]`` (None: not wanted), zeros following up to ``plain_pad`` columns; the rotated
+    ones to the columns from ``rot_offset`` of ``q_rot [T, heads, *]``, zeros following up to ``rot_pad``."""
+    T = positions.numel()
+    _chk(positions, "latent_rows positions", I32, (T,))
+    _chk(inv_freq, "latent_rows inv_freq", F32, (rot_dim // 2,))
+    st = [None, 0, 0, None, 0.0, None, None]
+    qa = [None, 0, 0, None, 0, 0, None, 0, 0]
+    heads = dim = 0
+    code = None
+    if store is not None:
+        src, col0, gain, eps, slots, cache = store
+        _chk(src, "latent_rows src", F32, (T, None))
+        _chk(gain, "latent_rows gain", F32, (rank,))
+        _chk(slots, "latent_rows slot_mapping", I32, (T,))
+        _chk(cache, "latent_rows cache", None, (None, 1, None, rank + rot_dim))
+        if DEBUG_BOUNDS:
+            _dbg_range(slots, -1, cache.shape[0] * cache.shape[2], "latent_rows slot_mapping")
+        st = [_ptr(src), src.shape[1], int(col0), _ptr(gain), float(eps), _ptr(slots), _ptr(cache)]
+        code = _code(cache, "latent_rows cache")
+    if query is not None:
+        q, qcol, heads, dim, q_plain, plain_pad, q_rot, rot_offset, rot_pad = query
+        _chk(q, "latent_rows q", F32, (T, None))
+        _chk(q_plain, "latent_rows q_plain", None, (T, heads, None))
+        _chk(q_rot, "latent_rows q_rot", None, (T, heads, None))
+        qcode = _code(q_rot, "latent_rows q_rot")
+        if (code is not None and code != qcode) or (q_plain is not None and _code(q_plain, "latent_rows q_plain") != qcode):
+            raise TypeError("latent_rows: cache and queries are of different types")
+        code = qcode
+        if rot_offset + max(rot_pad, rot_dim) > q_rot.shape[2]:
+            raise ValueError("latent_rows: the rotated parts do not fit their rows")
+        plain_pad = max(int(plain_pad), dim)
+        if q_plain is not None and plain_pad > q_plain.shape[2]:
+            raise ValueError("latent_rows: the unrotated parts do not fit their rows")
+        if q_plain is not None and q_plain is q_rot and plain_pad > rot_offset:
+            raise ValueError("latent_rows: unrotated and rotated parts overlap")
+        qa = [_ptr(q), q.shape[1], int(qcol), _ptr(q_plain), q_plain.shape[2] if q_plain is not None else 0, plain_pad,
+              q_rot.data_ptr() + rot_offset * q_rot.element_size(), q_rot.shape[2], int(rot_pad)]
+    check(library().mi_latent_rows(*st, *qa, _ptr(positions), _ptr(inv_freq), float(magnitude), code, T, int(heads),
+                                   int(dim), int(rot_dim), int(rank), _stream()), "latent_rows")
+
+
 def latent_store(src: torch.Tensor, col0: int, positions: torch.Tensor, inv_freq: Optional[torch.Tensor],
                  gain: torch.Tensor, eps: float, slot_mapping: torch.Tensor, cache: torch.Tensor, rank: int,
-                 rot_dim: int) -> None:
-    """The cached row of every token: columns ``col0 .. col0 + rank`` of the float32 rows ``src`` divided by
-    their root mean square (``eps`` inside the root) times ``gain``, then ``rot_dim`` columns rotated by
-    position in pairs of neighbours.  ``cache [pages, 1, page_size, rank + rot_dim]``; slot -1: not written."""
-    _chk(src, "latent_store src", F32)
-    T, ld = src.shape
-    _chk(positions, "latent_store positions", I32, (T,))
-    _chk(inv_freq, "latent_store inv_freq", F32, (rot_dim // 2,))
-    _chk(gain, "latent_store gain", F32, (rank,))
-    _chk(slot_mapping, "latent_store slot_mapping", I32, (T,))
-    _chk(cache, "latent_store cache", None, (None, 1, None, rank + rot_dim))
-    if DEBUG_BOUNDS:
-        _dbg_range(slot_mapping, -1, cache.shape[0] * cache.shape[2], "latent_store slot_mapping")
-    check(library().mi_latent_store(_ptr(src), ld, int(col0), _ptr(positions), _ptr(inv_freq), _ptr(gain), float(eps),
-                                    _ptr(slot_mapping), _ptr(cache), _code(cache, "latent_store cache"), T, int(rank),
-                                    int(rot_dim), _stream()), "latent_store")
+                 rot_dim: int, magnitude: float = 1.0) -> None:
+    """The cached row of every token (:func:`latent_rows` without queries)."""
+    latent_rows(positions, inv_freq, rank, rot_dim, store=(src, col0, gain, eps, slot_mapping, cache),
+                magnitude=magnitude)
 
 
 def latent_query(q: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[torch.Tensor], heads: int, dim: int,
-                 rot_dim: int, rank: int, out_dtype: torch.dtype, want_plain: bool):
-    """Float32 rows of ``heads`` queries ``[dim unrotated | rot_dim rotated]``: returns ``(q_full, q_plain)``
-    where ``q_full [T, heads, rank + rot_dim]`` (``out_dtype``) has its last ``rot_dim`` columns filled with the
-    parts rotated by position (pairs of neighbours; the first ``rank`` are left for the folded queries) and
-    ``q_plain [T, heads, dim]`` holds the unrotated parts in ``out_dtype`` (None unless wanted)."""
-    _chk(q, "latent_query q", F32)
-    T = q.shape[0]
-    _chk(q, "latent_query q", F32, (T, heads * (dim + rot_dim)))
-    _chk(positions, "latent_query positions", I32, (T,))
-    _chk(inv_freq, "latent_query inv_freq", F32, (rot_dim // 2,))
+                 rot_dim: int, rank: int, out_dtype: torch.dtype, want_plain: bool, col0: int = 0,
+                 magnitude: float = 1.0, store=None):
+    """Queries of the folded form (:func:`latent_rows`): returns ``(q_full, q_plain)`` where ``q_full [T, heads,
+    rank + rot_dim]`` (``out_dtype``) has its last ``rot_dim`` columns filled with the rotated parts (the first
+    ``rank`` are left for the folded queries) and ``q_plain [T, heads, dim]`` holds the unrotated parts (None unless
+    wanted).  ``store``: the cached rows of the same launch."""
+    T = positions.numel()
     q_full = torch.empty(T, heads, rank + rot_dim, dtype=out_dtype, device=q.device)
     q_plain = torch.empty(T, heads, dim, dtype=out_dtype, device=q.device) if want_plain else None
-    check(library().mi_latent_query(_ptr(q), _ptr(positions), _ptr(inv_freq), _ptr(q_plain), _ptr(q_full),
-                                    _code(q_full, "latent_query out"), T, heads, dim, rot_dim, rank, _stream()),
-          "latent_query")
+    latent_rows(positions, inv_freq, rank, rot_dim, store=store,
+                query=(q, col0, heads, dim, q_plain, dim, q_full, rank, rot_dim), magnitude=magnitude)
     return q_full, q_plain
 
 
@@ -1685,4 +1722,101 @@ def sigmoid_gate(a: torch.Tensor, head_major: bool, g: torch.Tensor, col0: int, 
     a_head, a_tok = (T * size, size) if head_major else (size, heads * size)
     check(library().mi_sigmoid_gate(_ptr(a), a_head, a_tok, _ptr(g), g.shape[1], int(col0), _ptr(out),
                                     _code(a, "sigmoid_gate a"), T, heads, size, _stream()), "sigmoid_gate")
+    return out
+
+
+# --------------------------------------------------------------------------- #
+# a residual of several streams
+# --------------------------------------------------------------------------- #
+
+def streams_embed(ids: torch.Tensor, table: torch.Tensor, scale: float, streams: int, norm=None, bigram=None,
+                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``norm(table[ids] * scale + second[row])`` written ``streams`` times: float32 ``[T, streams, H]``.
+
+    ``norm = (weight, eps)`` or None.  ``bigram = (second, buckets, mul_prev, mul_cur, positions, req_of_token,
+    token_ids, block_table, slot_mapping)`` or None: ``second [buckets + 1, H]``, ``row = (previous token * mul_prev +
+    token * mul_cur) mod buckets``, at position 0 the last row; the previous token of a portion's first token comes
+    from ``token_ids [pages, page_size]`` (int32), into which the ids of this step are written at ``slot_mapping``."""
+    _chk(ids, "streams_embed ids", I32)
+    _chk(table, "streams_embed table")
+    T = ids.numel()
+    V, H = table.shape
+    if out is None:
+        out = torch.empty(T, int(streams), H, dtype=F32, device=table.device)
+    _chk(out, "streams_embed out", F32, (T, int(streams), H))
+    if DEBUG_BOUNDS:
+        _dbg_range(ids, 0, V, "streams_embed ids")
+    weight, eps = norm if norm is not None else (None, 0.0)
+    _chk(weight, "streams_embed norm weight", None, (H,))
+    args = [None, 0, 0, 0, None, None, None, 0, 0]
+    positions = req = None
+    if bigram is not None:
+        second, buckets, mp, mc, positions, req, token_ids, bt, slots = bigram
+        _chk(second, "streams_embed second table", table.dtype, (int(buckets) + 1, H))
+        _chk(positions, "streams_embed positions", I32, (T,))
+        _chk(req, "streams_embed req_of_token", I32, (T,))
+        _chk(token_ids, "streams_embed token_ids", I32)
+        _chk(bt, "streams_embed block_table", I32)
+        _chk(slots, "streams_embed slot_mapping", I32, (T,))
+        if DEBUG_BOUNDS:
+            _dbg_range(slots, -1, token_ids.numel(), "streams_embed slot_mapping")
+            _dbg_range(req, 0, bt.shape[0], "streams_embed req_of_token")
+            _dbg_range(bt, -1, token_ids.shape[0], "streams_embed block_table")
+        args = [_ptr(second), int(buckets), int(mp), int(mc), _ptr(token_ids), _ptr(bt), _ptr(slots), bt.shape[1],
+                token_ids.shape[1]]
+    check(library().mi_streams_embed(
+        _ptr(ids), _ptr(positions), _ptr(req), _ptr(table), _code(table, "streams_embed table"), float(scale), *args,
+        _ptr(weight), _code(weight, "streams_embed norm weight") if weight is not None else 0, float(eps), _ptr(out), T,
+        H, V, int(streams), _stream()), "streams_embed")
+    return out
+
+
+def _chk_streams(xs, y, mix, w_out, what):
+    _chk(xs, what + " streams", F32)
+    T, S, H = xs.shape
+    _chk(y, what + " y", F32, (T, H))
+    _chk(mix, what + " mix", F32, (S, S))
+    _chk(w_out, what + " out weights", F32, (S,))
+    return T, S, H
+
+
+def streams_read(xs: torch.Tensor, pending, w_in: torch.Tensor, weight: torch.Tensor, eps: float,
+                 out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``pending = (y, mix, w_out)`` or None: ``x_t <- sum_s mix[s, t] x_s + w_out[t] y`` on the streams ``xs
+    [T, S, H]`` (float32, in place); then the RMS norm of ``sum_t w_in[t] x_t`` in ``out_dtype``.  With ``rows``
+    (int32) only those rows are formed and ``xs`` is left as it is."""
+    y, mix, w_out = pending if pending is not None else (None, None, None)
+    T, S, H = _chk_streams(xs, y, mix, w_out, "streams_read")
+    _chk(w_in, "streams_read in weights", F32, (S,))
+    _chk(weight, "streams_read norm weight", None, (H,))
+    _chk(rows, "streams_read rows", I32)
+    n = T if rows is None else rows.numel()
+    if DEBUG_BOUNDS:
+        _dbg_range(rows, 0, T, "streams_read rows")
+    out = torch.empty(n, H, dtype=out_dtype, device=xs.device)
+    check(library().mi_streams_read(_ptr(xs), _ptr(y), _ptr(mix), _ptr(w_out), _ptr(w_in), _ptr(rows), _ptr(weight),
+                                    _code(weight, "streams_read norm weight"), _ptr(out), _code(out, "streams_read out"),
+                                    n, S, H, float(eps), _stream()), "streams_read")
+    return out
+
+
+def streams_sum(xs: torch.Tensor, pending=None) -> torch.Tensor:
+    """The sum of the streams after the pending update (:func:`streams_read`), float32 ``[T, H]``; ``xs`` is left as
+    it is."""
+    y, mix, w_out = pending if pending is not None else (None, None, None)
+    T, S, H = _chk_streams(xs, y, mix, w_out, "streams_sum")
+    out = torch.empty(T, H, dtype=F32, device=xs.device)
+    check(library().mi_streams_sum(_ptr(xs), _ptr(y), _ptr(mix), _ptr(w_out), _ptr(out), T, S, H, _stream()),
+          "streams_sum")
+    return out
+
+
+def relu_glu(gu: torch.Tensor) -> torch.Tensor:
+    """``max(gu[:, :I], 0) * gu[:, I:]`` in the type of ``gu``."""
+    _chk(gu, "relu_glu gu")
+    T, two_i = gu.shape
+    if two_i % 2:
+        raise ValueError("relu_glu: the row holds gate and up halves of equal size")
+    out = torch.empty(T, two_i // 2, dtype=gu.dtype, device=gu.device)
+    check(library().mi_relu_glu(_ptr(gu), _ptr(out), _code(gu, "relu_glu gu"), T, two_i // 2, _stream()), "relu_glu")
     return out

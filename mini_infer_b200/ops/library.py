@@ -66,8 +66,11 @@ _SIGNATURES = {
     "mi_attn_prefill_tc_shared": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
     "mi_clamped_glu": [P, P, I, L, I, F, F, P],
     "mi_dense_f32_batched": [P, P, P, I, I, I, I, I, I, L, L, L, P],
-    "mi_latent_store": [P, I, I, P, P, P, F, P, P, I, I, I, I, P],
-    "mi_latent_query": [P, P, P, P, P, I, I, I, I, I, I, P],
+    "mi_latent_rows": [P, I, I, P, F, P, P, P, I, I, P, I, I, P, I, I, P, P, F, I, I, I, I, I, I, P],
+    "mi_streams_embed": [P, P, P, P, I, F, P, L, L, L, P, P, P, I, I, P, I, F, P, I, I, I, I, P],
+    "mi_streams_read": [P, P, P, P, P, P, P, I, P, I, I, I, I, F, P],
+    "mi_streams_sum": [P, P, P, P, P, I, I, I, P],
+    "mi_relu_glu": [P, P, I, L, I, P],
     "mi_sigmoid_gate": [P, L, L, P, I, I, P, I, I, I, I, P],
     "mi_causal_conv_residual": [P, I, P, I, P, L, P, P, P, P, I, I, I, I, I, I, P],
     "mi_norm_conv_decode": [P, P, I, F, P, P, L, P, P, P, I, I, I, I, P],

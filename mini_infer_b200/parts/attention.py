@@ -78,6 +78,8 @@ class GQAttention(Mixer):
             self.b_qkv = torch.cat(bs, dim=0).contiguous()
         self.w_o = prec.matrix(tensors[f"{self.prefix}o_proj.weight"], dev)
         self.inv_freq = self.position.table(dev)
+        if self.position.magnitude != 1.0:
+            raise ValueError("attention: a rotation that also stretches its pairs is not built for this mixer")
         if getattr(self.position, "pairing", "halves") != "halves":
             raise ValueError("attention: this part's kernels rotate by halves; a rotation of neighbouring "
                              "dimensions belongs to 'head_mix_attention'")

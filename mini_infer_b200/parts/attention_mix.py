@@ -136,6 +136,8 @@ class HeadMixAttention(Mixer):
         self.head_bias = tensors[n["head_bias"]].to(device=dev, dtype=torch.float32).contiguous() if self.logistic else None
         self.w_gate = m(tensors[n["gate"]], dev) if self.output_gate else None
         self.inv_freq = self.position.table(dev)
+        if self.position.magnitude != 1.0:
+            raise ValueError("head_mix_attention: a rotation that also stretches its pairs is not built for this mixer")
         self.rot_dim = self.position.rot_dim if self.inv_freq is not None else 0
         self.neighbours = getattr(self.position, "pairing", "halves") == "neighbours"
         # the blending weight joins float arithmetic (the first layer of a blend has none to apply)

@@ -18,7 +18,8 @@ Categories and what each must provide:
 ``feed_forward``  ``forward(x, ctx) -> y``, same shapes.
 ``block``         ``forward(layer, hidden, pending, ctx, cache) -> pending``: the
                   arrangement of norms, mixer and feed-forward around the residual.
-``embedding``     ``forward(token_ids) -> hidden`` float32.
+``embedding``     ``forward(token_ids) -> hidden`` float32, or ``forward_step(ctx, cache)`` for one that reads more
+                  of the step than its token ids (it may then keep something per token: ``cache_need()``).
 ``lm_head``       ``forward(x) -> logits`` float32.
 """
 
@@ -117,7 +118,7 @@ def configure_matmul_exactness() -> None:
 # what a part keeps between steps: see cache/needs.py
 # --------------------------------------------------------------------------- #
 
-from ..cache.needs import KVNeed, LatentNeed, PagedCacheNeed, StateNeed  # noqa: E402  (re-exported for part authors)
+from ..cache.needs import KVNeed, LatentNeed, PagedCacheNeed, StateNeed, TokenNeed  # noqa: E402  (re-exported for part authors)
 
 
 # --------------------------------------------------------------------------- #
@@ -255,6 +256,11 @@ class Deferred:
     def materialize(self) -> torch.Tensor:
         raise NotImplementedError
 
+    def residual(self, hidden: torch.Tensor) -> torch.Tensor:
+        """The residual stream ``[T, H]`` with this output in it (``hidden`` is left as it is)."""
+        left = self.materialize()
+        return hidden if left is None else hidden + left
+
 
 @dataclass
 class WeightedRowSum(Deferred):
@@ -296,6 +302,54 @@ class RoundedResidual(Deferred):
         return None
 
 
+@dataclass
+class StreamUpdate(Deferred):
+    """A residual of several streams ``x_s`` (``hidden [T, S, H]``) whose last sublayer's output ``y`` has not been
+    taken in yet: ``x_t <- sum_s mix[s, t] x_s + w_out[t] y``.  Only a consumer that knows the streams can take it
+    (:func:`read_streams`); what a reader of one row per token sees is the streams' sum."""
+
+    y: Any
+    mix: torch.Tensor
+    w_out: torch.Tensor
+
+    def parts(self):
+        return resolve(self.y), self.mix, self.w_out
+
+    def materialize(self) -> torch.Tensor:
+        raise TypeError("an update of several residual streams cannot be added to one of them")
+
+    def residual(self, hidden: torch.Tensor) -> torch.Tensor:
+        from ..ops import functional as F
+        return F.streams_sum(as_streams(hidden), self.parts())
+
+
+def as_streams(hidden: torch.Tensor) -> torch.Tensor:
+    """``[T, S, H]``: one row per token is one stream."""
+    return hidden if hidden.dim() == 3 else hidden.unsqueeze(1)
+
+
+_ONES: Dict[tuple, torch.Tensor] = {}
+
+
+def _stream_ones(n: int, device) -> torch.Tensor:
+    """Weights of one for the sum of ``n`` streams (kept: captured passes read the tensor they were captured with)."""
+    key = (int(n), str(device))
+    if key not in _ONES:
+        _ONES[key] = torch.ones(n, dtype=torch.float32, device=device)
+    return _ONES[key]
+
+
+def read_streams(hidden: torch.Tensor, pending, w_in: torch.Tensor, norm: "Norm",
+                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``norm(sum_t w_in[t] x_t)`` of the streams ``hidden [T, S, H]`` after their pending update (None, or a
+    :class:`StreamUpdate`, which is carried out on ``hidden`` unless ``rows`` selects rows): one kernel."""
+    from ..ops import functional as F
+    rms = norm.rms_parameters()
+    if rms is None:
+        raise ValueError("a norm of combined residual streams must be a plain RMS norm")
+    return F.streams_read(hidden, None if pending is None else pending.parts(), w_in, rms[0], rms[1], norm.rt.act, rows)
+
+
 def split_sum(pending):
     """``(a, b)`` with ``pending = a + b`` (either may be None) for a consumer whose kernel adds up to two
     pending tensors itself."""
@@ -325,7 +379,11 @@ class Norm(Part):
 
 
 def apply_norm(norm: "Norm", hidden: torch.Tensor, pending, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``norm.apply`` with a pending output that may be deferred."""
+    """``norm.apply`` with a pending output that may be deferred.  (``hidden`` of several streams, ``[T, S, H]``:
+    what is normalised is their sum.)"""
+    if hidden.dim() == 3 or isinstance(pending, StreamUpdate):
+        hidden = as_streams(hidden)
+        return read_streams(hidden, pending, _stream_ones(hidden.shape[1], hidden.device), norm, rows)
     if isinstance(pending, Deferred) and not norm.accepts_deferred:
         pending = pending.materialize()
     return norm.apply(hidden, pending, rows)
@@ -334,6 +392,7 @@ def apply_norm(norm: "Norm", hidden: torch.Tensor, pending, rows: Optional[torch
 class PositionEncoding(Part):
     category = "position"
     rot_dim = 0
+    magnitude = 1.0             # multiplies cosines and sines (a mixer that cannot apply it refuses another value)
 
     def table(self, device) -> Optional[torch.Tensor]:
         return None
@@ -367,9 +426,16 @@ class FeedForward(Part):
 
 class Embedding(Part):
     category = "embedding"
+    streams = 1                 # how many copies of its output the residual starts as: hidden [T, streams, H] above 1
+
+    def cache_need(self):
+        return None
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
+
+    def forward_step(self, ctx: StepContext, cache: Optional[CacheBinding]) -> torch.Tensor:
+        return self.forward(ctx.token_ids)
 
 
 class LMHead(Part):
@@ -390,6 +456,7 @@ class Block(Part):
 
     category = "block"
     accepts_deferred = False    # True: ``forward`` takes a Deferred as ``pending`` and may return one
+    streams = 1                 # parallel residual streams the arrangement works on (``hidden [T, streams, H]`` above 1)
     roles: Mapping[str, str] = {}
 
     def forward(self, layer: "BuiltLayer", hidden: torch.Tensor, pending: Optional[torch.Tensor],
@@ -422,13 +489,16 @@ class BuiltLayer:
 from .tuning import TUNING  # noqa: E402
 
 
-def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act_dtype: torch.dtype) -> torch.Tensor:
-    """``silu(x @ w_gate.T) * (x @ w_up.T)`` in the activation dtype; ``w_gate_up`` holds the gate
-    rows then the up rows (src/layers/mlp.cpp:255-279 runs two products and an elementwise kernel)."""
+def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act_dtype: torch.dtype,
+                  activation: str = "silu") -> torch.Tensor:
+    """``silu(x @ w_gate.T) * (x @ w_up.T)`` in the activation dtype (``activation`` ``relu``: a rectified gate);
+    ``w_gate_up`` holds the gate rows then the up rows (src/layers/mlp.cpp:255-279 runs two products and an
+    elementwise kernel)."""
     from ..ops import functional as F
     if x.is_cuda and x.shape[0] <= TUNING.dense_skinny_max_tokens and F.dense_skinny_takes(x, w_gate_up):
-        return F.dense_skinny(x, w_gate_up, swiglu_pair=True)
-    return F.swiglu(linear(x, w_gate_up, act_dtype))
+        return F.dense_skinny(x, w_gate_up, swiglu_pair=True, activation=activation)
+    gu = linear(x, w_gate_up, act_dtype)
+    return F.relu_glu(gu) if activation == "relu" else F.swiglu(gu)
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:

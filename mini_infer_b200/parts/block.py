@@ -19,7 +19,8 @@ from ..config.registry import part_class, register_part
 from ..ops import functional as F
 from .tuning import TUNING
 from .base import (Block, BuiltLayer, CacheBinding, Embedding, LMHead, RoundedResidual, Runtime, StepContext,
-                   TensorDecl, TensorSum, WeightedRowSum, apply_norm, linear, resolve, split_sum)
+                   StreamUpdate, TensorDecl, TensorSum, TokenNeed, WeightedRowSum, apply_norm, as_streams, linear,
+                   read_streams, resolve, split_sum)
 
 
 class PreNormResidual(Block):
@@ -40,9 +41,19 @@ class TokenEmbedding(Embedding):
     """params: ``vocab_size``, ``hidden_size``, optional ``tensor`` (the tensor's name below the prefix,
     default ``weight``) and ``norm`` (a ``PartSpec`` of category ``norm`` whose ``rms_parameters()`` are
     applied to every gathered row before it becomes the residual stream, which stays float32).
-    Tensor: ``<prefix>weight [V, H]``; no scaling (src/model/transformer_model.cpp:561-565)."""
+    Tensor: ``<prefix>weight [V, H]``; no scaling by default (src/model/transformer_model.cpp:561-565).
+
+    Further params, taken together by one kernel: ``scale`` (multiplies the gathered row, default 1); ``bigram``
+    (``{"tensor", "buckets", "mul_prev", "mul_cur"}``: the row ``(previous token * mul_prev + token * mul_cur) mod
+    buckets`` of a second table ``[buckets + 1, H]`` is added to it, for a sequence's first token the table's last row;
+    the previous token is kept in a paged cache of token ids behind a window of two); ``streams`` (the result is
+    written that many times, ``[T, streams, H]``, for an arrangement of parallel residual streams)."""
 
     graph_safe = True
+
+    @property
+    def kernel_files(self):
+        return ("residual_streams.cu",) if self._fused else ("elementwise.cu",)
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -50,12 +61,22 @@ class TokenEmbedding(Embedding):
         spec = self.params.get("norm")
         if spec is not None:
             self.norm = part_class("norm", spec.kind)(spec.params, prefix)
+        self.scale = float(self.params.get("scale", 1.0))
+        self.streams = int(self.params.get("streams", 1))
+        self.bigram = self.params.get("bigram")
+        self._fused = self.scale != 1.0 or self.streams != 1 or self.bigram is not None
 
     def _name(self) -> str:
         return self.prefix + self.params.get("tensor", "weight")
 
+    def cache_need(self):
+        return TokenNeed(window=2) if self.bigram is not None else None
+
     def tensor_decls(self) -> List[TensorDecl]:
         out = [TensorDecl(self._name(), (self.params["vocab_size"], self.params["hidden_size"]))]
+        if self.bigram is not None:
+            out.append(TensorDecl(self.prefix + self.bigram["tensor"],
+                                  (int(self.bigram["buckets"]) + 1, self.params["hidden_size"])))
         if self.norm is not None:
             out += self.norm.tensor_decls()
         return out
@@ -63,6 +84,8 @@ class TokenEmbedding(Embedding):
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.rt = rt
         self.weight = rt.precision.matrix(tensors[self._name()], rt.device)
+        if self.bigram is not None:
+            self.second = rt.precision.matrix(tensors[self.prefix + self.bigram["tensor"]], rt.device)
         if self.norm is not None:
             self.norm.load(tensors, rt)
             if self.norm.rms_parameters() is None:
@@ -74,6 +97,19 @@ class TokenEmbedding(Embedding):
             return hidden
         weight, eps = self.norm.rms_parameters()
         return F.add_rmsnorm(hidden, None, weight, eps, torch.float32)
+
+    def forward_step(self, ctx: StepContext, cache: Optional[CacheBinding]) -> torch.Tensor:
+        if not self._fused:
+            return self.forward(ctx.token_ids)
+        bigram = None
+        if self.bigram is not None:
+            view = ctx.kv_groups[cache.group]
+            bigram = (self.second, self.bigram["buckets"], self.bigram["mul_prev"], self.bigram["mul_cur"],
+                      ctx.positions, ctx.req_of_token, view.tensors["token"][cache.layer_slot], view.block_table,
+                      view.slot_mapping)
+        x = F.streams_embed(ctx.token_ids, self.weight, self.scale, self.streams,
+                            None if self.norm is None else self.norm.rms_parameters(), bigram)
+        return x if self.streams > 1 else x.view(x.shape[0], x.shape[2])
 
 
 class LinearHead(LMHead):
@@ -395,6 +431,62 @@ class ParallelResidual(Block):
         layer.mixer.prefetch_first(ctx, caches.get("mixer"))
 
 
+class HyperConnections(Block):
+    """Parallel residual streams ``x_1 .. x_S`` per token that every sublayer reads and writes through small matrices
+    of its own: ``u = sum_s in[s] x_s``, ``y = Part(Norm(u))``, then all streams at once from the old ones
+    ``x_t <- sum_s mix[s, t] x_s + out[t] y``; first around the mixer, then around the feed-forward.  The residual a
+    reader of one row per token sees is the streams' sum.
+
+    params: ``streams``, ``feed_forward`` (default True; False: a layer of a mixer alone, with the roles ``mixer_norm``
+    and ``mixer`` only), ``mixer_streams`` and ``feed_forward_streams`` (prefixes, below the layer's, of the tensors
+    ``in [S]``, ``out [S]`` and ``mix [S, S]`` of each sublayer).  The norms must be plain RMS norms.
+
+    A sublayer's output travels on as a :class:`StreamUpdate`; one kernel carries the update out, combines the streams
+    for the next sublayer and normalises, so the streams are read and written once per sublayer."""
+
+    graph_safe = True
+    accepts_deferred = True
+    kernel_files = ("residual_streams.cu",)
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        p = self.params
+        self.streams = int(p["streams"])
+        self.has_ff = bool(p.get("feed_forward", True))
+        self._names = {"mixer": prefix + p["mixer_streams"]}
+        self.roles = {"mixer_norm": "norm", "mixer": "mixer"}
+        if self.has_ff:
+            self._names["feed_forward"] = prefix + p["feed_forward_streams"]
+            self.roles.update({"feed_forward_norm": "norm", "feed_forward": "feed_forward"})
+
+    def tensor_decls(self) -> List[TensorDecl]:
+        S = self.streams
+        return [d for n in self._names.values() for d in (TensorDecl(n + "in", (S,), "stream"),
+                                                          TensorDecl(n + "out", (S,), "stream"),
+                                                          TensorDecl(n + "mix", (S, S), "stream"))]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        S = self.streams
+        f32 = lambda n, shape: tensors[n].to(device=rt.device, dtype=torch.float32).reshape(shape).contiguous()
+        self.weights = {part: (f32(n + "in", (S,)), f32(n + "mix", (S, S)), f32(n + "out", (S,)))
+                        for part, n in self._names.items()}
+
+    def forward(self, layer: BuiltLayer, hidden: torch.Tensor, pending, ctx: StepContext, caches):
+        xs = as_streams(hidden)
+        w_in, mix, w_out = self.weights["mixer"]
+        x = read_streams(xs, pending, w_in, layer.mixer_norm)
+        pending = StreamUpdate(layer.mixer.forward(x, ctx, caches.get("mixer")), mix, w_out)
+        if self.has_ff:
+            w_in, mix, w_out = self.weights["feed_forward"]
+            x = read_streams(xs, pending, w_in, layer.feed_forward_norm)
+            pending = StreamUpdate(layer.feed_forward.forward_deferred(x, ctx), mix, w_out)
+        return pending
+
+    def prefetch_layer(self, layer: BuiltLayer, ctx: StepContext, caches) -> None:
+        layer.mixer.prefetch_first(ctx, caches.get("mixer"))
+
+
 class StreamMerge(Block):
     """A run of no parts that re-enters the embedding into the residual stream:
     ``x <- W [x ; x0] + step[pass]`` with ``x0`` the embedding's output, ``W [H, 2H]`` (the columns of ``x``
@@ -431,6 +523,7 @@ register_part("block", "prenorm_residual", PreNormResidual)
 register_part("block", "parallel_residual", ParallelResidual)
 register_part("block", "output_norm_residual", OutputNormResidual)
 register_part("block", "sandwich_residual", SandwichResidual)
+register_part("block", "hyper_connections", HyperConnections)
 register_part("block", "stream_merge", StreamMerge)
 register_part("embedding", "token_embedding", TokenEmbedding)
 register_part("lm_head", "linear", LinearHead)

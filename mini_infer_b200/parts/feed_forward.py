@@ -55,7 +55,7 @@ class SwiGLUMLP(FeedForward):
 
 class GatedMLP(FeedForward):
     """``(act(x Wg^T) * (x Wu^T)) Wd^T`` with a choice of ``act``.  params: ``hidden_size``,
-    ``intermediate_size``, ``activation`` (``silu`` | ``gelu_tanh`` | ``clamped_swish``), optional ``gate``,
+    ``intermediate_size``, ``activation`` (``silu`` | ``relu`` | ``gelu_tanh`` | ``clamped_swish``), optional ``gate``,
     ``up``, ``down`` (tensor names below the prefix; default ``gate_proj.weight`` and so on).
 
     ``clamped_swish`` (params ``limit`` and optionally ``slope``, default 1.702) bounds both halves before
@@ -65,8 +65,11 @@ class GatedMLP(FeedForward):
     Tensors: ``<prefix><gate>, <prefix><up> [I, H]``, ``<prefix><down> [H, I]``."""
 
     graph_safe = True
-    kernel_files = ("elementwise.cu", "moe_skinny.cu", "residual_forms.cu")
-    ACTIVATIONS = ("silu", "gelu_tanh", "clamped_swish")
+    ACTIVATIONS = ("silu", "relu", "gelu_tanh", "clamped_swish")
+
+    @property
+    def kernel_files(self):
+        return ("elementwise.cu", "moe_skinny.cu", "residual_streams.cu" if self.activation == "relu" else "residual_forms.cu")
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -96,8 +99,8 @@ class GatedMLP(FeedForward):
         F.l2_prefetch(self.w_gate_up)
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        if self.activation == "silu":
-            return linear(linear_swiglu(x, self.w_gate_up, self.rt.act), self.w_down, torch.float32)
+        if self.activation in ("silu", "relu"):
+            return linear(linear_swiglu(x, self.w_gate_up, self.rt.act, self.activation), self.w_down, torch.float32)
         if self.activation == "clamped_swish":
             act = F.clamped_glu(linear(x, self.w_gate_up, torch.float32), self.limit, self.slope, self.rt.act)
             return linear(act, self.w_down, torch.float32)

@@ -18,7 +18,8 @@ from .base import Deferred, Norm, Runtime, TensorDecl, WeightedRowSum, split_sum
 class RMSNorm(Norm):
     """params: ``size``, ``eps``, optional ``tensor`` (the tensor's name below the prefix, default ``weight``)
     and ``one_plus`` (the checkpoint holds the gain's offset from one: ``y = x * rsqrt(mean(x^2) + eps) *
-    (1 + w)``; the sum is formed once, in float32, when the weights are loaded).
+    (1 + w)``; the sum is formed once, in float32, when the weights are loaded); ``gain`` (a constant that
+    multiplies the weight, in float32 at load: a factor on a head's logits, say, since the head is linear).
     Tensor: ``<prefix><tensor> [size]``."""
 
     graph_safe = True
@@ -39,6 +40,9 @@ class RMSNorm(Norm):
             self.weight = (tensors[self._name()].to(device=rt.device, dtype=torch.float32) + 1.0).contiguous()
         else:
             self.weight = rt.precision.small(tensors[self._name()], rt.device)
+        gain = float(self.params.get("gain", 1.0))
+        if gain != 1.0:
+            self.weight = (self.weight.to(torch.float32) * gain).contiguous()
 
     def rms_parameters(self):
         return self.weight, self.eps

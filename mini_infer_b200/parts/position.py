@@ -75,6 +75,37 @@ class ScaledRotaryEncoding(RotaryEncoding):
         return self._table[key]
 
 
+class YarnRotaryEncoding(RotaryEncoding):
+    """Rotary frequencies of which the slow ones are stretched, by a ramp over the pairs (YaRN).
+
+    params: as ``rope``, plus ``factor``, ``original``, ``fast``, ``slow``.  The pair that turns ``n`` times over
+    ``original`` positions has the (fractional) index ``at(n) = rot_dim ln(original / (2 pi n)) / (2 ln theta)``; with
+    ``lo = max(floor(at(fast)), 0)``, ``hi = min(ceil(at(slow)), rot_dim - 1)`` and ``ramp_i = clamp((i - lo) /
+    max(hi - lo, 0.001), 0, 1)`` pair ``i`` turns by ``f_i (1 - ramp_i) + f_i / factor ramp_i``.  Cosines and sines are
+    multiplied by ``magnitude = 0.1 ln(factor) + 1``."""
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.magnitude = 0.1 * math.log(float(self.params["factor"])) + 1.0
+
+    def table(self, device) -> Optional[torch.Tensor]:
+        key = str(device)
+        if key not in self._table:
+            p = self.params
+            factor, original, fast, slow = (float(p[k]) for k in ("factor", "original", "fast", "slow"))
+
+            def at(turns: float) -> float:
+                return self.rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
+
+            lo = max(math.floor(at(fast)), 0)
+            hi = min(math.ceil(at(slow)), self.rot_dim - 1)
+            i = torch.arange(self.rot_dim // 2, dtype=torch.float64)
+            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            f = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / self.rot_dim)
+            self._table[key] = (f / factor * ramp + f * (1.0 - ramp)).to(torch.float32).to(device)
+        return self._table[key]
+
+
 class NoPositionEncoding(PositionEncoding):
     graph_safe = True
     rot_dim = 0
@@ -86,4 +117,5 @@ class NoPositionEncoding(PositionEncoding):
 
 register_part("position", "rope", RotaryEncoding)
 register_part("position", "rope_scaled", ScaledRotaryEncoding)
+register_part("position", "rope_yarn", YarnRotaryEncoding)
 register_part("position", "none", NoPositionEncoding)
