@@ -11,6 +11,8 @@
 //                  (latent_query) the rotated part of every head's query into its place behind the folded part, and
 //                  the unrotated part in the activation type as the operand of the folding product; both at once
 //                  when one product of the layer's input holds queries and latent
+//   latent_gather  the cached rows of whole contexts, one after the other: latents [rows, c] and rotated key parts
+//                  [rows, r padded to 8], the operands of keys and values formed for all heads at once
 //   sigmoid_gate   out[t, h, :] = a[t, h, :] * sigmoid(g[t, h, :]), the gate on the heads' outputs
 //
 // The rotation pairs NEIGHBOURS: dimensions 2i and 2i + 1 turn by the angle position * inv_freq[i].  Angles,
@@ -114,6 +116,35 @@ latent_rows_kernel(LatentStoreArgs st, LatentQueryArgs qa, const int* __restrict
     }
 }
 
+// A warp per row.  The contexts of B requests follow one another; rows beyond their sum are zeros.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table,
+                     const int* __restrict__ kv_len, int B, int max_pages, int page_size,
+                     __nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict__ rot, int rows, int c, int r, int rp) {
+    wait_for_earlier_kernels();
+    const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (row >= rows) return;
+    int b = 0, pos = row;
+    while (b < B && pos >= kv_len[b]) { pos -= kv_len[b]; ++b; }
+    int page = -1;
+    if (b < B) page = block_table[(int64_t)b * max_pages + pos / page_size];
+    const __nv_bfloat16* src = cache + ((int64_t)(page < 0 ? 0 : page) * page_size + (page < 0 ? 0 : pos % page_size)) * (c + r);
+    __nv_bfloat16* dl = lat + (int64_t)row * c;
+    __nv_bfloat16* dr = rot + (int64_t)row * rp;
+    if (c % 8 == 0 && r % 8 == 0) {
+        const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+        for (int i = lane; i < (c + r) / 8; i += 32) {
+            const uint4 v = page < 0 ? zero : *(reinterpret_cast<const uint4*>(src) + i);
+            if (i * 8 < c) *(reinterpret_cast<uint4*>(dl) + i) = v;
+            else *(reinterpret_cast<uint4*>(dr) + (i - c / 8)) = v;
+        }
+        return;
+    }
+    const __nv_bfloat16 zero = __float2bfloat16_rn(0.f);
+    for (int i = lane; i < c; i += 32) dl[i] = page < 0 ? zero : src[i];
+    for (int i = lane; i < rp; i += 32) dr[i] = page < 0 || i >= r ? zero : src[c + i];
+}
+
 // out[t, h, j] = a[h * a_head + t * a_tok + j] * sigmoid(g[t * ldg + col0 + h * e + j])
 template <typename AT>
 __global__ void __launch_bounds__(256)
@@ -193,6 +224,18 @@ int mi_latent_rows(const float* src, int ld, int col0, const float* gain, float 
         launch_dependent(latent_rows_kernel<AT>, dim3(T, by), dim3(256), sizeof(float) * (r > 0 ? r : 1), stream, st,
                          qa, positions, inv_freq, magnitude, H, d, r, c));
     return finish_launch("latent_rows");
+}
+
+int mi_latent_gather(const void* cache, const int* block_table, const int* kv_len, int B, int max_pages, int page_size,
+                     void* lat, void* rot, int rows, int c, int r, int rp, cudaStream_t stream) {
+    if (rows <= 0) return kOk;
+    if (B < 1 || c < 1 || r < 0 || rp < r || max_pages < 1 || page_size < 1) {
+        set_last_error("latent_gather: %d requests, rows of %d + %d", B, c, r);
+        return kBadShape;
+    }
+    launch_dependent(latent_gather_kernel, dim3((rows + 7) / 8), dim3(256), 0, stream, (const __nv_bfloat16*)cache,
+                     block_table, kv_len, B, max_pages, page_size, (__nv_bfloat16*)lat, (__nv_bfloat16*)rot, rows, c, r, rp);
+    return finish_launch("latent_gather");
 }
 
 int mi_sigmoid_gate(const void* a, int64_t a_head, int64_t a_tok, const float* g, int ldg, int col0, void* out,

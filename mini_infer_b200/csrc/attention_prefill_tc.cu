@@ -35,7 +35,7 @@ using namespace mi::tc;
 
 constexpr int BQ = 128;            // queries per block (MMA M)
 constexpr int BN = 64;             // keys per tile
-constexpr int NK = 3;              // stages of the K ring
+constexpr int NK = 3;              // stages of the K ring (unless a form chooses others)
 constexpr int NV = 2;              // stages of the V ring
 constexpr int HALF_BYTES = 128 * 64 * 2;   // a tile of 128 rows x 64 columns: 16 KiB (Q, P)
 constexpr int KV_HALF = BN * 64 * 2;       // a tile of BN keys x 64 columns: 8 KiB
@@ -76,7 +76,18 @@ __device__ __forceinline__ void mbar_arrive_after_tmem(uint64_t* bar) {
 }
 
 struct Maps {
-    CUtensorMap q, k, v;
+    CUtensorMap q, k, v, kr;
+};
+
+// Keys and values that were formed from a latent before the call (UNFOLDED): token-major rows, all requests' contexts
+// one after the other, [rows, nh * d] unrotated keys (map k), [rows, nh * e] values (map v) and the rotated key part
+// that the heads share, [rows, r] (map kr).  A key tile is `d` columns of the head, in halves of 64, then the shared
+// part in halves of its own; q [tokens, nh, DK] is laid out alike, with zeros between what the two parts fill.
+struct Unfolded {
+    int d16, r16;               // steps of 16 columns that the unrotated and the rotated part take
+    int d, e;                   // columns of a head in the maps k and v
+    const float* gate;          // null, or rows of `ldg` floats: out *= logistic(gate[t, gcol + h e + :])
+    int ldg, gcol;
 };
 
 // DK, DV: key and value sizes in whole 64-column halves (a key row shorter than DK reads zeros beyond its end,
@@ -92,13 +103,13 @@ __device__ __forceinline__ float fast_tanh(float x) {
     return 1.0f - __fdividef(2.0f, fast_exp2(x * 2.8853900817779268f) + 1.0f);
 }
 
-template <int DK, int DV, bool CAPPED = false, bool LOGISTIC = false>
+template <int DK, int DV, bool CAPPED = false, bool LOGISTIC = false, bool UNFOLDED = false, int NK = pt::NK, int NV = pt::NV>
 __global__ void __launch_bounds__(192, 2)
 attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict__ block_table,
                        const int* __restrict__ q_start, const int* __restrict__ kv_len,
                        __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int max_pages,
                        int window, float scale_log2, int* __restrict__ status, int keep_first, int hpq,
-                       float cap_in, float cap_out, int sink, const float* __restrict__ head_bias) {
+                       float cap_in, float cap_out, int sink, const float* __restrict__ head_bias, Unfolded uf) {
     constexpr int DKH = DK / 64, DVH = DV / 64;           // 64-column halves of a key and of a value row
     constexpr uint32_t TMEM_COLS = 256;                   // S[0], S[1] (BN columns each), O (D): two blocks share an SM
     constexpr uint32_t COL_S = 0, COL_O = 2 * BN;
@@ -129,6 +140,9 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
     if (qt * BQ >= q_len) return;                         // uniform for the whole block
     const int kvl = kv_len[b];
     const int hk = h / (nh / nkv);
+    const int dh = UNFOLDED ? (uf.d16 + 3) / 4 : DKH;     // halves of the unrotated part
+    int kv_base = 0;                                      // first row of the request's context in the maps
+    if constexpr (UNFOLDED) for (int i = 0; i < b; ++i) kv_base += kv_len[i];
     const int nq = min(BQ, q_len - qt * BQ);
     const int p_lo = kvl - q_len / hpq + (qt * BQ) / hpq; // position of the tile's first query (hpq divides BQ)
     const int p_hi = p_lo + (nq - 1) / hpq;
@@ -193,7 +207,7 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
             int my_page = -1;                             // looked up before the wait: the latencies overlap
             if (lane < pages_per_tile) {
                 const int kpos = k0 + lane * page_size;
-                if (kpos < kvl) my_page = table[kpos / page_size];
+                if (kpos < kvl) my_page = UNFOLDED ? 0 : table[kpos / page_size];
             }
             bool ok = true;
             if (lane == 0) ok = mbar_wait(is_k ? &k_empty[s] : &v_empty[s], parity, abort_flag, is_k ? 11 : 21);
@@ -207,16 +221,24 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
                 const int pg = it / halves, hh = it - pg * halves;
                 const int page = tile_pages[pg];
                 if (page < 0) continue;
-                const int row = (page * nkv + hk) * page_size;
                 uint8_t* dst = (is_k ? sK : sV) + (size_t)s * halves * KV_HALF + hh * KV_HALF + (size_t)pg * page_bytes;
-                tma_load_2d(dst, is_k ? &maps.k : &maps.v, hh * 64, row, bar);
+                if constexpr (UNFOLDED) {
+                    const int row = kv_base + k0 + pg * page_size;
+                    if (!is_k) tma_load_2d(dst, &maps.v, h * uf.e + hh * 64, row, bar);
+                    else if (hh < dh) tma_load_2d(dst, &maps.k, h * uf.d + hh * 64, row, bar);
+                    else tma_load_2d(dst, &maps.kr, (hh - dh) * 64, row, bar);
+                } else {
+                    const int row = (page * nkv + hk) * page_size;
+                    tma_load_2d(dst, is_k ? &maps.k : &maps.v, hh * 64, row, bar);
+                }
             }
             __syncwarp();                                 // tile_pages is rewritten by the next call
             return true;
         };
-        for (int i = 0; i <= n_tiles + 1; ++i) {          // K runs two tiles ahead of V
+        constexpr int AHEAD = NK > 2 ? 2 : 1;             // K runs two tiles ahead of V (one with two stages)
+        for (int i = 0; i < n_tiles + AHEAD; ++i) {
             if (i < n_tiles && !load_tile(i, true)) break;
-            if (i >= 2 && !load_tile(i - 2, false)) break;
+            if (i >= AHEAD && !load_tile(i - AHEAD, false)) break;
         }
     } else if (warp == 1) {
         if (lane == 0) {
@@ -233,6 +255,8 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
                 const uint64_t dks = umma_desc(smem_u32(sK + (size_t)s * DKH * KV_HALF));
 #pragma unroll
                 for (int kk = 0; kk < DK / 16; ++kk) {
+                    // columns that neither part fills are left out (what lies in K there is another head's)
+                    if (UNFOLDED && !(kk < dh * 4 ? kk < uf.d16 : kk - dh * 4 < uf.r16)) continue;
                     const uint32_t sub = (uint32_t)(kk & 3) * 32;
                     umma_bf16(tmem_base + COL_S + buf * BN, dq + (((uint32_t)(kk >> 2) * HALF_BYTES + sub) >> 4),
                               dks + (((uint32_t)(kk >> 2) * KV_HALF + sub) >> 4), IDESC_S, kk > 0 ? 1u : 0u);
@@ -382,7 +406,10 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const float inv = LOGISTIC ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
-            __nv_bfloat16* dst = out + ((int64_t)(q0 + qt * BQ + r) * nh + h) * DV;
+            const int ev = UNFOLDED ? uf.e : DV;          // columns of a value (a multiple of 8)
+            __nv_bfloat16* dst = out + ((int64_t)(q0 + qt * BQ + r) * nh + h) * ev;
+            const float* gt = UNFOLDED && uf.gate && r < nq
+                                  ? uf.gate + (int64_t)(q0 + qt * BQ + r) * uf.ldg + uf.gcol + h * ev : nullptr;
 #pragma unroll 1
             for (int c0 = 0; c0 < DV; c0 += 32) {
                 uint32_t o[32];
@@ -391,6 +418,12 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
                 if (r < nq) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
+                        if (UNFOLDED && c0 + i >= ev) continue;
+                        if (UNFOLDED && gt) {
+#pragma unroll
+                            for (int k = 0; k < 8; ++k)
+                                o[i + k] = __float_as_uint(__fdividef(__uint_as_float(o[i + k]), 1.0f + __expf(-__ldg(gt + c0 + i + k))));
+                        }
                         uint4 w;
                         w.x = pack_bf16(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
                         w.y = pack_bf16(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
@@ -469,7 +502,7 @@ int mi_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, 
         set_last_error("prefill attention (tcgen05): operands must be 16-byte aligned");
         return kBadShape;
     }
-    pt::Maps maps;
+    pt::Maps maps = {};
     const uint64_t cache_rows = (uint64_t)num_pages * nkv * page_size;
     bool ok = pt::make_map_pitched(&maps.q, q, (uint64_t)T, (uint64_t)nh * d, (uint64_t)nh * d, pt::BQ) &&
               pt::make_map_pitched(&maps.k, k_cache, cache_rows, (uint64_t)d, (uint64_t)d, (uint32_t)page_size) &&
@@ -489,7 +522,7 @@ int mi_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, 
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, nh,    \
                                           nkv, page_size, max_pages, window, scale_log2, status,          \
-                                          keep_first, 1, cap_in, cap_out, sink, nullptr);                 \
+                                          keep_first, 1, cap_in, cap_out, sink, nullptr, pt::Unfolded{});                 \
     } while (0)
     if (cap > 0.f) { if (d == 64) MI_PT(64, true); else MI_PT(128, true); }
     else { if (d == 64) MI_PT(64, false); else MI_PT(128, false); }
@@ -522,7 +555,7 @@ int mi_attn_prefill_tc_logistic(const void* q, const void* k_cache, const void* 
         set_last_error("prefill attention (tcgen05): operands must be 16-byte aligned");
         return kBadShape;
     }
-    pt::Maps maps;
+    pt::Maps maps = {};
     const uint64_t cache_rows = (uint64_t)num_pages * nkv * page_size;
     bool ok = pt::make_map_pitched(&maps.q, q, (uint64_t)T, (uint64_t)nh * dk, (uint64_t)nh * dk, pt::BQ) &&
               pt::make_map_pitched(&maps.k, k_cache, cache_rows, (uint64_t)dk, (uint64_t)dk, (uint32_t)page_size) &&
@@ -541,7 +574,7 @@ int mi_attn_prefill_tc_logistic(const void* q, const void* k_cache, const void* 
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, nh,    \
                                           nkv, page_size, max_pages, window, scale_log2, status, 0, 1,    \
-                                          0.f, 0.f, 0, head_bias);                                        \
+                                          0.f, 0.f, 0, head_bias, pt::Unfolded{});                                        \
     } while (0)
     if (dk == 64) { if (dv == 64) MI_PTL(64, 64); else MI_PTL(64, 128); }
     else { if (dv == 64) MI_PTL(128, 64); else MI_PTL(128, 128); }
@@ -574,7 +607,7 @@ int mi_attn_prefill_tc_shared(const void* q, const void* cache, const int* block
         set_last_error("prefill attention (tcgen05): operands must be 16-byte aligned");
         return kBadShape;
     }
-    pt::Maps maps;
+    pt::Maps maps = {};
     const uint64_t cache_rows = (uint64_t)num_pages * page_size;
     bool ok = pt::make_map_pitched(&maps.q, q, (uint64_t)T * H, (uint64_t)dk, (uint64_t)dk, pt::BQ) &&
               pt::make_map_pitched(&maps.k, cache, cache_rows, (uint64_t)dk, (uint64_t)dk, (uint32_t)page_size) &&
@@ -594,7 +627,7 @@ int mi_attn_prefill_tc_shared(const void* q, const void* cache, const int* block
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, 1, 1,  \
                                           page_size, max_pages, window, scale_log2, status, keep_first, H,  \
-                                          0.f, 0.f, 0, nullptr);                                            \
+                                          0.f, 0.f, 0, nullptr, pt::Unfolded{});                                            \
     } while (0)
     if (dv == 64) {
         if (DKr == 64) MI_PTS(64, 64); else if (DKr == 128) MI_PTS(128, 64); else if (DKr == 192) MI_PTS(192, 64); else MI_PTS(256, 64);
@@ -602,6 +635,67 @@ int mi_attn_prefill_tc_shared(const void* q, const void* cache, const int* block
         if (DKr == 128) MI_PTS(128, 128); else if (DKr == 192) MI_PTS(192, 128); else MI_PTS(256, 128);
     }
 #undef MI_PTS
+    return finish_launch("attn_prefill_tc");
+}
+
+// The same kernel over keys and values that were formed from latents before the call (see Unfolded): q [T, nh, DK] with
+// DK = 64 (ceil(d / 64) + ceil(r / 64)), the rotated part from column 64 ceil(d / 64) on, zeros up to the next multiple
+// of 16 behind each part; kv [rows, kv_pitch] with the unrotated keys of the heads from column 0 and their values from
+// column v_col on; k_rot [rows, r_pitch]; out [T, nh, e].  `kv_len` gives the contexts that follow one another in the
+// rows.  Takes d and e multiples of 8, values up to 128, DK up to 256.
+int mi_attn_prefill_tc_unfolded_supported(int d, int r, int e) {
+    if (d < 8 || d % 8 || r < 2 || r % 2 || e < 8 || e % 8 || e > 128) return 0;
+    return (d + 63) / 64 + (r + 63) / 64 <= 4;
+}
+
+int mi_attn_prefill_tc_unfolded(const void* q, const void* kv, const void* k_rot, const int* q_start,
+                                const int* kv_len, void* out, int* status, int T, int B, int max_q_len, int nh, int d,
+                                int r, int e, int rows, int kv_pitch, int v_col, int r_pitch, int window, float scale,
+                                const float* gate, int ldg, int gcol, cudaStream_t stream) {
+    if (B <= 0 || max_q_len <= 0 || T <= 0) return kOk;
+    if (!mi_attn_prefill_tc_unfolded_supported(d, r, e) || nh < 1 || nh > 65535 || B > 65535 || rows < 1 ||
+        kv_pitch % 8 || v_col % 8 || v_col < nh * d || kv_pitch < v_col + nh * e || r_pitch % 8 || r_pitch < r ||
+        !(scale > 0.f) || window < 0 || (gate && (gcol < 0 || gcol + nh * e > ldg))) {
+        set_last_error("prefill attention over unfolded latents (tcgen05): %d heads of %d + %d, values of %d are not taken",
+                       nh, d, r, e);
+        return kBadShape;
+    }
+    if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(k_rot) |
+         reinterpret_cast<uintptr_t>(out)) & 15) {
+        set_last_error("prefill attention (tcgen05): operands must be 16-byte aligned");
+        return kBadShape;
+    }
+    const int DKr = ((d + 63) / 64 + (r + 63) / 64) * 64, DVr = (e + 63) / 64 * 64;
+    pt::Maps maps = {};
+    const __nv_bfloat16* kvp = (const __nv_bfloat16*)kv;
+    bool ok = pt::make_map_pitched(&maps.q, q, (uint64_t)T, (uint64_t)nh * DKr, (uint64_t)nh * DKr, pt::BQ) &&
+              pt::make_map_pitched(&maps.k, kvp, (uint64_t)rows, (uint64_t)nh * d, (uint64_t)kv_pitch, pt::BN) &&
+              pt::make_map_pitched(&maps.v, kvp + v_col, (uint64_t)rows, (uint64_t)nh * e, (uint64_t)kv_pitch, pt::BN) &&
+              pt::make_map_pitched(&maps.kr, k_rot, (uint64_t)rows, (uint64_t)r, (uint64_t)r_pitch, pt::BN);
+    if (!ok) {
+        set_last_error("prefill attention (tcgen05): cuTensorMapEncodeTiled failed");
+        return kLaunchFailed;
+    }
+    const pt::Unfolded uf = {(d + 15) / 16, (r + 15) / 16, d, e, gate, ldg, gcol};
+    const dim3 grid((max_q_len + pt::BQ - 1) / pt::BQ, nh, B);
+    const float scale_log2 = scale * 1.4426950408889634f;
+    // two blocks share an SM wherever their tiles fit: from 192 key columns on with two K stages and one V stage
+#define MI_PTU(KK, VV, NKS, NVS)                                                                          \
+    do {                                                                                                  \
+        const size_t smem = (size_t)(KK / 64) * pt::HALF_BYTES +                                          \
+                            (size_t)(NKS * (KK / 64) + NVS * (VV / 64)) * pt::KV_HALF + 256;              \
+        auto kern = pt::attn_prefill_tc_kernel<KK, VV, false, false, true, NKS, NVS>;                     \
+        cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
+        kern<<<grid, 192, smem, stream>>>(maps, nullptr, q_start, kv_len, (__nv_bfloat16*)out, nh, nh,    \
+                                          pt::BN, 0, window, scale_log2, status, 0, 1, 0.f, 0.f, 0,       \
+                                          nullptr, uf);                                                   \
+    } while (0)
+    if (DVr == 64) {
+        if (DKr == 128) MI_PTU(128, 64, 3, 2); else if (DKr == 192) MI_PTU(192, 64, 2, 2); else MI_PTU(256, 64, 2, 2);
+    } else {
+        if (DKr == 128) MI_PTU(128, 128, 3, 2); else if (DKr == 192) MI_PTU(192, 128, 2, 1); else MI_PTU(256, 128, 2, 2);
+    }
+#undef MI_PTU
     return finish_launch("attn_prefill_tc");
 }
 

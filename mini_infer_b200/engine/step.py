@@ -142,6 +142,7 @@ class ModelRunner:
         from ..parts.base import Part
         self._keyed_parts = [p for p in model.all_parts() if type(p).capture_key is not Part.capture_key
                              or type(p).side_outputs is not Part.side_outputs]
+        self._launches_follow_context = any(getattr(p, "launches_follow_context", False) for p in model.all_parts())
         self._graph_pool = None
         self.graph_replays = 0
         self.graph_kernel_launches = 0      # kernels of this library launched through graph replays
@@ -390,8 +391,14 @@ class ModelRunner:
         of the pass's bucket (calling it twice changes nothing more)."""
         B = ctx.num_requests
         if chunk:
-            # no launch shape of a prompt portion follows the context length
-            ctx.max_kv_len = self.max_context
+            # no launch shape of a prompt portion follows the context length, unless a part says so: then a pass is
+            # captured per power of two
+            bucket = self.max_context
+            if self._launches_follow_context:
+                bucket = max(1024, self.graph_chunk_tokens)
+                while bucket < ctx.max_kv_len:
+                    bucket *= 2
+            ctx.max_kv_len = min(bucket, self.max_context)
         else:
             # launch shapes that follow the context length (the splits of the decode attention) are captured
             # for the next power of two, at least 1024: a few graphs per batch size, and a short context is

@@ -1710,7 +1710,200 @@ def latent_query(q: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
     return q_full, q_plain
 
 
-def sigmoid_gate(a: torch.Tensor, head_major: bool, g: torch.Tensor, col0: int, heads: int, size: int) -> torch.Tensor:
+def latent_fold_takes(dim: int, rot_dim: int, rank: int) -> bool:
+    """Whether :func:`latent_fold` and :func:`latent_values` take heads of these sizes."""
+    groups = max(1, 256 // max(1, rank // 8))
+    return rank % 8 == 0 and 4 * (dim + 4 + groups * rank) <= 48 * 1024
+
+
+def latent_fold(q: torch.Tensor, col0: int, heads: int, dim: int, w_uk: torch.Tensor, positions: torch.Tensor,
+                inv_freq: Optional[torch.Tensor], rot_dim: int, magnitude: float = 1.0, store=None) -> torch.Tensor:
+    """For a step of few tokens: the folded queries ``[W_uk,h^T q_plain | rotated q_rot]`` (bfloat16 ``[T, heads, rank +
+    rot_dim]``) of the float32 query rows ``q`` from column ``col0``, ``w_uk [heads, dim, rank]`` bfloat16; ``store``
+    (as in :func:`latent_rows`): the cached rows of the same launch."""
+    T = positions.numel()
+    _chk(q, "latent_fold q", F32, (T, None))
+    _chk(positions, "latent_fold positions", I32, (T,))
+    _chk(inv_freq, "latent_fold inv_freq", F32, (rot_dim // 2,))
+    rank = w_uk.shape[2]
+    _chk(w_uk, "latent_fold w_uk", BF16, (heads, dim, rank))
+    st = [None, 0, 0, None, 0.0, None, None]
+    if store is not None:
+        src, kcol, gain, eps, slots, cache = store
+        _chk(src, "latent_fold src", F32, (T, None))
+        _chk(gain, "latent_fold gain", F32, (rank,))
+        _chk(slots, "latent_fold slot_mapping", I32, (T,))
+        _chk(cache, "latent_fold cache", BF16, (None, 1, None, rank + rot_dim))
+        if DEBUG_BOUNDS:
+            _dbg_range(slots, -1, cache.shape[0] * cache.shape[2], "latent_fold slot_mapping")
+        st = [_ptr(src), src.shape[1], int(kcol), _ptr(gain), float(eps), _ptr(slots), _ptr(cache)]
+    out = torch.empty(T, heads, rank + rot_dim, dtype=BF16, device=q.device)
+    check(library().mi_latent_fold(_ptr(q), q.shape[1], int(col0), _ptr(w_uk), *st, _ptr(positions), _ptr(inv_freq),
+                                   float(magnitude), _ptr(out), T, int(heads), int(dim), int(rot_dim), int(rank),
+                                   _stream()), "latent_fold")
+    return out
+
+
+def latent_values(part_o: torch.Tensor, part_ml: torch.Tensor, w_uv: torch.Tensor, gate: Optional[torch.Tensor],
+                  gate_col: int, out: torch.Tensor) -> torch.Tensor:
+    """For a step of few tokens: the partial results of :func:`attention_shared_tc` merged, times the head's value
+    matrix ``w_uv [heads, e, rank]`` (bfloat16), times the logistic of the gate (float32 rows, or None), into ``out
+    [T, heads * e]`` (bfloat16)."""
+    splits, rows, rank = part_o.shape
+    H, e, _ = w_uv.shape
+    T = out.shape[0]
+    _chk(part_o, "latent_values part_o", F32)
+    _chk(part_ml, "latent_values part_ml", F32, (splits, rows, 2))
+    _chk(w_uv, "latent_values w_uv", BF16, (H, e, rank))
+    _chk(gate, "latent_values gate", F32, (T, None))
+    _chk(out, "latent_values out", BF16, (T, H * e))
+    check(library().mi_latent_values(_ptr(part_o), _ptr(part_ml), _ptr(w_uv), _ptr(gate),
+                                     gate.shape[1] if gate is not None else 0, int(gate_col), _ptr(out), T, H, e, rank,
+                                     splits, rows, _stream()), "latent_values")
+    return out
+
+
+def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, kv_len: torch.Tensor, rows: int, rank: int,
+                  rot_dim: int):
+    """The cached rows (``[pages, 1, page_size, rank + rot_dim]`` bfloat16) of the requests' whole contexts, one after
+    the other: ``(latents [rows, rank], rotated key parts [rows, rot_dim rounded up to 8])``; rows beyond the sum of
+    the contexts are zeros."""
+    _chk(cache, "latent_gather cache", BF16, (None, 1, None, rank + rot_dim))
+    _chk(block_table, "latent_gather block_table", I32)
+    B = block_table.shape[0]
+    _chk(kv_len, "latent_gather kv_len", I32, (B,))
+    rp = (rot_dim + 7) // 8 * 8
+    lat = torch.empty(rows, rank, dtype=BF16, device=cache.device)
+    rot = torch.empty(rows, rp, dtype=BF16, device=cache.device)
+    if DEBUG_BOUNDS:
+        _dbg_range(block_table, -1, cache.shape[0], "latent_gather block_table")
+    check(library().mi_latent_gather(_ptr(cache), _ptr(block_table), _ptr(kv_len), B, block_table.shape[1],
+                                     cache.shape[2], _ptr(lat), _ptr(rot), int(rows), int(rank), int(rot_dim), rp,
+                                     _stream()), "latent_gather")
+    return lat, rot
+
+
+def prefill_attention_tc_unfolded_supported(dim: int, rot_dim: int, value_dim: int) -> bool:
+    return bool(library().mi_attn_prefill_tc_unfolded_supported(int(dim), int(rot_dim), int(value_dim)))
+
+
+def unfolded_query_layout(dim: int, rot_dim: int):
+    """``(columns of a head's padded query, first column of its rotated part)`` of
+    :func:`prefill_attention_tc_unfolded`."""
+    dh = (dim + 63) // 64
+    return 64 * (dh + (rot_dim + 63) // 64), 64 * dh
+
+
+def prefill_attention_tc_unfolded(q: torch.Tensor, kv: torch.Tensor, k_rot: torch.Tensor, q_start: torch.Tensor,
+                                  kv_len: torch.Tensor, max_q_len: int, dim: int, rot_dim: int, value_dim: int,
+                                  window: int, scale: float, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
+                                  gate_col: int = 0) -> torch.Tensor:
+    """Prompt attention (tcgen05) over keys and values formed from latents: ``kv [rows, heads * dim + heads *
+    value_dim]`` (unrotated keys of all heads, then values), ``k_rot [rows, >= rot_dim]`` (shared), the requests'
+    contexts one after the other; ``q [T, heads, *]`` padded as :func:`unfolded_query_layout` says.  Rows ``q_start[0]
+    .. q_start[B]`` of ``out [T, heads * value_dim]`` are written, times the logistic of ``gate`` (float32 rows of the
+    step's tokens from column ``gate_col``) if given."""
+    _chk(q, "prefill_attention_tc_unfolded q", BF16)
+    T, H, cols = q.shape
+    if cols != unfolded_query_layout(dim, rot_dim)[0]:
+        raise ValueError(f"prefill_attention_tc_unfolded: queries of {cols} columns")
+    rows, pitch = kv.shape
+    _chk(kv, "prefill_attention_tc_unfolded kv", BF16, (None, H * (dim + value_dim)))
+    _chk(k_rot, "prefill_attention_tc_unfolded k_rot", BF16, (rows, None))
+    B = q_start.numel() - 1
+    _chk(q_start, "prefill_attention_tc_unfolded q_start", I32)
+    _chk(kv_len, "prefill_attention_tc_unfolded kv_len", I32, (B,))
+    _chk(out, "prefill_attention_tc_unfolded out", BF16, (T, H * value_dim))
+    _chk(gate, "prefill_attention_tc_unfolded gate", F32, (T, None))
+    global _tc_pending
+    dev = q.device
+    if dev not in _tc_status:
+        _tc_status[dev] = torch.zeros(1, dtype=I32, device=dev)
+    if DEBUG_BOUNDS:
+        total = int(kv_len.sum())
+        if total > rows:
+            _bad("prefill_attention_tc_unfolded", f"contexts of {total} tokens in {rows} rows")
+    check(library().mi_attn_prefill_tc_unfolded(
+        _ptr(q), _ptr(kv), _ptr(k_rot), _ptr(q_start), _ptr(kv_len), _ptr(out), _ptr(_tc_status[dev]), T, B,
+        int(max_q_len), H, int(dim), int(rot_dim), int(value_dim), rows, pitch, H * int(dim), k_rot.shape[1],
+        int(window), float(scale), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_col), _stream()),
+        "prefill_attention_tc_unfolded")
+    _tc_pending = True
+    return out
+
+
+def attention_shared_tc_supported(dk: int, dv: int) -> bool:
+    return bool(library().mi_attn_shared_tc_supported(int(dk), int(dv)))
+
+
+def attention_shared_plain_supported(dk: int, dv: int) -> bool:
+    return bool(library().mi_attn_shared_plain_supported(int(dk), int(dv)))
+
+
+def attention_shared_splits(num_requests: int, max_q_len: int, heads: int, dk: int, dv: int, span: int) -> int:
+    """Into how many ranges of keys :func:`attention_shared_tc` cuts a step of few rows so that its blocks fill the
+    device: ``span`` is the longest range of keys that a query sees."""
+    rows = max_q_len * heads
+    bm = int(library().mi_attn_shared_tc_block_rows(rows, dk, dv))
+    if bm <= 0:
+        return 1
+    blocks = num_requests * -(-rows // bm)
+    target = 148 * (1 if dk > 256 else 2)
+    return max(1, min(-(-span // 64), target // blocks))
+
+
+def attention_shared_tc(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, q_start: torch.Tensor,
+                        kv_len: torch.Tensor, max_q_len: int, window: int, scale: float, value_dim: int,
+                        splits: int = 1, partial: bool = False):
+    """Causal attention of all heads over one shared key/value head (bfloat16 tensor cores): ``q [T, heads, dk]``,
+    ``cache [pages, 1, page_size, dk]`` whose rows' first ``value_dim`` numbers are the values.  ``splits``: ranges of
+    keys that blocks of their own work on.  Returns ``[T, heads, value_dim]``, or with ``partial`` the unmerged
+    ``(part_o [splits, T * heads, value_dim], part_ml [splits, T * heads, 2])`` for :func:`latent_values`."""
+    _chk(q, "attention_shared_tc q", BF16)
+    T, H, dk = q.shape
+    _chk(cache, "attention_shared_tc cache", BF16, (None, 1, None, dk))
+    B = block_table.shape[0]
+    _chk(block_table, "attention_shared_tc block_table", I32)
+    _chk(q_start, "attention_shared_tc q_start", I32, (B + 1,))
+    _chk(kv_len, "attention_shared_tc kv_len", I32, (B,))
+    if DEBUG_BOUNDS:
+        _dbg_batch("attention_shared_tc", q_start, kv_len, block_table, T, cache.shape[0], cache.shape[2], window, max_q_len)
+    part_o = part_ml = out = None
+    if splits > 1 or partial:
+        part_o = torch.empty(splits, T * H, value_dim, dtype=F32, device=q.device)
+        part_ml = torch.empty(splits, T * H, 2, dtype=F32, device=q.device)
+    if not partial:
+        out = torch.empty(T, H, value_dim, dtype=BF16, device=q.device)
+    check(library().mi_attn_shared_tc(
+        _ptr(q), _ptr(cache), _ptr(block_table), _ptr(q_start), _ptr(kv_len), _ptr(out), _ptr(part_o), _ptr(part_ml),
+        T, B, int(max_q_len), H, dk, int(value_dim), cache.shape[2], block_table.shape[1], int(window), float(scale),
+        int(splits), _stream()), "attention_shared_tc")
+    return (part_o, part_ml) if partial else out
+
+
+def attention_shared_plain(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, q_start: torch.Tensor,
+                           kv_len: torch.Tensor, max_q_len: int, window: int, scale: float, value_dim: int) -> torch.Tensor:
+    """:func:`attention_shared_tc` for any sizes and both storage types, on CUDA cores, with sums whose order depends
+    on a row's own position only."""
+    _chk(q, "attention_shared_plain q")
+    T, H, dk = q.shape
+    _chk(cache, "attention_shared_plain cache", q.dtype, (None, 1, None, dk))
+    B = block_table.shape[0]
+    _chk(block_table, "attention_shared_plain block_table", I32)
+    _chk(q_start, "attention_shared_plain q_start", I32, (B + 1,))
+    _chk(kv_len, "attention_shared_plain kv_len", I32, (B,))
+    if DEBUG_BOUNDS:
+        _dbg_batch("attention_shared_plain", q_start, kv_len, block_table, T, cache.shape[0], cache.shape[2], window, max_q_len)
+    out = torch.empty(T, H, value_dim, dtype=q.dtype, device=q.device)
+    check(library().mi_attn_shared_plain(
+        _ptr(q), _ptr(cache), _code(q, "attention_shared_plain q"), _ptr(block_table), _ptr(q_start), _ptr(kv_len),
+        _ptr(out), B, int(max_q_len), H, dk, int(value_dim), cache.shape[2], block_table.shape[1], int(window),
+        float(scale), _stream()), "attention_shared_plain")
+    return out
+
+
+def sigmoid_gate(a: torch.Tensor, head_major: bool, g: torch.Tensor, col0: int, heads: int, size: int,
+                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[t, h, :] = a[t, h, :] * logistic(g[t, col0 + h * size : ...])``; ``a`` is ``[T, heads, size]`` or,
     with ``head_major``, ``[heads, T, size]``; ``g`` float32 rows.  Returns ``[T, heads * size]`` in ``a``'s type."""
     _chk(a, "sigmoid_gate a")
@@ -1718,7 +1911,9 @@ def sigmoid_gate(a: torch.Tensor, head_major: bool, g: torch.Tensor, col0: int, 
     T = g.shape[0]
     if a.numel() != T * heads * size:
         raise ValueError("sigmoid_gate: sizes of the heads' outputs and of the gate differ")
-    out = torch.empty(T, heads * size, dtype=a.dtype, device=a.device)
+    if out is None:
+        out = torch.empty(T, heads * size, dtype=a.dtype, device=a.device)
+    _chk(out, "sigmoid_gate out", a.dtype, (T, heads * size))
     a_head, a_tok = (T * size, size) if head_major else (size, heads * size)
     check(library().mi_sigmoid_gate(_ptr(a), a_head, a_tok, _ptr(g), g.shape[1], int(col0), _ptr(out),
                                     _code(a, "sigmoid_gate a"), T, heads, size, _stream()), "sigmoid_gate")

@@ -71,6 +71,12 @@ _SIGNATURES = {
     "mi_streams_read": [P, P, P, P, P, P, P, I, P, I, I, I, I, F, P],
     "mi_streams_sum": [P, P, P, P, P, I, I, I, P],
     "mi_relu_glu": [P, P, I, L, I, P],
+    "mi_attn_shared_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P],
+    "mi_attn_shared_plain": [P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
+    "mi_latent_values": [P, P, P, P, I, I, P, I, I, I, I, I, I, P],
+    "mi_latent_fold": [P, I, I, P, P, I, I, P, F, P, P, P, P, F, P, I, I, I, I, I, P],
+    "mi_latent_gather": [P, P, P, I, I, I, P, P, I, I, I, I, P],
+    "mi_attn_prefill_tc_unfolded": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, P, I, I, P],
     "mi_sigmoid_gate": [P, L, L, P, I, I, P, I, I, I, I, P],
     "mi_causal_conv_residual": [P, I, P, I, P, L, P, P, P, P, I, I, I, I, I, I, P],
     "mi_norm_conv_decode": [P, P, I, F, P, P, L, P, P, P, I, I, I, I, P],
@@ -108,6 +114,10 @@ _OTHERS = {
     "mi_attn_prefill_tc_shared_supported": ([I, I, I, I], c_int),
     "mi_attn_prefill_tc_logistic_supported": ([I, I, I], c_int),
     "mi_attn_decode_split_size": ([], c_int),
+    "mi_attn_shared_tc_supported": ([I, I], c_int),
+    "mi_attn_shared_plain_supported": ([I, I], c_int),
+    "mi_attn_shared_tc_block_rows": ([I, I, I], c_int),
+    "mi_attn_prefill_tc_unfolded_supported": ([I, I, I], c_int),
 }
 
 # kernels that the engine itself calls, whatever the model: embedding, norms and the residual, the dense

@@ -105,6 +105,17 @@ class Tuning:
     scan_segment_tokens: int = 128
     scan_max_segments: int = 32
 
+    # Attention through a latent.  Steps of at most ``latent_small_max_tokens`` tokens run the head's key and value
+    # matrices inside kernels of their own, one block per (token, head), which read the matrices once per token;
+    # above, the library's batched products read them once.
+    latent_small_max_tokens: int = 16
+    # A prompt portion of at least this many tokens forms the keys and values of all heads from the latents of its whole
+    # context before the attention (2 c (d + e) operations per cached token and head, then 2 (d + r + e) per pair
+    # of query and key instead of 2 (2 c + r)); below, the key matrices are folded into the queries.
+    latent_unfold_min_tokens: int = 128
+    # ... unless the formed keys and values would take more than this many megabytes.
+    latent_unfold_max_mbytes: int = 4096
+
     parallel_residual_two_streams: bool = True
     # ... unless the mixer's kernels of a large step want whole SMs themselves (tensor-memory attention: its
     # blocks and those of the feed-forward's tensor-core products cannot sit on one SM, and a block that
