@@ -982,6 +982,103 @@ def run_bogetar(args):
                        _bogetar_kernel_work, _bogetar_twin_kernel_work, "moe_twin", graph_prompts=True)
 
 
+# --------------------------------------------------------------------------- #
+# --gedilorn: the Gedilorn design beside the closest built-in model (dense layers) at equal sizes
+# --------------------------------------------------------------------------- #
+GEDILORN_SIZES = {  # width, heads, unrotated and rotated size and value size of a head, latent size, feed-forward
+                    # width; heads of 128 and key/value heads of the dense twin
+    "0.5b": (1024, 16, 64, 32, 64, 128, 2816, 8, 2),
+    "2b": (2048, 16, 128, 64, 128, 512, 5632, 16, 4),
+    "4b": (2560, 40, 64, 32, 64, 256, 6400, 20, 4),
+}
+GEDILORN_LAYERS = 6
+GEDILORN_STREAMS = 3
+
+
+def gedilorn_config(size, window, vocab):
+    W, H, d, r, e, c, ff, _, _ = GEDILORN_SIZES[size]
+
+    def layer(kind, weights_of=None):
+        m = {"heads": H, "dim": d, "rot_dim": r, "vdim": e, "kv_rank": c, "scale": (d + r) ** -0.5,
+             "rot": {"base": 10000.0, "dims": r,
+                     "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        out = {"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff}}
+        return out if weights_of is None else dict(out, weights_of=weights_of)
+    plain, gated = "latent_attention", "latent_attention_2"
+    layers = [layer(gated), layer(plain), layer(gated), layer(gated), layer(plain, 1), layer(gated, 2)]
+    return {"architecture": "Gedilorn", "vocab": vocab, "width": W, "streams": GEDILORN_STREAMS, "norm": {"eps": 1e-6},
+            "logit_scale": 0.5, "layers": layers,
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 30011, "mul_prev": 7919, "mul_cur": 31}}}
+
+
+def gedilorn_twin_config(size, window, vocab):
+    """The closest built-in model: Qwen2-MoE with every layer dense (grouped-query attention over all keys, SwiGLU
+    feed-forward of the same width), as many layers as the design has layer runs."""
+    W, _, _, _, _, _, ff, H, G = GEDILORN_SIZES[size]
+    n = GEDILORN_LAYERS
+    return dict(A27B, vocab_size=vocab, hidden_size=W, intermediate_size=ff, num_hidden_layers=n,
+                num_attention_heads=H, num_key_value_heads=G, head_dim=128, num_experts=4, num_experts_per_tok=2,
+                moe_intermediate_size=64, shared_expert_intermediate_size=0, mlp_only_layers=list(range(n)),
+                use_sliding_window=False, max_position_embeddings=1 << 20)
+
+
+def _gedilorn_kernel_work(cfg, T, B, ctx, decode):
+    """Algorithmic bytes and floating-point operations of the design's own kernels for one step over all layer runs
+    (prefill of T tokens of one request, or a decode step of B requests at context ctx)."""
+    rows = B if decode else T
+    W, S = cfg["width"], cfg["streams"]
+    out = {}
+
+    def add(name, by, fl):
+        a = out.setdefault(name, [0.0, 0.0])
+        a[0] += by
+        a[1] += fl
+    for i, L in enumerate(cfg["layers"]):
+        m = L["mixer"]
+        H, d, r, e, c = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        gated = L["type"] == "latent_attention_2"
+        # streams read and written, the sublayer's output, what the next one reads; twice a layer, the first of all
+        # without an update
+        for j in range(2):
+            first = i == 0 and j == 0
+            add("streams_read_vec_kernel", rows * W * (S * 4 * (1 if first else 2) + (0 if first else 4) + 2), 0)
+        if decode:
+            add("sh::attn_shared_tc_kernel", B * ctx * (c + r) * 2 + B * H * (c + r) * 2 + B * H * c * 4,
+                B * ctx * H * (2.0 * (c + r) + 2.0 * c))
+            add("sh::latent_fold_kernel", H * d * c * 2 + B * H * ((d + r) * 4 + (c + r) * 2) + B * (c + r) * 6,
+                B * H * 2.0 * d * c)
+            add("sh::latent_values_kernel", H * e * c * 2 + B * H * (c * 4 + e * (6 if gated else 2)), B * H * 2.0 * e * c)
+        else:
+            pairs = T * (T + 1) / 2
+            add("pt::attn_prefill_tc_kernel", T * (H * (d + r) + H * (d + e) + r + H * e) * 2
+                + (T * H * e * 4 if gated else 0), pairs * H * 2.0 * (d + r + e))
+            add("latent_rows_kernel", T * ((c + r) * 6 + H * (d + r) * 6), 0)
+            add("latent_gather_kernel", T * (c + r) * 4, 0)
+            add("relu_glu_bf16x8_kernel", T * L["mlp"]["ff"] * 6, 0)
+    add("streams_embed_kernel", rows * W * (2 + 2 + 4 * S), 0)
+    return out
+
+
+def _gedilorn_twin_kernel_work(cfg, size, window, T, B, ctx, decode):
+    W, _, _, _, _, _, ff, H, G = GEDILORN_SIZES[size]
+    rows, n, d = (B if decode else T), GEDILORN_LAYERS, 128
+    if decode:
+        pairs, by = B * ctx, B * ctx * G * 2 * d * 2 + B * H * 2 * d * 2
+        attn = "attn_decode_split_kernel"
+    else:
+        pairs, by, attn = T * (T + 1) / 2, T * (H + G) * 2 * d * 2, "pt::attn_prefill_tc_kernel"
+    return {attn: [n * by, n * pairs * H * 4.0 * d],
+            "add_rmsnorm_vec_kernel": [(2 * n + 1) * rows * W * (3 * 4 + 2), 0.0],
+            "swiglu_bf16x8_kernel": [n * rows * ff * 6, 0.0],
+            "qkv_post_rows_kernel": [n * rows * (H + 2 * G) * d * 6, 0.0],
+            "embed_gather_kernel": [rows * W * 6, 0.0]}
+
+
+def run_gedilorn(args):
+    return _run_design(args, "gedilorn", args.gedilorn, 0, gedilorn_config, gedilorn_twin_config,
+                       _gedilorn_kernel_work, _gedilorn_twin_kernel_work, "dense_twin", graph_prompts=True)
+
+
 def run_reference(args):
     """The reference arm: Deyu-Kong/mini-infer itself, unmodified, built out of tree for sm_100 by
     ``baseline/build_reference.py`` and driven by ``baseline/reference_bench.cpp`` through its stock path
@@ -1126,6 +1223,9 @@ def main():
                     help="instead of the default workload: the Bogetar design beside Qwen2-MoE at "
                          "these sizes (comma-separated, of " + ", ".join(BOGETAR_SIZES) + "), see run_bogetar")
     ap.add_argument("--bogetar-window", type=int, default=1024, help="attention window of the --bogetar models")
+    ap.add_argument("--gedilorn", default="", metavar="SIZES",
+                    help="instead of the default workload: the Gedilorn design beside Qwen2-MoE with dense layers at "
+                         "these sizes (comma-separated, of " + ", ".join(GEDILORN_SIZES) + "), see run_gedilorn")
     ap.add_argument("--reference-timeout", type=int, default=1500, help="seconds the reference's program may take")
     ap.add_argument("--reference-prefill-batch", type=int, default=1,
                     help="prompts the reference's scheduler prefills per iteration (its cuBLAS handles, one per "
@@ -1151,6 +1251,8 @@ def main():
         return run_tofinex(args)
     if args.bogetar:
         return run_bogetar(args)
+    if args.gedilorn:
+        return run_gedilorn(args)
     return run_ours(args)
 
 

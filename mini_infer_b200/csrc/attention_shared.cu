@@ -15,8 +15,8 @@
 //                       row's own position only: the result does not depend on how a prompt was cut.
 //   latent_values       for steps of few tokens: the partial results of the splits merged, the head's value matrix
 //                       applied, the output gate, one block per (token, head)
-//   latent_fold         for steps of few tokens: a head's query folded by its key matrix, its rotated part, and (one
-//                       block per token) the cached row
+//   latent_fold         for steps of few tokens: every head's queries folded by its key matrix, their rotated parts,
+//                       and the tokens' cached rows
 
 #include "common.cuh"
 
@@ -397,7 +397,10 @@ attn_shared_plain_kernel(const AT* __restrict__ q, const AT* __restrict__ cache,
 // steps of few tokens: the head's matrices beside the attention
 // ---------------------------------------------------------------------------
 
-// grid (H, T).  out[t, h, :] = (W_uv,h . sum_s part) * logistic(gate) with w_uv [H, e, c] bfloat16 rows
+// grid (H, T).  out[t, h, :] = (W_uv,h . sum_s part) * logistic(gate) with w_uv [H, e, c] bfloat16 rows.  A warp owns e / 8
+// value columns, four at a time; a lane 8 latent numbers of every 256.  The matrix does not depend on the kernels
+// before: the first columns' rows are asked for before the wait.
+template <int CP>                                   // passes of 256 latent numbers
 __global__ void __launch_bounds__(256)
 latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                      const __nv_bfloat16* __restrict__ w_uv, const float* __restrict__ gate, int ldg, int gcol,
@@ -406,6 +409,20 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
     float* wgt = vsm + c;
     const int h = blockIdx.x, t = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int c8n = c / 8;
+    const int per = (e + 7) / 8, i_lo = warp * per, i_hi = min(e, i_lo + per);
+    const uint4* wrow = reinterpret_cast<const uint4*>(w_uv + (size_t)h * e * c);
+    uint4 w[4][CP];
+    auto fetch = [&](int i0) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+#pragma unroll
+            for (int p = 0; p < CP; ++p) {
+                const int c8 = lane + 32 * p;
+                w[k][p] = i0 + k < i_hi && c8 < c8n ? __ldg(wrow + (size_t)(i0 + k) * c8n + c8) : make_uint4(0, 0, 0, 0);
+            }
+    };
+    fetch(i_lo);
     wait_for_earlier_kernels();
     const size_t row = (size_t)t * H + h;
     if (warp == 0) {
@@ -414,48 +431,51 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
         m = warp_max(m);
         float l = 0.f;
         for (int s = lane; s < splits; s += 32) {
-            const float ms = part_ml[((size_t)s * total_rows + row) * 2], ls = part_ml[((size_t)s * total_rows + row) * 2 + 1];
-            const float w = ls > 0.f ? exp2_fast(ms - m) : 0.f;
-            wgt[s] = w;
-            l += ls * w;
+            const float2 ml = *reinterpret_cast<const float2*>(part_ml + ((size_t)s * total_rows + row) * 2);
+            const float x = ml.y > 0.f ? exp2_fast(ml.x - m) : 0.f;
+            wgt[s] = x;
+            l += ml.y * x;
         }
         l = warp_sum(l);
         const float inv = l > 0.f ? 1.f / l : 0.f;
         for (int s = lane; s < splits; s += 32) wgt[s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < c; i += 256) {
-        float o = 0.f;
-#pragma unroll 4
+    for (int i = threadIdx.x * 2; i < c; i += 512) {
+        float2 o = make_float2(0.f, 0.f);
+#pragma unroll 8
         for (int s = 0; s < splits; ++s) {
-            const float w = wgt[s];
-            if (w != 0.f) o += part_o[((size_t)s * total_rows + row) * c + i] * w;
-        }
-        vsm[i] = o;
-    }
-    __syncthreads();
-    const int c8n = c / 8;
-    for (int i0 = warp * 4; i0 < e; i0 += 32) {     // four value columns at a time: their loads fly together
-        float s[4] = {0.f, 0.f, 0.f, 0.f};
-        for (int c8 = lane; c8 < c8n; c8 += 32) {
-            const float4 a = *reinterpret_cast<const float4*>(vsm + c8 * 8), bq = *reinterpret_cast<const float4*>(vsm + c8 * 8 + 4);
-            uint4 w[4];
-#pragma unroll
-            for (int k = 0; k < 4; ++k)
-                w[k] = i0 + k < e ? __ldg(reinterpret_cast<const uint4*>(w_uv + ((size_t)h * e + i0 + k) * c) + c8)
-                                  : make_uint4(0, 0, 0, 0);
-#pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&w[k]);
-                const float2 x0 = __bfloat1622float2(p[0]), x1 = __bfloat1622float2(p[1]),
-                             x2 = __bfloat1622float2(p[2]), x3 = __bfloat1622float2(p[3]);
-                s[k] += a.x * x0.x + a.y * x0.y + a.z * x1.x + a.w * x1.y + bq.x * x2.x + bq.y * x2.y + bq.z * x3.x + bq.w * x3.y;
+            const float x = wgt[s];
+            if (x != 0.f) {                         // an empty split wrote nothing
+                const float2 v = __ldg(reinterpret_cast<const float2*>(part_o + ((size_t)s * total_rows + row) * c + i));
+                o.x += v.x * x;
+                o.y += v.y * x;
             }
         }
+        *reinterpret_cast<float2*>(vsm + i) = o;
+    }
+    __syncthreads();
+    for (int i0 = i_lo; i0 < i_hi; i0 += 4) {
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int p = 0; p < CP; ++p) {
+            const int c8 = lane + 32 * p;
+            if (c8 < c8n) {
+                const float4 a = *reinterpret_cast<const float4*>(vsm + c8 * 8), bq = *reinterpret_cast<const float4*>(vsm + c8 * 8 + 4);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const __nv_bfloat162* x = reinterpret_cast<const __nv_bfloat162*>(&w[k][p]);
+                    const float2 x0 = __bfloat1622float2(x[0]), x1 = __bfloat1622float2(x[1]),
+                                 x2 = __bfloat1622float2(x[2]), x3 = __bfloat1622float2(x[3]);
+                    s[k] += a.x * x0.x + a.y * x0.y + a.z * x1.x + a.w * x1.y + bq.x * x2.x + bq.y * x2.y + bq.z * x3.x + bq.w * x3.y;
+                }
+            }
+        }
+        if (i0 + 4 < i_hi) fetch(i0 + 4);           // the next columns' rows fly during the sums over the lanes
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
             const float v = warp_sum(s[k]);
-            if (lane == 0 && i0 + k < e) {
+            if (lane == 0 && i0 + k < i_hi) {
                 float o = v;
                 if (gate) o = v / (1.0f + expf(-gate[(size_t)t * ldg + gcol + h * e + i0 + k]));
                 out[row * e + i0 + k] = __float2bfloat16_rn(o);
@@ -464,37 +484,58 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
     }
 }
 
-// grid (H, T).  q_full[t, h] = [W_uk,h^T q_plain | rot(q_rot)], w_uk [H, d, c] bfloat16; block 0 of a token also writes
-// the cached row (src null: none).  Query rows: [d | r] floats per head from column q_col.
+// grid (H, ceil(c / 32)), all tokens (at most TT) at once: q_full[t, h] = [W_uk,h^T q_plain | rot(q_rot)] with w_uk
+// [H, d, c] bfloat16 read once.  A block owns 32 latent columns of one head: a thread 8 of them and every 64th query
+// dimension.  The first block of a head rotates its queries; the tokens' cached rows (src null: none) are shared out
+// over all blocks.  Query rows: [d | r] floats per head from column q_col.
+constexpr int kFoldCols = 32;
+template <int TT>
 __global__ void __launch_bounds__(256)
 latent_fold_kernel(const float* __restrict__ q, int q_ld, int q_col, const __nv_bfloat16* __restrict__ w_uk,
                    const float* __restrict__ src, int ld, int col0, const float* __restrict__ gain, float eps,
                    const int* __restrict__ slot_mapping, __nv_bfloat16* __restrict__ cache,
                    const int* __restrict__ positions, const float* __restrict__ inv_freq, float magnitude,
-                   __nv_bfloat16* __restrict__ q_full, int H, int d, int r, int c) {
-    extern __shared__ __align__(16) float fs[];     // [d] query, [groups][c] partial sums
+                   __nv_bfloat16* __restrict__ q_full, int T, int H, int d, int r, int c) {
+    extern __shared__ __align__(16) float fs[];     // [T][d] queries
+    __shared__ float part[8][TT][kFoldCols];
     __shared__ float red[32];
+    const int h = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int col = blockIdx.y * kFoldCols + (lane & 3) * 8, g = warp * 8 + (lane >> 2);
+    const bool mine = col < c;
+    const __nv_bfloat16* w = w_uk + (size_t)h * d * c + col;
+    uint4 first = make_uint4(0, 0, 0, 0);           // the matrix does not depend on the kernels before
+    if (mine && g < d) first = __ldg(reinterpret_cast<const uint4*>(w + (size_t)g * c));
     wait_for_earlier_kernels();
-    const int h = blockIdx.x, t = blockIdx.y;
-    const float* row = q + (size_t)t * q_ld + q_col + (size_t)h * (d + r);
-    const float pos = (float)positions[t];
-    __nv_bfloat16* out = q_full + ((size_t)t * H + h) * (c + r);
-    for (int i = threadIdx.x; i < d; i += 256) fs[i] = row[i];
-    for (int i = threadIdx.x; i < r / 2; i += 256) {
-        const float ang = pos * inv_freq[i];
-        const float cs = cosf(ang) * magnitude, sn = sinf(ang) * magnitude;
-        const float u = row[d + 2 * i], v = row[d + 2 * i + 1];
-        out[c + 2 * i] = __float2bfloat16_rn(u * cs - v * sn);
-        out[c + 2 * i + 1] = __float2bfloat16_rn(v * cs + u * sn);
+    for (int i = threadIdx.x; i < T * d; i += 256) {
+        const int t = i / d;
+        fs[i] = q[(size_t)t * q_ld + q_col + (size_t)h * (d + r) + (i - t * d)];
     }
-    if (src && h == 0) {
-        const int slot = slot_mapping[t];
-        if (slot >= 0) {
+    if (blockIdx.y == 0) {
+        const int half = r / 2;
+        for (int idx = threadIdx.x; idx < T * half; idx += 256) {
+            const int t = idx / half, i = idx - t * half;
+            const float ang = (float)positions[t] * inv_freq[i];
+            const float cs = cosf(ang) * magnitude, sn = sinf(ang) * magnitude;
+            const float* row = q + (size_t)t * q_ld + q_col + (size_t)h * (d + r) + d;
+            const float u = row[2 * i], v = row[2 * i + 1];
+            __nv_bfloat16* out = q_full + ((size_t)t * H + h) * (c + r) + c;
+            out[2 * i] = __float2bfloat16_rn(u * cs - v * sn);
+            out[2 * i + 1] = __float2bfloat16_rn(v * cs + u * sn);
+        }
+    }
+    if (src) {
+        // from the last block down: the first block of a head has its rotations to do
+        const int nb = gridDim.x * gridDim.y, bid = nb - 1 - (blockIdx.y * gridDim.x + blockIdx.x);
+        for (int t = bid; t < T; t += nb) {
+            const int slot = slot_mapping[t];
+            if (slot < 0) continue;
             const float* kr = src + (size_t)t * ld + col0;
             float ss = 0.f;
             for (int i = threadIdx.x; i < c; i += 256) { const float x = kr[i]; ss += x * x; }
             ss = block_sum(ss, red);
             const float inv = 1.0f / sqrtf(ss / (float)c + eps);
+            const float pos = (float)positions[t];
             __nv_bfloat16* dst = cache + (size_t)slot * (c + r);
             for (int i = threadIdx.x; i < c; i += 256) dst[i] = __float2bfloat16_rn(kr[i] * inv * gain[i]);
             for (int i = threadIdx.x; i < r / 2; i += 256) {
@@ -507,36 +548,54 @@ latent_fold_kernel(const float* __restrict__ q, int q_ld, int q_col, const __nv_
         }
     }
     __syncthreads();
-    // a thread owns 8 latent columns of every groups-th query dimension
-    const int c8n = c / 8, groups = 256 / c8n > 0 ? 256 / c8n : 1;
-    float* part = fs + ((d + 3) & ~3);
-    for (int base = 0; base < c8n; base += 256 / groups) {
-        const int g = threadIdx.x / (256 / groups), c8 = base + threadIdx.x % (256 / groups);
-        float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (g < groups && c8 < c8n) {
-            const uint4* w = reinterpret_cast<const uint4*>(w_uk + (size_t)h * d * c) + c8;
-#pragma unroll 8
-            for (int i = g; i < d; i += groups) {
-                const uint4 v = __ldg(w + (size_t)i * c8n);
-                const float x = fs[i];
-                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v);
+    float acc[TT][8];
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    const float2 f = __bfloat1622float2(p[k]);
-                    a[2 * k] += x * f.x;
-                    a[2 * k + 1] += x * f.y;
-                }
+    for (int t = 0; t < TT; ++t)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) acc[t][k] = 0.f;
+    if (mine) {
+        uint4 v = first;
+        for (int i = g; i < d; i += 64) {
+            const uint4 now = v;
+            if (i + 64 < d) v = __ldg(reinterpret_cast<const uint4*>(w + (size_t)(i + 64) * c));
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&now);
+            float f[8];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 x = __bfloat1622float2(p[k]);
+                f[2 * k] = x.x;
+                f[2 * k + 1] = x.y;
             }
-            float4* dst = reinterpret_cast<float4*>(part + (size_t)g * c + c8 * 8);
-            dst[0] = make_float4(a[0], a[1], a[2], a[3]);
-            dst[1] = make_float4(a[4], a[5], a[6], a[7]);
+#pragma unroll
+            for (int t = 0; t < TT; ++t)
+                if (t < T) {
+                    const float x = fs[t * d + i];
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) acc[t][k] += x * f[k];
+                }
         }
     }
+    // the 8 lanes of a warp that share columns, then the warps
+#pragma unroll
+    for (int t = 0; t < TT; ++t)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+#pragma unroll
+            for (int o = 4; o < 32; o <<= 1) acc[t][k] += __shfl_xor_sync(0xffffffffu, acc[t][k], o);
+        }
+    if (lane < 4)
+#pragma unroll
+        for (int t = 0; t < TT; ++t)
+#pragma unroll
+            for (int k = 0; k < 8; ++k) part[warp][t][lane * 8 + k] = acc[t][k];
     __syncthreads();
-    for (int i = threadIdx.x; i < c; i += 256) {
+    for (int idx = threadIdx.x; idx < T * kFoldCols; idx += 256) {
+        const int t = idx / kFoldCols, i = idx - t * kFoldCols, cc = blockIdx.y * kFoldCols + i;
+        if (cc >= c) continue;
         float s = 0.f;
-        for (int g = 0; g < groups; ++g) s += part[(size_t)g * c + i];
-        out[i] = __float2bfloat16_rn(s);
+#pragma unroll
+        for (int x = 0; x < 8; ++x) s += part[x][t][i];
+        q_full[((size_t)t * H + h) * (c + r) + cc] = __float2bfloat16_rn(s);
     }
 }
 
@@ -646,33 +705,46 @@ int mi_attn_shared_plain(const void* q, const void* cache, int adtype, const int
 int mi_latent_values(const float* part_o, const float* part_ml, const void* w_uv, const float* gate, int ldg, int gcol,
                      void* out, int T, int H, int e, int c, int splits, int total_rows, cudaStream_t stream) {
     if (T <= 0) return kOk;
-    if (c % 8 || c < 8 || e < 1 || H < 1 || splits < 1 || T > 65535 || total_rows < T * H ||
+    if (c % 8 || c < 8 || c > 512 || e < 1 || H < 1 || splits < 1 || T > 65535 || total_rows < T * H ||
         (gate && (gcol < 0 || gcol + H * e > ldg)) || (c + splits) * sizeof(float) > 48 * 1024) {
         set_last_error("latent_values: %d heads of %d values from latents of %d, %d splits", H, e, c, splits);
         return kBadShape;
     }
-    launch_dependent(sh::latent_values_kernel, dim3(H, T), dim3(256), sizeof(float) * (c + splits), stream, part_o,
-                     part_ml, (const __nv_bfloat16*)w_uv, gate, ldg, gcol, (__nv_bfloat16*)out, H, e, c, splits,
-                     total_rows);
+#define MI_LV(CP)                                                                                                  \
+    launch_dependent(sh::latent_values_kernel<CP>, dim3(H, T), dim3(256), sizeof(float) * (c + splits), stream, part_o, \
+                     part_ml, (const __nv_bfloat16*)w_uv, gate, ldg, gcol, (__nv_bfloat16*)out, H, e, c, splits,   \
+                     total_rows)
+    if (c <= 256) MI_LV(1);
+    else MI_LV(2);
+#undef MI_LV
     return finish_launch("latent_values");
 }
+
+int mi_latent_fold_max_tokens() { return 16; }
 
 int mi_latent_fold(const float* q, int q_ld, int q_col, const void* w_uk, const float* src, int ld, int col0,
                    const float* gain, float eps, const int* slot_mapping, void* cache, const int* positions,
                    const float* inv_freq, float magnitude, void* q_full, int T, int H, int d, int r, int c,
                    cudaStream_t stream) {
     if (T <= 0) return kOk;
-    if (c % 8 || c < 8 || d < 1 || H < 1 || r < 0 || r % 2 || (r > 0 && !inv_freq) || T > 65535 || q_col < 0 ||
+    if (c % 8 || c < 8 || c > 512 || d < 1 || H < 1 || r < 0 || r % 2 || (r > 0 && !inv_freq) || T > 65535 || q_col < 0 ||
         q_col + H * (d + r) > q_ld || (src && (col0 < 0 || col0 + c + r > ld || !gain || !slot_mapping || !cache))) {
         set_last_error("latent_fold: %d heads of %d + %d over latents of %d", H, d, r, c);
         return kBadShape;
     }
-    const int c8n = c / 8, groups = 256 / c8n > 0 ? 256 / c8n : 1;
-    const size_t smem = sizeof(float) * (((d + 3) & ~3) + (size_t)groups * c);
-    if (smem > 48 * 1024) { set_last_error("latent_fold: heads of %d over latents of %d", d, c); return kBadShape; }
-    launch_dependent(sh::latent_fold_kernel, dim3(H, T), dim3(256), smem, stream, q, q_ld, q_col,
-                     (const __nv_bfloat16*)w_uk, src, ld, col0, gain, eps, slot_mapping, (__nv_bfloat16*)cache,
-                     positions, inv_freq, magnitude, (__nv_bfloat16*)q_full, H, d, r, c);
+    const size_t smem = sizeof(float) * (size_t)T * d;
+    if (smem > 24 * 1024 || T > mi_latent_fold_max_tokens()) {
+        set_last_error("latent_fold: %d tokens, heads of %d", T, d);
+        return kBadShape;
+    }
+#define MI_LF(TT)                                                                                                  \
+    launch_dependent(sh::latent_fold_kernel<TT>, dim3(H, (c + sh::kFoldCols - 1) / sh::kFoldCols), dim3(256), smem, \
+                     stream, q, q_ld, q_col, (const __nv_bfloat16*)w_uk, src, ld, col0, gain, eps, slot_mapping,   \
+                     (__nv_bfloat16*)cache, positions, inv_freq, magnitude, (__nv_bfloat16*)q_full, T, H, d, r, c)
+    if (T <= 4) MI_LF(4);
+    else if (T <= 8) MI_LF(8);
+    else MI_LF(16);
+#undef MI_LF
     return finish_launch("latent_fold");
 }
 

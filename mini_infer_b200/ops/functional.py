@@ -1712,8 +1712,11 @@ def latent_query(q: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
 
 def latent_fold_takes(dim: int, rot_dim: int, rank: int) -> bool:
     """Whether :func:`latent_fold` and :func:`latent_values` take heads of these sizes."""
-    groups = max(1, 256 // max(1, rank // 8))
-    return rank % 8 == 0 and 4 * (dim + 4 + groups * rank) <= 48 * 1024
+    return rank % 8 == 0 and 8 <= rank <= 512 and 4 * dim * latent_fold_max_tokens() <= 24 * 1024
+
+
+def latent_fold_max_tokens() -> int:
+    return int(library().mi_latent_fold_max_tokens())
 
 
 def latent_fold(q: torch.Tensor, col0: int, heads: int, dim: int, w_uk: torch.Tensor, positions: torch.Tensor,

@@ -114,6 +114,7 @@ _OTHERS = {
     "mi_attn_prefill_tc_shared_supported": ([I, I, I, I], c_int),
     "mi_attn_prefill_tc_logistic_supported": ([I, I, I], c_int),
     "mi_attn_decode_split_size": ([], c_int),
+    "mi_latent_fold_max_tokens": ([], c_int),
     "mi_attn_shared_tc_supported": ([I, I], c_int),
     "mi_attn_shared_plain_supported": ([I, I], c_int),
     "mi_attn_shared_tc_block_rows": ([I, I, I], c_int),

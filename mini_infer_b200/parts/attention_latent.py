@@ -135,6 +135,7 @@ class LatentAttention(Mixer):
                              f"kernel holds")
         self._tensor_cores = not f32 and F.attention_shared_tc_supported(dk, self.c)
         self._small = self._tensor_cores and F.latent_fold_takes(self.d, self.r, self.c)
+        self._small_max = min(TUNING.latent_small_max_tokens, F.latent_fold_max_tokens()) if self._small else 0
         self._unfold = (not f32 and self.c % 8 == 0
                         and F.prefill_attention_tc_unfolded_supported(self.d, self.r, self.e))
         # prompt portions on the tensor-memory attention: its blocks want whole SMs (a block arrangement that
@@ -178,6 +179,8 @@ class LatentAttention(Mixer):
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
         view = ctx.kv_groups[cache.group]
         rows = view.tensors["latent"][cache.layer_slot]              # [pages, 1, page_size, c + r]
+        if ctx.prefetch is not None:
+            ctx.prefetch([self.w_ukv, self.w_o])
         # gate, this token's cached row, queries
         y = linear(x, self.w_in, torch.float32) if self.w_in is not None else None
         q = y
@@ -189,8 +192,6 @@ class LatentAttention(Mixer):
             if not cache.writes:
                 raise RuntimeError("latent attention: a layer with a latent projection of its own must own its cache")
             store = (y, self.kv_col, self.dkv_gain, self.eps, view.slot_mapping, rows)
-        if ctx.prefetch is not None:
-            ctx.prefetch([self.w_o])
         if self.rt.act == torch.float32:
             v = self._forward_f32(q, y, store, ctx, view, rows)
         else:
@@ -235,7 +236,7 @@ class LatentAttention(Mixer):
         gate = y[:T] if self.gated else None
         table, q_start, kv_len = view.block_table[:B], ctx.q_start[:B + 1], ctx.kv_len[:B]
         mag = self.position.magnitude
-        if self._small and T <= TUNING.latent_small_max_tokens:
+        if T <= self._small_max:
             q_full = F.latent_fold(q, self.q_col, H, d, self.w_uk, positions, self.inv_freq, r, mag, store)
             splits = F.attention_shared_splits(B, max_q_len, H, c + r, c, self._span(max_kv_len))
             part_o, part_ml = F.attention_shared_tc(q_full, rows, table, q_start, kv_len, max_q_len, self.window,
