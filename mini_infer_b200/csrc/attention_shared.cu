@@ -405,8 +405,9 @@ __global__ void __launch_bounds__(256)
 latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                      const __nv_bfloat16* __restrict__ w_uv, const float* __restrict__ gate, int ldg, int gcol,
                      __nv_bfloat16* __restrict__ out, int H, int e, int c, int splits, int total_rows) {
-    extern __shared__ __align__(16) float vsm[];    // [c] merged row, then [splits] weights
-    float* wgt = vsm + c;
+    extern __shared__ __align__(16) float vsm[];    // [c] merged row, [512] or more shares of it, [splits] weights
+    float* share = vsm + c;
+    float* wgt = share + (c > 512 ? c : 512);
     const int h = blockIdx.x, t = blockIdx.y;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int c8n = c / 8;
@@ -425,6 +426,19 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
     fetch(i_lo);
     wait_for_earlier_kernels();
     const size_t row = (size_t)t * H + h;
+    // The threads form groups that own all columns, two a thread, and every ng-th split.  The partial results are asked
+    // for while the splits' weights are formed.
+    const int half = c / 2, ng = 256 / half, g = threadIdx.x / half, i2 = (threadIdx.x - g * half) * 2;
+    const bool mine = g < ng;
+    const float2* po = reinterpret_cast<const float2*>(part_o + row * c + i2);
+    const size_t step = (size_t)total_rows * half;
+    constexpr int PF = 8;
+    float2 pv[PF];
+#pragma unroll
+    for (int j = 0; j < PF; ++j) {
+        const int s = g + j * ng;
+        pv[j] = mine && s < splits ? __ldg(po + s * step) : make_float2(0.f, 0.f);
+    }
     if (warp == 0) {
         float m = -INFINITY;
         for (int s = lane; s < splits; s += 32) m = fmaxf(m, part_ml[((size_t)s * total_rows + row) * 2]);
@@ -441,20 +455,32 @@ latent_values_kernel(const float* __restrict__ part_o, const float* __restrict__
         for (int s = lane; s < splits; s += 32) wgt[s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x * 2; i < c; i += 512) {
+    if (mine) {
         float2 o = make_float2(0.f, 0.f);
-#pragma unroll 8
-        for (int s = 0; s < splits; ++s) {
-            const float x = wgt[s];
-            if (x != 0.f) {                         // an empty split wrote nothing
-                const float2 v = __ldg(reinterpret_cast<const float2*>(part_o + ((size_t)s * total_rows + row) * c + i));
-                o.x += v.x * x;
-                o.y += v.y * x;
-            }
+#pragma unroll
+        for (int j = 0; j < PF; ++j) {
+            const int s = g + j * ng;
+            const float x = s < splits ? wgt[s] : 0.f;
+            if (x != 0.f) { o.x += pv[j].x * x; o.y += pv[j].y * x; }      // an empty split wrote nothing
         }
-        *reinterpret_cast<float2*>(vsm + i) = o;
+#pragma unroll 4
+        for (int s = g + PF * ng; s < splits; s += ng) {
+            const float x = wgt[s];
+            const float2 v = x != 0.f ? __ldg(po + s * step) : make_float2(0.f, 0.f);
+            o.x += v.x * x;
+            o.y += v.y * x;
+        }
+        *reinterpret_cast<float2*>((ng > 1 ? share + (size_t)g * c : vsm) + i2) = o;
     }
     __syncthreads();
+    if (ng > 1) {
+        for (int i = threadIdx.x; i < c; i += 256) {
+            float o = 0.f;
+            for (int k = 0; k < ng; ++k) o += share[(size_t)k * c + i];
+            vsm[i] = o;
+        }
+        __syncthreads();
+    }
     for (int i0 = i_lo; i0 < i_hi; i0 += 4) {
         float s[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -706,12 +732,12 @@ int mi_latent_values(const float* part_o, const float* part_ml, const void* w_uv
                      void* out, int T, int H, int e, int c, int splits, int total_rows, cudaStream_t stream) {
     if (T <= 0) return kOk;
     if (c % 8 || c < 8 || c > 512 || e < 1 || H < 1 || splits < 1 || T > 65535 || total_rows < T * H ||
-        (gate && (gcol < 0 || gcol + H * e > ldg)) || (c + splits) * sizeof(float) > 48 * 1024) {
+        (gate && (gcol < 0 || gcol + H * e > ldg)) || (2 * c + 512 + splits) * sizeof(float) > 48 * 1024) {
         set_last_error("latent_values: %d heads of %d values from latents of %d, %d splits", H, e, c, splits);
         return kBadShape;
     }
 #define MI_LV(CP)                                                                                                  \
-    launch_dependent(sh::latent_values_kernel<CP>, dim3(H, T), dim3(256), sizeof(float) * (c + splits), stream, part_o, \
+    launch_dependent(sh::latent_values_kernel<CP>, dim3(H, T), dim3(256), sizeof(float) * (c + 512 + splits), stream, part_o, \
                      part_ml, (const __nv_bfloat16*)w_uv, gate, ldg, gcol, (__nv_bfloat16*)out, H, e, c, splits,   \
                      total_rows)
     if (c <= 256) MI_LV(1);

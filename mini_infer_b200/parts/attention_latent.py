@@ -179,8 +179,6 @@ class LatentAttention(Mixer):
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
         view = ctx.kv_groups[cache.group]
         rows = view.tensors["latent"][cache.layer_slot]              # [pages, 1, page_size, c + r]
-        if ctx.prefetch is not None:
-            ctx.prefetch([self.w_ukv, self.w_o])
         # gate, this token's cached row, queries
         y = linear(x, self.w_in, torch.float32) if self.w_in is not None else None
         q = y

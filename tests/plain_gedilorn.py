@@ -157,7 +157,10 @@ def forward(config: dict, weights: Dict[str, torch.Tensor], tokens: List[int], d
     x = embedding_output(config, w, tokens)
     xs = x[:, None, :].repeat(1, int(config["streams"]), 1)
     for i, layer in enumerate(config["layers"]):
-        p = f"l{layer.get('weights_of', i)}."
+        own = i
+        while config["layers"][own].get("weights_of") is not None:
+            own = config["layers"][own]["weights_of"]
+        p = f"l{own}."
         h = rnd(rms_norm(streams_read(xs, w[p + "hc1.in"]), w[p + "norm1"], eps))
         y = latent_attention_mixer(h, w, p + "mix.", layer["mixer"], eps, layer["type"] == "latent_attention_2", rnd)
         xs = streams_update(xs, w[p + "hc1.mix"], w[p + "hc1.out"], y)
