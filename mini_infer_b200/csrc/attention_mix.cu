@@ -456,7 +456,7 @@ static size_t mix_smem(int H, int G, int dk, int dv, int esize, int qt, int kt) 
 static MixPlan plan_attn_mix(int H, int G, int dk, int dv, int esize, bool decode) {
     MixPlan p = {1, 32, 1, 0, false};
     const int cpl = (dv + 31) / 32;
-    const int max_rows = 8 * (cpl >= 8 ? 8 : 16);
+    const int max_rows = 8 * (cpl > 4 ? 8 : 16);         // rows of a block: RPW of the form that is launched (5 to 8: CPL 8)
     if (H > max_rows) return p;
     int qt = max_rows / H;
     if (qt > 16) qt = 16;

@@ -107,18 +107,18 @@ def make_weights(cfg: dict, seed: int) -> Dict[str, torch.Tensor]:
         w[p + "norm1"] = gain(W)
         streams(p + "hc1.")
         q = p + "mix."
-        w[q + "q"] = lin(H * (d + r), W, 2.0)
-        w[q + "dkv"], w[q + "dkv.norm"] = lin(c + r, W, 1.5), gain(c)
-        w[q + "uk"], w[q + "uv"] = lin(H * d, c, 1.5), lin(H * e, c, 1.5)
+        w[q + "q"] = lin(H * (d + r), W, 1.5)
+        w[q + "dkv"], w[q + "dkv.norm"] = lin(c + r, W), gain(c)
+        w[q + "uk"], w[q + "uv"] = lin(H * d, c, 1.2), lin(H * e, c, 1.2)
         if L["type"] == GATED:
             w[q + "g"] = lin(H * e, W, 2.0)
-        w[q + "o"] = lin(W, H * e, 2.0)
+        w[q + "o"] = lin(W, H * e, 1.5)
         if L.get("mlp") is not None:
             ff = L["mlp"]["ff"]
             w[p + "norm2"] = gain(W)
             streams(p + "hc2.")
             q = p + "mlp."
-            w[q + "gate"], w[q + "up"], w[q + "down"] = lin(ff, W, 1.5), lin(ff, W, 1.5), lin(W, ff, 1.5)
+            w[q + "gate"], w[q + "up"], w[q + "down"] = lin(ff, W), lin(ff, W), lin(W, ff, 1.5)
     return {k: v.to(torch.bfloat16) for k, v in w.items()}
 
 

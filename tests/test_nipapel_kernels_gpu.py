@@ -83,7 +83,8 @@ def plain_attention(q, k, v, window, keep, scale):
 
 @pytest.mark.parametrize("H,G,d,e,window,keep", [(4, 2, 16, 8, 9, 3), (6, 3, 24, 40, 64, 1), (1, 1, 20, 96, 1, 1),
                                                  (5, 1, 8, 8, 17, 40), (16, 4, 64, 128, 40, 4), (3, 3, 130, 200, 23, 9),
-                                                 (2, 2, 12, 12, 5, 0), (2, 1, 12, 12, 0, 6)])
+                                                 (2, 2, 12, 12, 5, 0), (2, 1, 12, 12, 0, 6), (12, 1, 40, 160, 30, 2),
+                                                 (16, 4, 24, 200, 50, 0)])
 def test_attention_with_kept_first_keys_against_plain_in_any_cut(H, G, d, e, window, keep):
     T = 75
     g = torch.Generator().manual_seed(H * 10 + d)
