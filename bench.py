@@ -724,8 +724,9 @@ def _nipapel_kernel_work(cfg, T, B, ctx, decode):
     (prefill of T tokens of one request, or a decode step of B requests at context ctx)."""
     rows = B if decode else T
     out = {}
-    # decode steps take the split kernel; prompt portions the tensor-memory attention where the sizes allow
+    # decode steps take the split kernels; prompt portions the tensor-memory attention where the sizes allow
     attention_kernels = ("attn_mix_tc_kernel",) if decode else ("attn_mix_tc_kernel", "pt::attn_prefill_tc_kernel")
+    latent_kernel = "sh::attn_shared_tc_kernel" if decode else "pt::attn_prefill_tc_kernel"
 
     def add(name, by, fl):
         a = out.setdefault(name, [0.0, 0.0])
@@ -744,13 +745,13 @@ def _nipapel_kernel_work(cfg, T, B, ctx, decode):
             add("rope_store_kernel", rows * (H * d + G * (d + e)) * 6, 0)
         else:
             H, d, r, e, c = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-            by = (B * keys * (c + r) * 2 + B * H * (2 * c + r) * 2) if decode else T * (H * (2 * c + r) + c + r) * 2
-            for name in attention_kernels:
-                add(name, by, pairs * H * (2.0 * (c + r) + 2.0 * c))
-            if m.get("kv_from") is None:
-                add("latent_store_kernel", rows * (c + r) * 6, 0)
-            add("latent_query_kernel", rows * H * ((d + r) * 4 + (d + r) * 2), 0)
-            add("sigmoid_gate_kernel", rows * H * e * (2 + 4 + 2), 0)
+            if decode:
+                add(latent_kernel, B * keys * (c + r) * 2 + B * H * (c + r) * 2 + B * H * c * 4,
+                    pairs * H * (2.0 * (c + r) + 2.0 * c))
+            else:       # over keys and values formed from the latents, the output gate in the epilogue
+                add(latent_kernel, T * (H * (d + r) + H * (d + e) + r + H * e) * 2 + T * H * e * 4,
+                    pairs * H * 2.0 * (d + r + e))
+                add("latent_rows_kernel", rows * ((0 if m.get("kv_from") is not None else (c + r) * 6) + H * (d + r) * 6), 0)
         if L["mlp"]["kind"] == "dense":
             add("clamped_glu_kernel", rows * L["mlp"]["ff"] * (8 + 2), 0)
     return out
