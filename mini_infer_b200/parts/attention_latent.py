@@ -220,9 +220,10 @@ class LatentAttention(Mixer):
             return v
         if first:
             # the decoding requests in front (a token each); the rows of all tokens are cached by this launch
-            F.latent_rows(ctx.positions, self.inv_freq, self.c, self.r, store=store,
-                          magnitude=self.position.magnitude) if store is not None else None
-            store = None
+            if store is not None:
+                F.latent_rows(ctx.positions, self.inv_freq, self.c, self.r, store=store,
+                              magnitude=self.position.magnitude)
+                store = None
             self._folded(q, y, None, ctx, view, rows, v, first, first, 1, ctx.leading_decodes_max_kv_len)
         self._unfolded(q, y, store, ctx, view, rows, v, first)
         return v

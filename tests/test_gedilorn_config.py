@@ -128,7 +128,7 @@ def test_a_model_names_the_kernel_sources_it_needs():
 # --------------------------------------------------------------------------- #
 
 @pytest.mark.parametrize("dims,base,scaling", [
-    (16, 10000.0, (8.0, 2048, 32.0, 1.0)), (64, 250000.0, (40.0, 4096, 32.0, 1.0)), (4, 100.0, (4.0, 64, 8.0, 0.5)),
+    (20, 10000.0, (6.0, 1024, 32.0, 1.0)), (64, 100000.0, (40.0, 4096, 32.0, 1.0)), (4, 100.0, (4.0, 64, 8.0, 0.5)),
     (2, 50.0, (2.0, 16, 4.0, 1.0)), (32, 500.0, (3.0, 100, 1.0, 1.0)), (8, 10000.0, (2.0, 16, 1e9, 1e-9)),
     (24, 30.0, (16.0, 1 << 20, 1.0, 0.5)), (12, 1e6, (1.0, 512, 32.0, 1.0))])
 def test_yarn_frequencies(dims, base, scaling):
@@ -142,7 +142,7 @@ def test_yarn_frequencies(dims, base, scaling):
 
 
 def test_yarn_leaves_fast_pairs_and_divides_slow_ones():
-    f, _ = pg.yarn_frequencies(64, 10000.0, {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0})
+    f, _ = pg.yarn_frequencies(64, 10000.0, {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0})
     plain, one = pg.yarn_frequencies(64, 10000.0, None)
     assert one == 1.0 and f[0] == plain[0] and f[-1] == pytest.approx(plain[-1] / 8.0)
     ratio = [a / b for a, b in zip(f, plain)]
