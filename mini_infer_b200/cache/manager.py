@@ -47,6 +47,15 @@ class CacheGroupSpec:
         return int(self.need.window)
 
     @property
+    def chunk(self) -> int:
+        return int(getattr(self.need, "chunk", 0) or 0)
+
+    @property
+    def forgets(self) -> bool:
+        """Whether pages are given back while a request lives (a window or a chunk has passed them)."""
+        return self.window > 0 or self.chunk > 0
+
+    @property
     def keep_first(self) -> int:
         """Tokens at the start of a request that a window group keeps for good."""
         return int(getattr(self.need, "keep_first", 0) or 0)
@@ -184,14 +193,14 @@ class CacheManager:
 
     def commit(self, rid: Hashable) -> None:
         """The step that wrote the reserved tokens is done: count them, and give back the
-        pages that every future query's window has passed."""
+        pages that every future query's window (or chunk) has passed."""
         r = self._req[rid]
         r.num_tokens += r.reserved
         r.reserved = 0
         for g, spec in enumerate(self.groups):
-            if spec.window > 0:
-                first_needed = r.num_tokens - spec.window + 1     # oldest key the next query reads
-                dead = max(0, first_needed) // self.page_size      # pages wholly below it
+            if spec.forgets:
+                first_needed = spec.need.first_needed(r.num_tokens)     # oldest key the next query reads
+                dead = first_needed // self.page_size                   # pages wholly below it
                 table = r.tables[g]
                 kept = -(-spec.keep_first // self.page_size)       # pages that hold a token every query reads
                 for i in range(kept, min(dead, len(table))):
@@ -211,10 +220,10 @@ class CacheManager:
         # a window group has given back the pages its window had passed; going back further than that
         # would leave the next query attending over keys that are gone
         for g, spec in enumerate(self.groups):
-            if spec.window > 0 and num_tokens < r.num_tokens:
-                first_needed = max(0, num_tokens - spec.window + 1) // self.page_size
+            if spec.forgets and num_tokens < r.num_tokens:
+                first_needed = spec.need.first_needed(num_tokens) // self.page_size
                 if any(p < 0 for p in r.tables[g][first_needed:keep]):   # (kept first pages are never released)
-                    raise ValueError(f"CacheManager.truncate: group {g} (window {spec.window}) has released pages "
+                    raise ValueError(f"CacheManager.truncate: group {g} (window {spec.window}, chunk {spec.chunk}) has released pages "
                                      f"that a query at position {num_tokens} would read; a request can go back "
                                      f"only as far as its window has not moved on")
         for g, table in enumerate(r.tables):

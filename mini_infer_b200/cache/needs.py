@@ -25,12 +25,20 @@ class PagedCacheNeed:
 
     ``window = 0`` keeps every token's entry, ``window = W`` only the last ``W`` (older pages are given
     back) and, with ``keep_first = F``, the first ``F`` tokens of the request as well (their pages are never
-    given back while the request lives).  ``pages_fraction`` is the share of the engine's page budget that
+    given back while the request lives).  ``chunk = C`` (without a window) keeps the entries of the chunk of
+    ``C`` positions that the next token lies in.  ``pages_fraction`` is the share of the engine's page budget that
     the group of this need gets (1.0 = as many pages as a full-history group)."""
 
     window: int = 0
     pages_fraction: float = 1.0
     keep_first: int = 0
+    chunk: int = 0
+
+    def first_needed(self, num_tokens: int) -> int:
+        """The oldest token (beside the kept first ones) whose entry the token at position ``num_tokens`` reads."""
+        if self.chunk > 0:
+            return num_tokens // self.chunk * self.chunk
+        return max(0, num_tokens - self.window + 1) if self.window > 0 else 0
 
     def tensors(self, page_size: int) -> List[PageTensor]:
         """The tensors of one layer, per page of ``page_size`` tokens."""
@@ -43,7 +51,7 @@ class PagedCacheNeed:
     def group_key(self) -> tuple:
         """Layers whose needs have the same key share a page pool and a block table per request."""
         return (type(self).__name__, self.geometry(), int(self.window), float(self.pages_fraction),
-                int(self.keep_first) if self.window > 0 else 0)
+                int(self.keep_first) if self.window > 0 or self.chunk > 0 else 0, int(self.chunk))
 
     def bytes_per_page(self, page_size: int, act_itemsize: int) -> int:
         total = 0
@@ -66,6 +74,7 @@ class KVNeed(PagedCacheNeed):
     pages_fraction: float = 1.0
     value_dim: int = 0
     keep_first: int = 0
+    chunk: int = 0
 
     def tensors(self, page_size: int) -> List[PageTensor]:
         return [("k", (self.num_kv_heads, page_size, self.head_dim), None),

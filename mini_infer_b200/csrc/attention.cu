@@ -247,14 +247,13 @@ attn_decode_split_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cach
                          const int* __restrict__ block_table, const int* __restrict__ q_start,
                          const int* __restrict__ kv_len, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int nh, int nkv, int page_size, int max_pages,
-                         int max_splits, int window, float scale, float cap) {
+                         int max_splits, int window, float scale, float cap, int chunk) {
     constexpr int E = D / 8;  // elements per thread
     wait_for_earlier_kernels();
     const int b = blockIdx.z, h = blockIdx.y, sp = blockIdx.x;
     const int kvl = kv_len[b];
     const int pos = kvl - 1;
-    int k_first = 0;
-    if (window > 0) k_first = max(0, pos - window + 1);
+    const int k_first = first_visible(pos, window, chunk);
     // never more splits than the caller's scratch holds (a caller whose max_splits is too small for its
     // longest request gets a result over fewer keys, never an access outside the scratch)
     const int n_splits = min(decode_splits<SPLIT>(kvl), max_splits);
@@ -363,19 +362,22 @@ constexpr int MERGE_CAP = 512;
 template <typename AT, int D, int SPLIT>
 __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          const int* __restrict__ q_start, const int* __restrict__ kv_len,
-                                         AT* __restrict__ out, int nh, int max_splits, int window, int sink) {
+                                         AT* __restrict__ out, int nh, int max_splits, int window, int sink,
+                                         AttnForm form) {
+    const int chunk = form.chunk;
     __shared__ float sm_w[MERGE_CAP], sm_l[MERGE_CAP], sm_red[4];
     wait_for_earlier_kernels();
     const int b = blockIdx.y, h = blockIdx.x;
     const int kvl = kv_len[b];
     const int pos = kvl - 1;
-    int k_first = 0;
-    if (window > 0) k_first = max(0, pos - window + 1);
+    const int k_first = first_visible(pos, window, chunk);
     const int n_splits = min(decode_splits<SPLIT>(kvl), max_splits);
     const int first_split = min(k_first / SPLIT, n_splits - 1);
     const int64_t base = ((int64_t)b * nh + h) * max_splits;
     const int t = q_start[b];
     const int n = n_splits - first_split;
+    const float s0 = form.sink_score ? form.sink_score[h] : 0.f;
+    const float hg = head_gate(form, t, h);
     if (n <= MERGE_CAP) {
         const float2* ml = reinterpret_cast<const float2*>(part_ml) + base + first_split;
         float mx = -INFINITY;
@@ -390,16 +392,16 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const
         __syncthreads();
         float m_all = -INFINITY;
         for (int w = 0; w < (int)(blockDim.x + 31) / 32; ++w) m_all = fmaxf(m_all, sm_red[w]);
-        // one key more, of score 0 and without a value: it joins the reference and the sum, not the rows
-        if (sink) m_all = fmaxf(m_all, 0.f);
+        // one key more, without a value: it joins the reference and the sum, not the rows
+        if (sink) m_all = fmaxf(m_all, s0);
         for (int s = threadIdx.x; s < n; s += blockDim.x) {
             const float m = sm_w[s];
             sm_w[s] = m == -INFINITY ? 0.f : expf(m - m_all);
         }
         __syncthreads();
-        float l = sink ? expf(-m_all) : 0.f;
+        float l = sink ? expf(s0 - m_all) : 0.f;
         for (int s = 0; s < n; ++s) l += sm_w[s] * sm_l[s];
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = (l > 0.f ? 1.f / l : 0.f) * hg;
         const float* po = part_o + (base + first_split) * D;
         for (int c = threadIdx.x; c < D; c += blockDim.x) {
             float o = 0.f;
@@ -411,13 +413,13 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const
     }
     float m_all = -INFINITY;
     for (int s = first_split; s < n_splits; ++s) m_all = fmaxf(m_all, part_ml[(base + s) * 2]);
-    if (sink) m_all = fmaxf(m_all, 0.f);
-    float l = sink ? expf(-m_all) : 0.f;
+    if (sink) m_all = fmaxf(m_all, s0);
+    float l = sink ? expf(s0 - m_all) : 0.f;
     for (int s = first_split; s < n_splits; ++s) {
         const float m = part_ml[(base + s) * 2];
         l += (m == -INFINITY ? 0.f : expf(m - m_all)) * part_ml[(base + s) * 2 + 1];
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const float inv = (l > 0.f ? 1.f / l : 0.f) * hg;
     for (int c = threadIdx.x; c < D; c += blockDim.x) {
         float o = 0.f;
         for (int s = first_split; s < n_splits; ++s) {
@@ -499,8 +501,14 @@ int mi_attn_decode_split_form(const void* q, const void* k_cache, const void* v_
                               const int* block_table, const int* q_start, const int* kv_len, void* out,
                               float* part_o, float* part_ml, int B, int nh, int nkv, int d, int page_size,
                               int max_pages, int max_splits, int split, int window, float scale, float cap, int sink,
+                              int chunk, const float* sink_score, const float* gate, int64_t ld_gate,
                               cudaStream_t stream) {
     if (B <= 0) return kOk;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sink_score && !sink)) {
+        set_last_error("decode attention: chunks of %d go without a window (%d), a sink's scores with a sink", chunk, window);
+        return kBadShape;
+    }
+    const AttnForm form = {chunk, sink_score, gate, ld_gate};
     if (cap < 0.f) { set_last_error("decode attention: a cap of %g", (double)cap); return kBadShape; }
     if (!mi_attn_decode_supported(d)) {
         set_last_error("decode attention: head_dim %d is not built (64, 128, 256)", d);
@@ -524,9 +532,9 @@ int mi_attn_decode_split_form(const void* q, const void* k_cache, const void* v_
     do {                                                                                                  \
         launch_dependent(attn_decode_split_kernel<AT, DD, SS>, grid, dim3(128), 0, stream,                \
             (const AT*)q, (const AT*)k_cache, (const AT*)v_cache, block_table, q_start, kv_len, part_o,  \
-            part_ml, nh, nkv, page_size, max_pages, max_splits, window, scale, cap);                      \
+            part_ml, nh, nkv, page_size, max_pages, max_splits, window, scale, cap, chunk);               \
         launch_dependent(attn_decode_merge_kernel<AT, DD, SS>, mgrid, dim3(DD <= 128 ? DD : 128), 0, stream, \
-            part_o, part_ml, q_start, kv_len, (AT*)out, nh, max_splits, window, sink);                    \
+            part_o, part_ml, q_start, kv_len, (AT*)out, nh, max_splits, window, sink, form);              \
     } while (0)
 #define MI_DEC_D(SS) do { if (d == 64) MI_DEC(64, SS); else if (d == 128) MI_DEC(128, SS); else MI_DEC(256, SS); } while (0)
     MI_DISPATCH_1(adtype, AT,
@@ -541,8 +549,8 @@ int mi_attn_decode_split(const void* q, const void* k_cache, const void* v_cache
                          int nh, int nkv, int d, int page_size, int max_pages, int max_splits, int split, int window,
                          float scale, cudaStream_t stream) {
     return mi_attn_decode_split_form(q, k_cache, v_cache, adtype, block_table, q_start, kv_len, out, part_o, part_ml,
-                                     B, nh, nkv, d, page_size, max_pages, max_splits, split, window, scale, 0.f, 0,
-                                     stream);
+                                     B, nh, nkv, d, page_size, max_pages, max_splits, split, window, scale, 0.f, 0, 0,
+                                     nullptr, nullptr, 0, stream);
 }
 
 // The same with the default split size.

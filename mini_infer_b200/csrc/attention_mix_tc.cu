@@ -61,7 +61,7 @@ attn_mix_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
                    const int* __restrict__ kv_len, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                    float* __restrict__ part_ml, int H, int G, int dk, int page_size, int max_pages, int window,
                    float scale, float cap, int splits, int hgroups, int keep_first, int vrs, int sink,
-                   const float* __restrict__ head_bias) {
+                   const float* __restrict__ head_bias, AttnForm form) {
     constexpr int DV = NT * 8;
     constexpr int SP = KT + 1;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -108,7 +108,8 @@ attn_mix_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         // a key more of score 0 and no value (`sink`): of an unsplit step the running maximum starts at 0 and
         // the running sum at 1 (in one lane of the quad that shares a row); a split step leaves it to the merge
         const bool sunk = sink && splits == 1;
-        m_run[hh][0] = m_run[hh][1] = sunk ? 0.f : -INFINITY;
+        const int hs = min(h_lo + warp + kTcWarps * hh, H - 1);
+        m_run[hh][0] = m_run[hh][1] = sunk ? (form.sink_score ? form.sink_score[hs] : 0.f) : -INFINITY;
         l_run[hh][0] = l_run[hh][1] = (sunk && (lane & 3) == 0) ? 1.f : 0.f;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
@@ -116,13 +117,11 @@ attn_mix_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
             for (int x = 0; x < 4; ++x) acc[hh][nt][x] = 0.f;
     }
 
-    int k_begin = 0;
-    if (window > 0) k_begin = max(0, p_lo - window + 1);
-    k_begin = (k_begin / KT) * KT;
+    int k_begin = (first_visible(p_lo, window, form.chunk) / KT) * KT;
     int k_end = min(kvl, p_hi + 1);
     // behind a window the first keep_first keys stay visible: tiles over [0, sink_end) come before the
     // window's tiles (see attention_mix.cu); of a split step the last block takes them
-    int sink_end = window > 0 ? min(min(keep_first, k_begin), k_end) : 0;
+    int sink_end = window > 0 || form.chunk > 0 ? min(min(keep_first, k_begin), k_end) : 0;
     if (splits > 1) {
         if (keep_first > 0 && split == splits - 1) {
             k_begin = k_end;                     // the kept first keys alone
@@ -237,7 +236,7 @@ attn_mix_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
         for (int e = tid; e < kTcQ * KT; e += 256) {
             const int i = e / KT, j = e - i * KT;
             const int kj = kt + j, pos = p_lo + i;
-            const bool vis = i < nq && kj <= pos && (window == 0 || kj > pos - window || kj < keep_first) &&
+            const bool vis = i < nq && kj <= pos && (kj >= first_visible(pos, window, form.chunk) || kj < keep_first) &&
                              slot_of[j] >= 0;
             if (!vis) {
                 for (int h = h_lo; h < h_hi; ++h) S2[((h - h_lo) * kTcQ + i) * SP + j] = -INFINITY;
@@ -359,8 +358,13 @@ attn_mix_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
                     if ((lane & 3) == 0) { part_ml[base * 2] = m_run[hh][0]; part_ml[base * 2 + 1] = l0; }
                 }
             } else {
-                const float i0 = head_bias ? 1.f : (l0 > 0.f ? 1.f / l0 : 0.f);
-                const float i1 = head_bias ? 1.f : (l1 > 0.f ? 1.f / l1 : 0.f);
+                float i0 = head_bias ? 1.f : (l0 > 0.f ? 1.f / l0 : 0.f);
+                float i1 = head_bias ? 1.f : (l1 > 0.f ? 1.f / l1 : 0.f);
+                if (form.gate) {
+                    const int64_t row = q0 + qt * kTcQ + r0;
+                    if (r0 < nq) i0 *= head_gate(form, row, h);
+                    if (r0 + 8 < nq) i1 *= head_gate(form, row + 8, h);
+                }
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
                     if (r0 < nq)
@@ -381,7 +385,7 @@ constexpr int kMergeMaxSplits = 12288;          // two floats a split in shared 
 __global__ void __launch_bounds__(128)
 attn_mix_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                       const int* __restrict__ q_start, __nv_bfloat16* __restrict__ out, int H, int DV, int splits,
-                      int sink, int plain_sum) {
+                      int sink, int plain_sum, AttnForm form) {
     extern __shared__ float merge_sh[];         // [splits] weights, [splits] sums
     float* wgt = merge_sh;
     float* lsum = merge_sh + splits;
@@ -393,7 +397,7 @@ attn_mix_merge_kernel(const float* __restrict__ part_o, const float* __restrict_
         for (int c = threadIdx.x; c < DV; c += blockDim.x) {
             float o = 0.f;
             for (int s = 0; s < splits; ++s) o += part_o[(((size_t)b * splits + s) * H + h) * DV + c];
-            out[((size_t)row0 * H + h) * DV + c] = __float2bfloat16_rn(o);
+            out[((size_t)row0 * H + h) * DV + c] = __float2bfloat16_rn(o * head_gate(form, row0, h));
         }
         return;
     }
@@ -403,15 +407,16 @@ attn_mix_merge_kernel(const float* __restrict__ part_o, const float* __restrict_
         lsum[s] = ml.y;
     }
     __syncthreads();
-    float m = sink ? 0.f : -INFINITY;           // the key of score 0 that `sink` adds counts here, once
+    const float s0 = form.sink_score ? form.sink_score[h] : 0.f;
+    float m = sink ? s0 : -INFINITY;            // the key that `sink` adds counts here, once
     for (int s = 0; s < splits; ++s) m = fmaxf(m, wgt[s]);
     __syncthreads();
     for (int s = threadIdx.x; s < splits; s += blockDim.x) wgt[s] = wgt[s] == -INFINITY ? 0.f : expf(wgt[s] - m);
     __syncthreads();
-    float l = sink ? expf(-m) : 0.f;
+    float l = sink ? expf(s0 - m) : 0.f;
     for (int s = 0; s < splits; ++s) l += lsum[s] * wgt[s];        // in split order
-    const float inv = l > 0.f ? 1.f / l : 0.f;
     const int row = q_start[b];
+    const float inv = (l > 0.f ? 1.f / l : 0.f) * head_gate(form, row, h);
     for (int c = threadIdx.x; c < DV; c += blockDim.x) {
         float o = 0.f;
         for (int s = 0; s < splits; ++s) {
@@ -460,8 +465,15 @@ int mi_attn_mix_tc_form(const void* q, const void* k_cache, const void* v_cache,
                         const int* block_table, const int* q_start, const int* kv_len, void* out, float* part_o,
                         float* part_ml, int B, int max_q_len, int H, int G, int dk, int dv, int page_size,
                         int max_pages, int window, float scale, float cap, int splits, int keep_first, int vrs,
-                        int sink, const float* head_bias, cudaStream_t stream) {
+                        int sink, const float* head_bias, int chunk, const float* sink_score, const float* gate,
+                        int64_t ld_gate, cudaStream_t stream) {
     if (B <= 0 || max_q_len <= 0) return kOk;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sink_score && !sink)) {
+        set_last_error("mixed-head attention (tensor cores): chunks of %d go without a window (%d), a sink's scores with a sink",
+                       chunk, window);
+        return kBadShape;
+    }
+    const AttnForm form = {chunk, sink_score, gate, ld_gate};
     if (head_bias && sink) {
         set_last_error("mixed-head attention (tensor cores): a key more belongs to a softmax, not to weights that are not normalised");
         return kBadShape;
@@ -490,7 +502,7 @@ int mi_attn_mix_tc_form(const void* q, const void* k_cache, const void* v_cache,
         launch_dependent(attn_mix_tc_kernel<HPW, NT, KT>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)q, \
                          (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, mix, block_table, q_start, \
                          kv_len, (__nv_bfloat16*)out, part_o, part_ml, H, G, dk, page_size, max_pages, window,  \
-                         scale, cap, splits, hgroups, keep_first, vrs, sink, head_bias);                        \
+                         scale, cap, splits, hgroups, keep_first, vrs, sink, head_bias, form);                  \
     } while (0)
 #define MI_TC_KT(HPW, NT) do { if (kt == 32) MI_TC_LAUNCH(HPW, NT, 32); else MI_TC_LAUNCH(HPW, NT, 16); } while (0)
     if (dv == 128) {
@@ -507,7 +519,7 @@ int mi_attn_mix_tc_form(const void* q, const void* k_cache, const void* v_cache,
             cudaFuncSetAttribute(attn_mix_merge_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)merge_smem);
         launch_dependent(attn_mix_merge_kernel, dim3(H, B), dim3(128), merge_smem, stream, (const float*)part_o,
                          (const float*)part_ml, q_start, (__nv_bfloat16*)out, H, dv, splits, sink,
-                         head_bias ? 1 : 0);
+                         head_bias ? 1 : 0, form);
         launched = 2;
     }
     return finish_launch("attn_mix_tc", launched);
@@ -519,7 +531,7 @@ int mi_attn_mix_tc(const void* q, const void* k_cache, const void* v_cache, cons
                    float scale, float cap, int splits, int keep_first, int vrs, int sink, cudaStream_t stream) {
     return mi_attn_mix_tc_form(q, k_cache, v_cache, mix, block_table, q_start, kv_len, out, part_o, part_ml, B,
                                max_q_len, H, G, dk, dv, page_size, max_pages, window, scale, cap, splits, keep_first,
-                               vrs, sink, nullptr, stream);
+                               vrs, sink, nullptr, 0, nullptr, nullptr, 0, stream);
 }
 
 }  // extern "C"

@@ -109,7 +109,7 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
                        const int* __restrict__ q_start, const int* __restrict__ kv_len,
                        __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int max_pages,
                        int window, float scale_log2, int* __restrict__ status, int keep_first, int hpq,
-                       float cap_in, float cap_out, int sink, const float* __restrict__ head_bias, Unfolded uf) {
+                       float cap_in, float cap_out, int sink, const float* __restrict__ head_bias, Unfolded uf, AttnForm form) {
     constexpr int DKH = DK / 64, DVH = DV / 64;           // 64-column halves of a key and of a value row
     constexpr uint32_t TMEM_COLS = 256;                   // S[0], S[1] (BN columns each), O (D): two blocks share an SM
     constexpr uint32_t COL_S = 0, COL_O = 2 * BN;
@@ -146,14 +146,13 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
     const int nq = min(BQ, q_len - qt * BQ);
     const int p_lo = kvl - q_len / hpq + (qt * BQ) / hpq; // position of the tile's first query (hpq divides BQ)
     const int p_hi = p_lo + (nq - 1) / hpq;
-    int k_begin = 0;
-    if (window > 0) k_begin = max(0, p_lo - window + 1);
-    k_begin = (k_begin / BN) * BN;
+    const bool bounded = window > 0 || form.chunk > 0;    // keys before some position are out of sight
+    const int k_begin = (first_visible(p_lo, window, form.chunk) / BN) * BN;
     const int k_end = min(kvl, p_hi + 1);
     // Behind a window the first keep_first keys of a request stay visible: tiles over [0, sink_end) come
     // before the window's tiles.  Keys between the two are seen by no query of this block (k_begin is not
     // above any query's window).
-    const int sink_end = window > 0 ? min(min(keep_first, k_begin), k_end) : 0;
+    const int sink_end = bounded ? min(min(keep_first, k_begin), k_end) : 0;
     const int n_sink = (sink_end + BN - 1) / BN;
     const int n_tiles = n_sink + (k_end - k_begin + BN - 1) / BN;  // >= 1: the query's own key is visible
     auto tile_start = [&](int j) { return j < n_sink ? j * BN : k_begin + (j - n_sink) * BN; };
@@ -290,8 +289,8 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
         const int p_row = p_lo + r / hpq;                 // position of this thread's query
         const int vis_hi = min(p_row, kvl - 1);           // last visible key
-        const int vis_lo = window > 0 ? p_row - window + 1 : 0;   // first visible key
-        float m_ref = sink ? 0.f : -INFINITY;             // reference of the exponentials, in log2 units
+        const int vis_lo = first_visible(p_row, window, form.chunk);   // first visible key
+        float m_ref = sink ? (form.sink_score ? form.sink_score[h] * 1.4426950408889634f : 0.f) : -INFINITY;   // reference of the exponentials, in log2 units
         float l_run = sink ? 1.f : 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
@@ -313,7 +312,7 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
                     v[i] = __float_as_uint(fast_tanh(__uint_as_float(v[i]) * cap_in) * cap_out);
             }
             // does any (row, key) of this tile need the mask?
-            const bool masked = (k0 + BN - 1 > p_lo) || (k0 + BN > kvl) || (window > 0 && k0 < p_hi - window + 1);
+            const bool masked = (k0 + BN - 1 > p_lo) || (k0 + BN > kvl) || (bounded && k0 < first_visible(p_hi, window, form.chunk));
             // below a row's window only kept first keys are visible: of a tile of kept first keys those below
             // sink_end (such a tile lies below every window, so it is always masked key by key), of a window's
             // tile those below keep_first
@@ -405,7 +404,8 @@ attn_prefill_tc_kernel(const __grid_constant__ Maps maps, const int* __restrict_
         }
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float inv = LOGISTIC ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
+            float inv = LOGISTIC ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
+            if (form.gate && r < nq) inv *= head_gate(form, q0 + qt * BQ + r, h);
             const int ev = UNFOLDED ? uf.e : DV;          // columns of a value (a multiple of 8)
             __nv_bfloat16* dst = out + ((int64_t)(q0 + qt * BQ + r) * nh + h) * ev;
             const float* gt = UNFOLDED && uf.gate && r < nq
@@ -478,8 +478,14 @@ int mi_attn_prefill_tc_supported(int d, int page_size) {
 int mi_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                        const int* q_start, const int* kv_len, void* out, int* status, int T, int B, int max_q_len,
                        int nh, int nkv, int d, int page_size, int num_pages, int max_pages, int window, float scale,
-                       int keep_first, float cap, int sink, cudaStream_t stream) {
+                       int keep_first, float cap, int sink, int chunk, const float* sink_score, const float* gate,
+                       int64_t ld_gate, cudaStream_t stream) {
     if (B <= 0 || max_q_len <= 0 || T <= 0) return kOk;
+    if (chunk < 0 || (chunk > 0 && window > 0) || (sink_score && !sink)) {
+        set_last_error("prefill attention (tcgen05): chunks of %d go without a window (%d), a sink's scores with a sink", chunk, window);
+        return kBadShape;
+    }
+    const AttnForm form = {chunk, sink_score, gate, ld_gate};
     if (cap < 0.f || !(scale > 0.f)) {
         set_last_error("prefill attention (tcgen05): a cap of %g on scores scaled by %g", (double)cap, (double)scale);
         return kBadShape;
@@ -522,7 +528,7 @@ int mi_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, 
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, nh,    \
                                           nkv, page_size, max_pages, window, scale_log2, status,          \
-                                          keep_first, 1, cap_in, cap_out, sink, nullptr, pt::Unfolded{});                 \
+                                          keep_first, 1, cap_in, cap_out, sink, nullptr, pt::Unfolded{}, form);           \
     } while (0)
     if (cap > 0.f) { if (d == 64) MI_PT(64, true); else MI_PT(128, true); }
     else { if (d == 64) MI_PT(64, false); else MI_PT(128, false); }
@@ -574,7 +580,7 @@ int mi_attn_prefill_tc_logistic(const void* q, const void* k_cache, const void* 
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, nh,    \
                                           nkv, page_size, max_pages, window, scale_log2, status, 0, 1,    \
-                                          0.f, 0.f, 0, head_bias, pt::Unfolded{});                                        \
+                                          0.f, 0.f, 0, head_bias, pt::Unfolded{}, AttnForm{});                            \
     } while (0)
     if (dk == 64) { if (dv == 64) MI_PTL(64, 64); else MI_PTL(64, 128); }
     else { if (dv == 64) MI_PTL(128, 64); else MI_PTL(128, 128); }
@@ -627,7 +633,7 @@ int mi_attn_prefill_tc_shared(const void* q, const void* cache, const int* block
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, block_table, q_start, kv_len, (__nv_bfloat16*)out, 1, 1,  \
                                           page_size, max_pages, window, scale_log2, status, keep_first, H,  \
-                                          0.f, 0.f, 0, nullptr, pt::Unfolded{});                                            \
+                                          0.f, 0.f, 0, nullptr, pt::Unfolded{}, AttnForm{});                                \
     } while (0)
     if (dv == 64) {
         if (DKr == 64) MI_PTS(64, 64); else if (DKr == 128) MI_PTS(128, 64); else if (DKr == 192) MI_PTS(192, 64); else MI_PTS(256, 64);
@@ -688,7 +694,7 @@ int mi_attn_prefill_tc_unfolded(const void* q, const void* kv, const void* k_rot
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);               \
         kern<<<grid, 192, smem, stream>>>(maps, nullptr, q_start, kv_len, (__nv_bfloat16*)out, nh, nh,    \
                                           pt::BN, 0, window, scale_log2, status, 0, 1, 0.f, 0.f, 0,       \
-                                          nullptr, uf);                                                   \
+                                          nullptr, uf, AttnForm{});                                                   \
     } while (0)
     if (DVr == 64) {
         if (DKr == 128) MI_PTU(128, 64, 3, 2); else if (DKr == 192) MI_PTU(192, 64, 2, 2); else MI_PTU(256, 64, 2, 2);

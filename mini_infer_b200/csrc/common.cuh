@@ -150,6 +150,26 @@ inline cudaError_t launch_dependent(void (*kernel)(P...), dim3 grid, dim3 block,
     return cudaLaunchKernelEx(&lc, kernel, static_cast<P>(args)...);
 }
 
+// What else an attention over the paged cache may be asked for (all zero: nothing).
+//   chunk > 0      (then without a window) a query at position p sees the keys of its own chunk only, those from
+//                  p - p % chunk on: chunks are counted from the request's first token
+//   sink_score     [heads]: the softmax counts one key more, of score sink_score[h] (not scaled) and without a value
+//   gate           rows of ld_gate floats: head h's output of token t is multiplied by logistic(gate[t * ld_gate + h])
+struct AttnForm {
+    int chunk;
+    const float* sink_score;
+    const float* gate;
+    int64_t ld_gate;
+};
+// first key that a window or a chunk lets a query at position p see
+__device__ __forceinline__ int first_visible(int p, int window, int chunk) {
+    if (chunk > 0) return p - p % chunk;
+    return window > 0 ? max(0, p - window + 1) : 0;
+}
+__device__ __forceinline__ float head_gate(const AttnForm& f, int64_t t, int h) {
+    return f.gate ? 1.0f / (1.0f + expf(-f.gate[t * f.ld_gate + h])) : 1.0f;
+}
+
 void set_last_error(const char* fmt, ...);
 
 // Checks cudaGetLastError after a launcher queued `n_kernels` kernels and counts them.

@@ -173,7 +173,7 @@ grouped_gemm_skinny_pairs_kernel(const __nv_bfloat16* __restrict__ A, const int*
 // (so a block keeps 8 x 2 KB x unroll of weight loads in flight) and their partial sums are added
 // in warp order through shared memory: the order of additions depends on K only.
 // MODE 0 writes float; MODE 1 holds gate and up rows (W has 2 * Nout rows) and writes
-// silu(gate) * up as bfloat16.  Tile j of NT holds rows 8j .. 8j+7.
+// silu(gate) * up as bfloat16; MODE 2 writes max(., 0)^2 as bfloat16.  Tile j of NT holds rows 8j .. 8j+7.
 template <int MODE, int NT, int WARPS = 8>
 __device__ __forceinline__ void splitk_tile(const __nv_bfloat16* __restrict__ A, const int* src, const int* dst,
                                             const __nv_bfloat16* __restrict__ W, const float* __restrict__ bias,
@@ -254,6 +254,10 @@ __device__ __forceinline__ void splitk_tile(const __nv_bfloat16* __restrict__ A,
                 if (bias) { s0 += bias[f]; s1 += bias[Nout + f]; }
                 const float rs = glu_row_scale(glu, orow);
                 reinterpret_cast<__nv_bfloat16*>(C)[at] = __float2bfloat16_rn(glu_join(s0 * rs, s1 * rs, glu));
+            } else if (MODE == 2) {
+                if (bias) s0 += bias[f];
+                s0 = fmaxf(s0, 0.f);
+                reinterpret_cast<__nv_bfloat16*>(C)[at] = __float2bfloat16_rn(s0 * s0);
             } else {
                 if (bias) s0 += bias[f];
                 reinterpret_cast<float*>(C)[at] = s0;
@@ -510,8 +514,9 @@ int mi_grouped_gemm_skinny_pairs(const void* A, const int* topk_idx, const void*
 // Largest step (in rows) that the dense decode-sized product takes.
 int mi_dense_skinny_max_rows() { return 32; }
 
-// C = A @ W^T (+ bias) for rows <= 32.  A [rows, Kd], W [Nout (mode 0) or 2*Nout (mode 1), Kd] bfloat16;
-// bias float or null; C float [rows, Nout] (mode 0), bfloat16 silu(gate)*up (mode 1) or max(gate, 0)*up (mode 2).
+// C = A @ W^T (+ bias) for rows <= 32.  A [rows, Kd], W [Nout (modes 0 and 3) or 2*Nout (mode 1), Kd] bfloat16;
+// bias float or null; C float [rows, Nout] (mode 0), bfloat16 silu(gate)*up (mode 1) or max(gate, 0)*up (mode 2),
+// bfloat16 max(., 0)^2 of the product (mode 3).
 int mi_dense_skinny(const void* A, const void* W, const float* bias, void* C, int rows, int Nout, int Kd,
                     int mode, cudaStream_t stream) {
     if (Kd <= 0 || Kd % 32 != 0) {
@@ -548,7 +553,11 @@ int mi_dense_skinny(const void* A, const void* W, const float* bias, void* C, in
     }
 #define MI_DENSE_SKINNY(MODE, NT) launch_dependent(dense_skinny_kernel<MODE, NT>, grid, block, 0, stream, a, w, bias, C, rows, Nout, Kd, glu)
     const GluForm glu = {mode == 2 ? 2 : 0, 0.f, 0.f, nullptr};
-    if (mode >= 1) {
+    if (mode == 3) {
+        if (rows <= 8) MI_DENSE_SKINNY(2, 1);
+        else if (rows <= 16) MI_DENSE_SKINNY(2, 2);
+        else MI_DENSE_SKINNY(2, 4);
+    } else if (mode >= 1) {
         if (rows <= 8) MI_DENSE_SKINNY(1, 1);
         else if (rows <= 16) MI_DENSE_SKINNY(1, 2);
         else MI_DENSE_SKINNY(1, 4);

@@ -38,10 +38,13 @@ constexpr int kMaxTaps = 8;
 // come from the request's state (time-major: state[j * C + c] is the input at local position
 // j - (taps-1)), zeros for a fresh request because a new slot is zeroed.
 // ---------------------------------------------------------------------------
-// RES: out = x_t + conv(x)_t, in the type OT, instead of silu(conv(x)_t).
-template <typename WT, typename OT, bool RES>
+// FORM: silu(conv(x)_t); kConvResidual: x_t + conv(x)_t; kConvPlain: conv(x)_t; in the type OT.  `in_bias` (or null): a
+// number per channel that is added to every input of the step (the state holds inputs with it; what lies before a
+// request's first token is zero).
+enum ConvForm : int { kConvSilu = 0, kConvResidual = 1, kConvPlain = 2 };
+template <typename WT, typename OT, int FORM>
 __global__ void __launch_bounds__(256)
-causal_conv_silu_kernel(const float* __restrict__ x, int ldx, const WT* __restrict__ w, const WT* __restrict__ bias,
+causal_conv_silu_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ in_bias, const WT* __restrict__ w, const WT* __restrict__ bias,
                         const float* __restrict__ state, int64_t state_stride, const int* __restrict__ q_start,
                         const int* __restrict__ req_of_token, const int* __restrict__ state_slot,
                         OT* __restrict__ out, int ld_out, int C, int taps, int T) {
@@ -51,7 +54,7 @@ causal_conv_silu_kernel(const float* __restrict__ x, int ldx, const WT* __restri
     float wt[kMaxTaps];
 #pragma unroll
     for (int j = 0; j < kMaxTaps; ++j) wt[j] = j < taps ? to_float(w[(int64_t)c * taps + j]) : 0.f;
-    const float bv = bias ? to_float(bias[c]) : 0.f;
+    const float bv = bias ? to_float(bias[c]) : 0.f, ib = in_bias ? in_bias[c] : 0.f;
     const int per = (T + gridDim.y - 1) / gridDim.y;         // a block's tokens are neighbours in time: their inputs overlap
     for (int t = blockIdx.y * per; t < min(T, (blockIdx.y + 1) * per); ++t) {
         const int b = req_of_token[t];
@@ -62,19 +65,20 @@ causal_conv_silu_kernel(const float* __restrict__ x, int ldx, const WT* __restri
         for (int j = 0; j < kMaxTaps; ++j) {
             if (j < taps) {
                 const int s = i - (taps - 1 - j);      // local position of the input of tap j
-                const float v = s >= 0 ? x[(int64_t)(t - (taps - 1 - j)) * ldx + c] : st[(int64_t)(s + taps - 1) * C + c];
+                const float v = s >= 0 ? x[(int64_t)(t - (taps - 1 - j)) * ldx + c] + ib : st[(int64_t)(s + taps - 1) * C + c];
                 acc += wt[j] * v;
             }
         }
-        out[(int64_t)t * ld_out + c] = from_float<OT>(RES ? x[(int64_t)t * ldx + c] + acc : silu_f(acc));
+        out[(int64_t)t * ld_out + c] = from_float<OT>(
+            FORM == kConvResidual ? x[(int64_t)t * ldx + c] + acc : (FORM == kConvSilu ? silu_f(acc) : acc));
     }
 }
 
 // The same for four neighbouring channels per thread, sixteen bytes per access: rows, state and output whose
 // channel offsets and strides are multiples of four floats.
-template <typename WT, typename OT, bool RES>
+template <typename WT, typename OT, int FORM>
 __global__ void __launch_bounds__(128)
-causal_conv_silu_vec4_kernel(const float* __restrict__ x, int ldx, const WT* __restrict__ w, const WT* __restrict__ bias,
+causal_conv_silu_vec4_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ in_bias, const WT* __restrict__ w, const WT* __restrict__ bias,
                              const float* __restrict__ state, int64_t state_stride, const int* __restrict__ q_start,
                              const int* __restrict__ req_of_token, const int* __restrict__ state_slot,
                              OT* __restrict__ out, int ld_out, int C, int taps, int T) {
@@ -88,6 +92,8 @@ causal_conv_silu_vec4_kernel(const float* __restrict__ x, int ldx, const WT* __r
         for (int j = 0; j < kMaxTaps; ++j) wt[k][j] = j < taps ? to_float(w[(int64_t)(c + k) * taps + j]) : 0.f;
     float4 bv = make_float4(0.f, 0.f, 0.f, 0.f);
     if (bias) bv = make_float4(to_float(bias[c]), to_float(bias[c + 1]), to_float(bias[c + 2]), to_float(bias[c + 3]));
+    float4 ib = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (in_bias) ib = make_float4(in_bias[c], in_bias[c + 1], in_bias[c + 2], in_bias[c + 3]);
     const int per = (T + gridDim.y - 1) / gridDim.y;
     for (int t = blockIdx.y * per; t < min(T, (blockIdx.y + 1) * per); ++t) {
         const int b = req_of_token[t];
@@ -98,14 +104,17 @@ causal_conv_silu_vec4_kernel(const float* __restrict__ x, int ldx, const WT* __r
         for (int j = 0; j < kMaxTaps; ++j) {
             if (j < taps) {
                 const int s = i - (taps - 1 - j);
-                const float4 v = *reinterpret_cast<const float4*>(
+                float4 v = *reinterpret_cast<const float4*>(
                     s >= 0 ? x + (int64_t)(t - (taps - 1 - j)) * ldx + c : st + (int64_t)(s + taps - 1) * C + c);
+                if (in_bias && s >= 0) { v.x += ib.x; v.y += ib.y; v.z += ib.z; v.w += ib.w; }
                 acc.x += wt[0][j] * v.x; acc.y += wt[1][j] * v.y; acc.z += wt[2][j] * v.z; acc.w += wt[3][j] * v.w;
             }
         }
-        if (RES) {
+        if (FORM == kConvResidual) {
             const float4 xt = *reinterpret_cast<const float4*>(x + (int64_t)t * ldx + c);
             store4(out + (int64_t)t * ld_out + c, make_float4(xt.x + acc.x, xt.y + acc.y, xt.z + acc.z, xt.w + acc.w));
+        } else if (FORM == kConvPlain) {
+            store4(out + (int64_t)t * ld_out + c, acc);
         } else {
             store4(out + (int64_t)t * ld_out + c, make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w)));
         }
@@ -115,7 +124,7 @@ causal_conv_silu_vec4_kernel(const float* __restrict__ x, int ldx, const WT* __r
 // The last taps-1 inputs of every request after this step; one thread per (request, channel) moves its
 // entries in ascending order, so an entry is read before it is overwritten.
 __global__ void __launch_bounds__(256)
-conv_state_update_kernel(const float* __restrict__ x, int ldx, float* __restrict__ state, int64_t state_stride,
+conv_state_update_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ in_bias, float* __restrict__ state, int64_t state_stride,
                          const int* __restrict__ q_start, const int* __restrict__ state_slot, int C, int taps) {
     wait_for_earlier_kernels();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -123,9 +132,10 @@ conv_state_update_kernel(const float* __restrict__ x, int ldx, float* __restrict
     if (c >= C) return;
     const int q0 = q_start[b], n = q_start[b + 1] - q0;
     float* st = state + (int64_t)state_slot[b] * state_stride;
+    const float ib = in_bias ? in_bias[c] : 0.f;
     for (int j = 0; j < taps - 1; ++j) {
         const int s = n + j - (taps - 1);              // local position that becomes entry j
-        st[(int64_t)j * C + c] = s >= 0 ? x[(int64_t)(q0 + s) * ldx + c] : st[(int64_t)(n + j) * C + c];
+        st[(int64_t)j * C + c] = s >= 0 ? x[(int64_t)(q0 + s) * ldx + c] + ib : st[(int64_t)(n + j) * C + c];
     }
 }
 
@@ -731,10 +741,10 @@ using namespace mi;
 
 extern "C" {
 
-// form 0: silu(conv(x) + bias), float out; form 1: x + conv(x) in the type `odtype`
-static int launch_causal_conv(const float* x, int ldx, const void* w, const void* bias, int wdtype, float* state,
+// kConvSilu and kConvPlain: float out; kConvResidual: in the type `odtype`
+static int launch_causal_conv(const float* x, int ldx, const float* in_bias, const void* w, const void* bias, int wdtype, float* state,
                               int64_t state_stride, const int* q_start, const int* req_of_token, const int* state_slot,
-                              void* out, int odtype, int ld_out, int C, int taps, int T, int B, bool residual,
+                              void* out, int odtype, int ld_out, int C, int taps, int T, int B, int form,
                               cudaStream_t stream) {
     if (T <= 0 || C <= 0) return kOk;
     if (taps < 1 || taps > kMaxTaps) {
@@ -752,47 +762,58 @@ static int launch_causal_conv(const float* x, int ldx, const void* w, const void
     if (ty > 65535) ty = 65535;
     const bool vec4 = C % 4 == 0 && ldx % 4 == 0 && ld_out % 4 == 0 && state_stride % 4 == 0 &&
                       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(state)) & 15) == 0;
-#define MI_CONV_LAUNCH(OT, RES)                                                                                       \
+#define MI_CONV_LAUNCH(OT, FORM)                                                                                      \
     do {                                                                                                              \
         if (vec4) {                                                                                                   \
             MI_DISPATCH_1(wdtype, WT,                                                                                 \
-                launch_dependent(causal_conv_silu_vec4_kernel<WT, OT, RES>, dim3((C / 4 + 127) / 128, ty), dim3(128), 0, \
-                                 stream, x, ldx, (const WT*)w, (const WT*)bias, (const float*)state, state_stride,    \
+                launch_dependent(causal_conv_silu_vec4_kernel<WT, OT, FORM>, dim3((C / 4 + 127) / 128, ty), dim3(128), 0, \
+                                 stream, x, ldx, in_bias, (const WT*)w, (const WT*)bias, (const float*)state, state_stride,    \
                                  q_start, req_of_token, state_slot, (OT*)out, ld_out, C, taps, T));                   \
         } else {                                                                                                      \
             MI_DISPATCH_1(wdtype, WT,                                                                                 \
-                launch_dependent(causal_conv_silu_kernel<WT, OT, RES>, dim3(cb, ty), dim3(256), 0, stream, x, ldx,     \
+                launch_dependent(causal_conv_silu_kernel<WT, OT, FORM>, dim3(cb, ty), dim3(256), 0, stream, x, ldx, in_bias, \
                                  (const WT*)w, (const WT*)bias, (const float*)state, state_stride, q_start,           \
                                  req_of_token, state_slot, (OT*)out, ld_out, C, taps, T));                            \
         }                                                                                                             \
     } while (0)
-    if (!residual) MI_CONV_LAUNCH(float, false);
-    else if (odtype == kBF16) MI_CONV_LAUNCH(__nv_bfloat16, true);
-    else if (odtype == kF32) MI_CONV_LAUNCH(float, true);
+    if (form == kConvSilu) MI_CONV_LAUNCH(float, kConvSilu);
+    else if (form == kConvPlain) MI_CONV_LAUNCH(float, kConvPlain);
+    else if (odtype == kBF16) MI_CONV_LAUNCH(__nv_bfloat16, kConvResidual);
+    else if (odtype == kF32) MI_CONV_LAUNCH(float, kConvResidual);
     else return kBadDType;
 #undef MI_CONV_LAUNCH
     int launched = 1;
     if (taps > 1) {
-        launch_dependent(conv_state_update_kernel, dim3(cb, B), dim3(256), 0, stream, x, ldx, state, state_stride,
+        launch_dependent(conv_state_update_kernel, dim3(cb, B), dim3(256), 0, stream, x, ldx, in_bias, state, state_stride,
                          q_start, state_slot, C, taps);
         launched = 2;
     }
-    return finish_launch(residual ? "causal_conv_residual" : "causal_conv_silu", launched);
+    return finish_launch(form == kConvResidual ? "causal_conv_residual" : "causal_conv", launched);
 }
 
 int mi_causal_conv_silu(const float* x, int ldx, const void* w, const void* bias, int wdtype, float* state,
                         int64_t state_stride, const int* q_start, const int* req_of_token, const int* state_slot,
                         float* out, int ld_out, int C, int taps, int T, int B, cudaStream_t stream) {
-    return launch_causal_conv(x, ldx, w, bias, wdtype, state, state_stride, q_start, req_of_token, state_slot, out,
-                              kF32, ld_out, C, taps, T, B, false, stream);
+    return launch_causal_conv(x, ldx, nullptr, w, bias, wdtype, state, state_stride, q_start, req_of_token, state_slot, out,
+                              kF32, ld_out, C, taps, T, B, kConvSilu, stream);
 }
 
 // out[t, c] = x[t, c] + sum_j w[c, j] * x(t - (taps-1-j), c) in the type `odtype`; state as above
 int mi_causal_conv_residual(const float* x, int ldx, const void* w, int wdtype, float* state, int64_t state_stride,
                             const int* q_start, const int* req_of_token, const int* state_slot, void* out, int odtype,
                             int ld_out, int C, int taps, int T, int B, cudaStream_t stream) {
-    return launch_causal_conv(x, ldx, w, nullptr, wdtype, state, state_stride, q_start, req_of_token, state_slot, out,
-                              odtype, ld_out, C, taps, T, B, true, stream);
+    return launch_causal_conv(x, ldx, nullptr, w, nullptr, wdtype, state, state_stride, q_start, req_of_token, state_slot, out,
+                              odtype, ld_out, C, taps, T, B, kConvResidual, stream);
+}
+
+// out[t, c] = bias[c] + sum_j w[c, j] * in(t - (taps-1-j), c) with in = x + in_bias (null: x), float; state as above
+// (it holds `in`)
+int mi_causal_conv_plain(const float* x, int ldx, const float* in_bias, const void* w, const void* bias, int wdtype,
+                         float* state, int64_t state_stride, const int* q_start, const int* req_of_token,
+                         const int* state_slot, float* out, int ld_out, int C, int taps, int T, int B,
+                         cudaStream_t stream) {
+    return launch_causal_conv(x, ldx, in_bias, w, bias, wdtype, state, state_stride, q_start, req_of_token, state_slot,
+                              out, kF32, ld_out, C, taps, T, B, kConvPlain, stream);
 }
 
 // One token per request (checked by the caller): norm in groups, x + conv(x), the state moved on, in one launch.

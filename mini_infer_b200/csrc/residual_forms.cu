@@ -14,6 +14,9 @@
 //   out_norm_add          hidden[t] += mult * y[t] / rms(y[t]) * w, and the new row once more in the activation
 //                         type: a block whose parts read the residual itself and whose OUTPUT is normalised;
 //                         y may be a sum of rows that is formed here and never written out
+//   normed_pair_add       hidden[t] += a y1 / rms(y1) * w1 + b y2 / rms(y2) * w2 (two parts that read the same input, each
+//                         output normalised by itself), and, if asked, the norm that follows of the new row
+//   squared_relu          out = max(x, 0)^2
 //   softcap_rows          z <- cap * tanh(z / cap) in place (capped logits)
 
 #include "common.cuh"
@@ -305,6 +308,111 @@ group_rmsnorm_kernel(const float* __restrict__ x, const int* __restrict__ rows, 
     }
 }
 
+// One block per row.  `w` null: only the residual is updated.  `rows` (with w): the rows to normalise, in order; the
+// residual is then left as it is.  VPT > 0: rows of 4 n floats kept in registers (H <= 1024 VPT); 0: any row, read again.
+struct NormedPair {
+    const float* y1;
+    const float* y2;
+    const float* w1;
+    const float* w2;
+    float a, b, eps1, eps2;
+};
+
+template <typename AT, typename WT, int VPT>
+__global__ void __launch_bounds__(256)
+normed_pair_add_kernel(float* __restrict__ hidden, NormedPair p, const int* __restrict__ rows, const WT* __restrict__ w,
+                       AT* __restrict__ out, int H, float eps) {
+    __shared__ float scratch[32];
+    wait_for_earlier_kernels();
+    const int64_t src = rows ? rows[blockIdx.x] : blockIdx.x;
+    float* h = hidden + src * H;
+    const float* y1 = p.y1 + src * H;
+    const float* y2 = p.y2 + src * H;
+    AT* o = out ? out + (int64_t)blockIdx.x * H : nullptr;
+    float s1 = 0.f, s2 = 0.f, ss = 0.f;
+    if constexpr (VPT > 0) {
+        const int nv = H >> 2;
+        float4 v1[VPT], v2[VPT], v[VPT];
+#pragma unroll
+        for (int j = 0; j < VPT; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            v1[j] = v2[j] = v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < nv) {
+                v1[j] = reinterpret_cast<const float4*>(y1)[i];
+                v2[j] = reinterpret_cast<const float4*>(y2)[i];
+                v[j] = reinterpret_cast<const float4*>(h)[i];
+            }
+            s1 += (v1[j].x * v1[j].x + v1[j].y * v1[j].y) + (v1[j].z * v1[j].z + v1[j].w * v1[j].w);
+            s2 += (v2[j].x * v2[j].x + v2[j].y * v2[j].y) + (v2[j].z * v2[j].z + v2[j].w * v2[j].w);
+        }
+        s1 = block_sum(s1, scratch);
+        s2 = block_sum(s2, scratch);
+        const float r1 = p.a / sqrtf(s1 / (float)H + p.eps1), r2 = p.b / sqrtf(s2 / (float)H + p.eps2);
+#pragma unroll
+        for (int j = 0; j < VPT; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i < nv) {
+                const float4 a = reinterpret_cast<const float4*>(p.w1)[i], b = reinterpret_cast<const float4*>(p.w2)[i];
+                v[j].x += v1[j].x * r1 * a.x + v2[j].x * r2 * b.x;
+                v[j].y += v1[j].y * r1 * a.y + v2[j].y * r2 * b.y;
+                v[j].z += v1[j].z * r1 * a.z + v2[j].z * r2 * b.z;
+                v[j].w += v1[j].w * r1 * a.w + v2[j].w * r2 * b.w;
+                if (!rows) reinterpret_cast<float4*>(h)[i] = v[j];
+            }
+            ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+        }
+        if (!w) return;
+        ss = block_sum(ss, scratch);
+        const float rr = 1.0f / sqrtf(ss / (float)H + eps);
+#pragma unroll
+        for (int j = 0; j < VPT; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (i < nv) {
+                const int c = 4 * i;
+                store4(o + c, make_float4(v[j].x * rr * to_float(w[c]), v[j].y * rr * to_float(w[c + 1]),
+                                          v[j].z * rr * to_float(w[c + 2]), v[j].w * rr * to_float(w[c + 3])));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) { s1 += y1[i] * y1[i]; s2 += y2[i] * y2[i]; }
+        s1 = block_sum(s1, scratch);
+        s2 = block_sum(s2, scratch);
+        const float r1 = p.a / sqrtf(s1 / (float)H + p.eps1), r2 = p.b / sqrtf(s2 / (float)H + p.eps2);
+        auto value = [&](int i) { return h[i] + (y1[i] * r1 * p.w1[i] + y2[i] * r2 * p.w2[i]); };
+        for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = value(i); ss += v * v; }
+        ss = block_sum(ss, scratch);
+        const float rr = 1.0f / sqrtf(ss / (float)H + eps);
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float v = value(i);
+            if (!rows) h[i] = v;
+            if (w) o[i] = from_float<AT>(v * rr * to_float(w[i]));
+        }
+    }
+}
+
+__device__ __forceinline__ float squared_relu_f(float x) { const float v = fmaxf(x, 0.f); return v * v; }
+
+template <typename AT>
+__global__ void squared_relu_kernel(const AT* __restrict__ x, AT* __restrict__ out, int64_t total) {
+    wait_for_earlier_kernels();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x)
+        out[i] = from_float<AT>(squared_relu_f(to_float(x[i])));
+}
+
+__global__ void squared_relu_bf16x8_kernel(const uint4* __restrict__ x, uint4* __restrict__ out, int64_t total_vec) {
+    wait_for_earlier_kernels();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total_vec; i += (int64_t)gridDim.x * blockDim.x) {
+        uint4 v = x[i];
+        __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 f = __bfloat1622float2(p[j]);
+            p[j] = __floats2bfloat162_rn(squared_relu_f(f.x), squared_relu_f(f.y));
+        }
+        out[i] = v;
+    }
+}
+
 __global__ void softcap_rows_kernel(float* __restrict__ z, int64_t total, float cap) {
     wait_for_earlier_kernels();
     for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -459,6 +567,48 @@ static int out_norm_add_groups(float* hidden, const float* y, const float* rows,
         launch_dependent(out_norm_add_kernel<AT, WT>, dim3(T, groups), dim3(256), smem, stream, hidden, s, (const WT*)w,
                          (AT*)x_out, H, eps, mult, gs));
     return finish_launch("out_norm_add");
+}
+
+// hidden [T, H] += a y1 / rms(y1) w1 + b y2 / rms(y2) w2; out (with w): the RMS norm of the new rows, or of `rows` of them
+// (hidden is then left as it is)
+int mi_normed_pair_add(float* hidden, const float* y1, const float* w1, float a, float eps1, const float* y2, const float* w2,
+                       float b, float eps2, const int* rows, const void* w, int wdtype, void* out, int adtype, int n_rows,
+                       int H, float eps, cudaStream_t stream) {
+    if (n_rows <= 0 || H <= 0) return kOk;
+    if ((w == nullptr) != (out == nullptr) || (rows && !w)) {
+        set_last_error("normed_pair_add: a norm's weight comes with its output, a row list with a norm");
+        return kBadShape;
+    }
+    const NormedPair p = {y1, y2, w1, w2, a, b, eps1, eps2};
+    const bool vec = H % 4 == 0 && H <= 8192 &&
+                     ((reinterpret_cast<uintptr_t>(hidden) | reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(y2) |
+                       reinterpret_cast<uintptr_t>(w1) | reinterpret_cast<uintptr_t>(w2) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+#define MI_PAIR(VPT)                                                                                                  \
+    MI_DISPATCH_2(adtype, AT, wdtype, WT,                                                                             \
+        launch_dependent(normed_pair_add_kernel<AT, WT, VPT>, dim3(n_rows), dim3(256), 0, stream, hidden, p, rows,    \
+                         (const WT*)w, (AT*)out, H, eps))
+    if (!vec) { MI_PAIR(0); }
+    else if (H <= 1024) { MI_PAIR(1); }
+    else if (H <= 2048) { MI_PAIR(2); }
+    else if (H <= 4096) { MI_PAIR(4); }
+    else { MI_PAIR(8); }
+#undef MI_PAIR
+    return finish_launch("normed_pair_add");
+}
+
+int mi_squared_relu(const void* x, void* out, int adtype, int64_t total, cudaStream_t stream) {
+    if (total <= 0) return kOk;
+    int64_t blocks = (total / (adtype == kBF16 ? 8 : 1) + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    if (blocks < 1) blocks = 1;
+    if (adtype == kBF16 && total % 8 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+        launch_dependent(squared_relu_bf16x8_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const uint4*)x, (uint4*)out,
+                         total / 8);
+        return finish_launch("squared_relu");
+    }
+    MI_DISPATCH_1(adtype, AT,
+        launch_dependent(squared_relu_kernel<AT>, dim3((unsigned)blocks), dim3(256), 0, stream, (const AT*)x, (AT*)out, total));
+    return finish_launch("squared_relu");
 }
 
 int mi_softcap_rows(float* z, int64_t total, float cap, cudaStream_t stream) {

@@ -99,10 +99,15 @@ class Model:
                         raise ValueError(f"schedule[{pos}] reads the cache of schedule[{e.cache_from}], "
                                          f"whose geometry differs")
                     # the owner keeps a token's entry for as long as any of its readers looks back
-                    if (need.window, need.keep_first) != (src.window, src.keep_first):
-                        window = 0 if 0 in (need.window, src.window) else max(need.window, src.window)
-                        widened = dataclasses.replace(src, window=window,
-                                                      keep_first=max(need.keep_first, src.keep_first))
+                    if (need.window, need.keep_first, need.chunk) != (src.window, src.keep_first, src.chunk):
+                        # (a chunk lies within a window of its size)
+                        spans = (need.window or need.chunk, src.window or src.chunk)
+                        same_chunk = need.chunk == src.chunk
+                        widened = dataclasses.replace(
+                            src, window=0 if 0 in spans or (same_chunk and src.chunk) else max(spans),
+                            keep_first=max(need.keep_first, src.keep_first))
+                        if src.chunk and not same_chunk:
+                            widened = dataclasses.replace(widened, chunk=0)
                         needs[e.cache_from][role] = widened
                         paged[:] = [(o, widened if o == (e.cache_from, role) else n) for o, n in paged]
                     continue

@@ -96,7 +96,7 @@ def _dbg_offsets(offsets: torch.Tensor, n_rows: int, what: str) -> None:
 
 
 def _dbg_batch(what: str, q_start: torch.Tensor, kv_len: torch.Tensor, block_table: torch.Tensor, T: int,
-               num_pages: int, page_size: int, window: int, max_q_len: Optional[int] = None) -> None:
+               num_pages: int, page_size: int, window: int, max_q_len: Optional[int] = None, chunk: int = 0) -> None:
     """The layout of a ragged batch over a paged cache: ``q_start`` rises within 0 .. T (a call may cover
     only the first or the last requests of a step's rows), every request's length covers its new tokens and
     fits its table, and every page that a query of this step reads (all of them, or those its window reaches)
@@ -114,11 +114,28 @@ def _dbg_batch(what: str, q_start: torch.Tensor, kv_len: torch.Tensor, block_tab
         if n < n_q or n > max_pages * page_size:
             _bad(what, f"request {b}: kv_len {n} with {n_q} new tokens and a table of {max_pages} pages of {page_size}")
         first = 0 if window <= 0 else max(0, n - n_q - window + 1)
+        if chunk > 0:
+            first = (n - n_q) // chunk * chunk
         row = bt[b]
         for i in range(first // page_size, -(-n // page_size)):
             p = int(row[i])
             if not 0 <= p < num_pages:
                 _bad(what, f"request {b} reads page entry {i} = {p}, the cache has {num_pages} pages")
+
+
+def _attn_form(what: str, nh: int, T: int, window: int, sink: bool, chunk: int, sink_score: Optional[torch.Tensor],
+               gate: Optional[torch.Tensor], gate_col: int):
+    """The arguments that chunks, a sink's scores and a gate per head add to an attention call (see
+    :func:`attention_mix`)."""
+    _chk(sink_score, what + " sink_score", F32, (nh,))
+    if chunk < 0 or (chunk > 0 and window > 0) or (sink_score is not None and not sink):
+        raise ValueError(f"{what}: chunks of {chunk} go without a window ({window}), scores of a sink with a sink")
+    if gate is None:
+        return int(chunk), _ptr(sink_score), None, 0
+    if not gate.is_cuda or gate.dtype != F32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] != T \
+            or not 0 <= gate_col <= gate.shape[1] - nh:
+        raise ValueError(f"{what}: the gate must be float32 rows for {T} tokens with {nh} columns from {gate_col} on")
+    return int(chunk), _ptr(sink_score), gate.data_ptr() + 4 * gate_col, gate.stride(0)
 
 
 _raw_stream = getattr(torch._C, "_cuda_getCurrentRawStream", None)
@@ -353,11 +370,13 @@ def prefill_attention_tc_supported(d: int, page_size: int) -> bool:
 def prefill_attention_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                          q_start: torch.Tensor, kv_len: torch.Tensor, max_q_len: int, window: int = 0,
                          scale: Optional[float] = None, out: Optional[torch.Tensor] = None,
-                         keep_first: int = 0, softcap: float = 0.0, sink: bool = False) -> torch.Tensor:
+                         keep_first: int = 0, softcap: float = 0.0, sink: bool = False, chunk: int = 0,
+                         sink_score: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                         gate_col: int = 0) -> torch.Tensor:
     """Same contract as :func:`attention`, on the tcgen05 tensor cores (TMA-fed, accumulators in
     tensor memory): bfloat16, head sizes 64 and 128, pages of 8 to 128 tokens.  ``softcap`` (0: none): every
     scaled score becomes ``softcap * tanh(score / softcap)``; ``sink``: the softmax counts one key more, of
-    score 0 and without a value.  Call
+    score 0 and without a value; ``chunk``, ``sink_score``, ``gate``: as in :func:`attention_mix`.  Call
     :func:`check_tc_status` after the step: a wait inside the kernel that ran out is reported there."""
     global _tc_pending
     _chk(q, "prefill_attention_tc q", BF16)
@@ -381,11 +400,13 @@ def prefill_attention_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         _tc_status[dev] = torch.zeros(1, dtype=I32, device=dev)
     if DEBUG_BOUNDS:
         _dbg_batch("prefill_attention_tc", q_start, kv_len, block_table, T, num_pages, page_size, int(window),
-                   int(max_q_len))
+                   int(max_q_len), int(chunk))
     check(library().mi_attn_prefill_tc(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(q_start),
                                        _ptr(kv_len), _ptr(out), _ptr(_tc_status[dev]), T, B, int(max_q_len), nh, nkv,
                                        d, page_size, num_pages, max_pages, int(window), float(scale),
-                                       int(keep_first), float(softcap), int(bool(sink)), _stream()),
+                                       int(keep_first), float(softcap), int(bool(sink)),
+                                       *_attn_form("prefill_attention_tc", nh, T, int(window), bool(sink), int(chunk),
+                                                   sink_score, gate, gate_col), _stream()),
           "prefill_attention_tc")
     _tc_pending = True
     return out
@@ -482,10 +503,11 @@ def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      q_start: torch.Tensor, kv_len: torch.Tensor, part_o: torch.Tensor, part_ml: torch.Tensor,
                      max_splits: int, window: int = 0, scale: Optional[float] = None,
                      out: Optional[torch.Tensor] = None, split: Optional[int] = None, softcap: float = 0.0,
-                     sink: bool = False) -> torch.Tensor:
+                     sink: bool = False, chunk: int = 0, sink_score: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> torch.Tensor:
     """Split-KV attention when every request brings exactly one token.  ``softcap`` (0: none): every scaled
     score becomes ``softcap * tanh(score / softcap)``; ``sink``: the softmax counts one key more, of score 0
-    and without a value.
+    and without a value; ``chunk``, ``sink_score``, ``gate``: as in :func:`attention_mix`.
 
     ``part_o`` (``>= B*nh*max_splits*d`` floats) and ``part_ml`` (``>= B*nh*max_splits*2``)
     are scratch; ``max_splits >= ceil(longest kv_len / split)`` with ``split`` keys per split
@@ -517,7 +539,7 @@ def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     if split is None:
         split = decode_split_size()
     if DEBUG_BOUNDS:
-        _dbg_batch("decode_attention", q_start, kv_len, block_table, T, k_cache.shape[0], page_size, int(window), 1)
+        _dbg_batch("decode_attention", q_start, kv_len, block_table, T, k_cache.shape[0], page_size, int(window), 1, int(chunk))
         longest = int(kv_len.max())
         if max_splits * int(split) < longest - int(split) // 4:
             _bad("decode_attention", f"{max_splits} splits of {split} keys cannot hold the longest request ({longest})")
@@ -525,7 +547,8 @@ def decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                                               _ptr(block_table), _ptr(q_start), _ptr(kv_len), _ptr(out), _ptr(part_o),
                                               _ptr(part_ml), B, nh, nkv, d, page_size, max_pages, int(max_splits),
                                               int(split), int(window), float(scale), float(softcap), int(bool(sink)),
-                                              _stream()), "decode_attention")
+                                              *_attn_form("decode_attention", nh, T, int(window), bool(sink), int(chunk),
+                                                          sink_score, gate, gate_col), _stream()), "decode_attention")
     return out
 
 
@@ -800,12 +823,13 @@ def dense_skinny_takes(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def dense_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                 swiglu_pair: bool = False, activation: str = "silu") -> torch.Tensor:
+                 swiglu_pair: bool = False, activation: str = "silu", squared_relu: bool = False) -> torch.Tensor:
     """``x @ w.T (+ bias)`` for a step of a few tokens (decode), every weight read once.
 
     ``x`` [T, K] and ``w`` [N, K] bfloat16, ``bias`` float32 [N] or None.  Returns float32
     [T, N]; with ``swiglu_pair`` the rows of ``w`` are N/2 gate rows then N/2 up rows and the
-    result is ``silu(gate) * up`` (``activation`` ``relu``: ``max(gate, 0) * up``) as bfloat16 [T, N/2].
+    result is ``silu(gate) * up`` (``activation`` ``relu``: ``max(gate, 0) * up``) as bfloat16 [T, N/2].  With
+    ``squared_relu`` the result is ``max(., 0)^2`` of the product as bfloat16 [T, N].
     """
     _chk(x, "dense_skinny x", BF16)
     T, Kd = x.shape
@@ -816,10 +840,10 @@ def dense_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
     nout = wrows // 2 if swiglu_pair else wrows
     if bias is not None:
         _chk(bias, "dense_skinny bias", F32, (wrows,))
-    out = torch.empty(T, nout, dtype=BF16 if swiglu_pair else F32, device=x.device)
+    out = torch.empty(T, nout, dtype=BF16 if swiglu_pair or squared_relu else F32, device=x.device)
     check(library().mi_dense_skinny(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), T, nout, Kd,
-                                    {"silu": 1, "relu": 2}[activation] if swiglu_pair else 0, _stream()),
-          "dense_skinny")
+                                    {"silu": 1, "relu": 2}[activation] if swiglu_pair else (3 if squared_relu else 0),
+                                    _stream()), "dense_skinny")
     return out
 
 
@@ -1230,6 +1254,37 @@ def causal_conv_silu(x: torch.Tensor, col0: int, channels: int, w: torch.Tensor,
     return out
 
 
+def causal_conv(x: torch.Tensor, col0: int, channels: int, in_bias: Optional[torch.Tensor], w: torch.Tensor,
+                bias: Optional[torch.Tensor], state: torch.Tensor, state_offset: int, q_start: torch.Tensor,
+                req_of_token: torch.Tensor, state_slot: torch.Tensor) -> torch.Tensor:
+    """As :func:`causal_conv_silu` without an activation, on the inputs ``x + in_bias`` (``in_bias`` float32
+    ``[channels]`` or None): what lies before a request's first token is zero, not the bias, and the state holds the
+    inputs with it."""
+    _chk(x, "causal_conv x", F32)
+    T, ld = x.shape
+    C = int(channels)
+    _chk(w, "causal_conv w", None, (C, None))
+    taps = w.shape[1]
+    _chk(bias, "causal_conv bias", w.dtype, (C,))
+    _chk(in_bias, "causal_conv in_bias", F32, (C,))
+    _chk(state, "causal_conv state", F32)
+    if col0 < 0 or col0 + C > ld or state.dim() != 2 or state_offset + (taps - 1) * C > state.shape[1]:
+        raise ValueError("causal_conv: columns or state section out of range")
+    B = state_slot.numel()
+    _chk(q_start, "causal_conv q_start", I32, (B + 1,))
+    _chk(req_of_token, "causal_conv req_of_token", I32, (T,))
+    _chk(state_slot, "causal_conv state_slot", I32, (B,))
+    if DEBUG_BOUNDS:
+        _dbg_range(state_slot, 0, state.shape[0], "causal_conv state_slot")
+        _dbg_range(req_of_token, 0, B, "causal_conv req_of_token")
+    out = torch.empty(T, C, dtype=F32, device=x.device)
+    check(library().mi_causal_conv_plain(x.data_ptr() + 4 * col0, ld, _ptr(in_bias), _ptr(w), _ptr(bias),
+                                         _code(w, "causal_conv w"), state.data_ptr() + 4 * state_offset, state.shape[1],
+                                         _ptr(q_start), _ptr(req_of_token), _ptr(state_slot), _ptr(out), C, C, taps, T, B,
+                                         _stream()), "causal_conv")
+    return out
+
+
 def causal_conv_residual(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, state_offset: int,
                          q_start: torch.Tensor, req_of_token: torch.Tensor, state_slot: torch.Tensor,
                          out_dtype: torch.dtype) -> torch.Tensor:
@@ -1437,6 +1492,290 @@ def gated_group_rmsnorm(y: torch.Tensor, gate: torch.Tensor, gate_col: int, weig
 
 
 # --------------------------------------------------------------------------- #
+# matrix memories with one gate per head
+# --------------------------------------------------------------------------- #
+
+class LogGates:
+    """The gates of a matrix memory that come from the projections: a log input gate ``cap tanh((z + bi) / cap)`` from
+    the ``heads`` columns ``col_i ..`` and a log forget gate ``logsigmoid(cap tanh((z + bf) / cap))`` from ``col_f ..``."""
+
+    def __init__(self, col_i: int, col_f: int, bi: torch.Tensor, bf: torch.Tensor, cap: float):
+        self.col_i, self.col_f, self.bi, self.bf, self.cap = int(col_i), int(col_f), bi, bf, float(cap)
+
+
+class MemoryState:
+    """Where a request's memory lies in its float32 state row: ``S [heads, d, dv]`` at ``s``; with log gates ``n [heads,
+    d]`` at ``n`` and ``m [heads]`` at ``m``."""
+
+    def __init__(self, heads: int, d: int, dv: int, log_gates: bool):
+        up = lambda v: -(-v // 4) * 4                      # sections on 16-byte boundaries
+        self.heads, self.d, self.dv, self.log_gates = int(heads), int(d), int(dv), bool(log_gates)
+        self.s = 0
+        self.n = up(heads * d * dv)
+        self.m = self.n + (up(heads * d) if log_gates else 0)
+        self.floats = self.m + (up(heads) if log_gates else 0)
+
+
+def _chk_memory(what, proj, cols, st: MemoryState, state, q_start, state_slot):
+    _chk(proj, what + " proj", F32)
+    _chk(state, what + " state", F32)
+    B = state_slot.numel()
+    _chk(q_start, what + " q_start", I32, (B + 1,))
+    _chk(state_slot, what + " state_slot", I32, (B,))
+    sizes = (st.heads * st.d, st.heads * st.d, st.heads * st.dv)
+    if any(c < 0 or c + n > proj.shape[1] for c, n in zip(cols, sizes)) or st.floats > state.shape[1]:
+        raise ValueError(f"{what}: columns of the projections or the state are out of range")
+    if DEBUG_BOUNDS:
+        _dbg_range(state_slot, 0, state.shape[0], what + " state_slot")
+    return B
+
+
+def _chk_gates(what, proj, gates, decay, heads):
+    if (gates is None) == (decay is None):
+        raise ValueError(f"{what}: either log gates or fixed decays")
+    _chk(decay, what + " decay", F32, (heads,))
+    if gates is not None:
+        _chk(gates.bi, what + " bi", F32, (heads,))
+        _chk(gates.bf, what + " bf", F32, (heads,))
+        if gates.col_i + heads > proj.shape[1] or gates.col_f + heads > proj.shape[1]:
+            raise ValueError(f"{what}: the gates' columns are out of range")
+
+
+def memory_chunk_tokens() -> int:
+    """Tokens per chunk of :func:`memory_scan` with ``chunks``."""
+    return int(library().mi_memory_chunk_tokens())
+
+
+def memory_scan(proj: torch.Tensor, cols: Tuple[int, int, int], st: MemoryState, state: torch.Tensor,
+                q_start: torch.Tensor, state_slot: torch.Tensor, gates: Optional[LogGates] = None,
+                decay: Optional[torch.Tensor] = None, q_scale: float = 1.0, silu: bool = False, chunks: bool = False,
+                max_q_len: int = 0):
+    """``S <- keep S + write k v^T``, ``o = S^T q`` per head over every request's portion; q, k (``heads x d``) and v
+    (``heads x dv``) are the columns ``cols`` of the float32 rows ``proj``, through silu first with ``silu``; q also
+    times ``q_scale``.
+
+    ``decay`` (float32 ``[heads]``): ``keep = decay``, ``write = 1``; returns ``o`` float32 ``[T, heads*dv]``.
+    ``gates``: with a running maximum ``m <- max(f + m, i)``, ``keep = exp(f + m_before - m)``, ``write = exp(i - m)``,
+    and ``n <- keep n + write k`` beside S; returns ``(o, n . q [T, heads], gates [T, heads, 4])`` for
+    :func:`memory_finish` (``gates[..., 2] = exp(-m)``).
+
+    The walk goes token by token in one order whatever the cut of a step.  ``chunks`` (bfloat16 path): on the tensor
+    cores over chunks of :func:`memory_chunk_tokens` tokens, q, k and v rounded to bfloat16, what the recurrence makes
+    held in float (as pairs of bfloat16 where it is an operand); ``max_q_len`` is the longest portion."""
+    what = "memory_scan"
+    B = _chk_memory(what, proj, cols, st, state, q_start, state_slot)
+    H, d, dv = st.heads, st.d, st.dv
+    _chk_gates(what, proj, gates, decay, H)
+    T, dev, lib = proj.shape[0], proj.device, library()
+    new = lambda *shape: torch.empty(*shape, dtype=F32, device=dev)
+    g = logs = den = None
+    if gates is not None:
+        g, den = new(T, H, 4), new(T, H)
+        logs = new(T, H, 4) if chunks else None
+        check(lib.mi_memory_gates(_ptr(proj), proj.shape[1], gates.col_i, gates.col_f, _ptr(gates.bi), _ptr(gates.bf),
+                                  gates.cap, _ptr(state), state.shape[1], st.m, _ptr(q_start), _ptr(state_slot), _ptr(g),
+                                  _ptr(logs), B, H, _stream()), "memory_gates")
+    out = new(T, H * dv)
+    head = (_ptr(proj), proj.shape[1], int(cols[0]), int(cols[1]), int(cols[2]), int(bool(silu)), float(q_scale),
+            _ptr(state), state.shape[1], st.s, st.n)
+    if chunks:
+        n = T // memory_chunk_tokens() + B
+        U, keep = new(n * H * d * dv), new(n * H)
+        Un = new(n * H * d) if gates is not None else None
+        check(lib.mi_memory_chunks(*head, _ptr(g), _ptr(logs), _ptr(decay), _ptr(q_start), _ptr(state_slot), _ptr(out),
+                                   _ptr(den), _ptr(U), _ptr(Un), _ptr(keep), B, int(max_q_len), H, d, dv, _stream()),
+              "memory_chunks")
+    else:
+        check(lib.mi_memory_walk(*head, _ptr(g), _ptr(decay), _ptr(q_start), _ptr(state_slot), _ptr(out), _ptr(den), B, H,
+                                 d, dv, _stream()), "memory_walk")
+    return out if gates is None else (out, den, g)
+
+
+def memory_finish(o: torch.Tensor, den: torch.Tensor, gates: torch.Tensor, gate: torch.Tensor, gate_col: int,
+                  weight: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """``rmsnorm_head(o / (max(|den|, gates[..., 2]) + 1e-6)) * weight * logistic(gate)`` with a weight per column."""
+    T, n = o.shape
+    H = den.shape[1]
+    dv = n // H
+    _chk(o, "memory_finish o", F32)
+    _chk(den, "memory_finish den", F32, (T, H))
+    _chk(gates, "memory_finish gates", F32, (T, H, 4))
+    _chk(gate, "memory_finish gate", F32, (T, None))
+    _chk(weight, "memory_finish weight", F32, (n,))
+    if gate_col + n > gate.shape[1]:
+        raise ValueError("memory_finish: the gate's columns are out of range")
+    out = torch.empty(T, n, dtype=out_dtype, device=o.device)
+    check(library().mi_memory_finish(_ptr(o), _ptr(den), _ptr(gates), gate.data_ptr() + 4 * gate_col, gate.shape[1],
+                                     _ptr(weight), _ptr(out), _code(out, "memory_finish out"), T, H, dv, float(eps),
+                                     _stream()), "memory_finish")
+    return out
+
+
+def memory_decode(proj: torch.Tensor, cols: Tuple[int, int, int], st: MemoryState, state: torch.Tensor,
+                  q_start: torch.Tensor, state_slot: torch.Tensor, gates: Optional[LogGates] = None,
+                  decay: Optional[torch.Tensor] = None, q_scale: float = 1.0, silu: bool = False, gate_col: int = 0,
+                  weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  out_dtype: torch.dtype = F32) -> torch.Tensor:
+    """:func:`memory_scan` when every request brings exactly ONE token, in one launch.  With ``gates`` the finished row
+    (:func:`memory_finish`, the output gate in the columns ``gate_col ..`` of ``proj``) in ``out_dtype``; with ``decay``
+    the read-out as float32."""
+    what = "memory_decode"
+    B = _chk_memory(what, proj, cols, st, state, q_start, state_slot)
+    H, d, dv = st.heads, st.d, st.dv
+    _chk_gates(what, proj, gates, decay, H)
+    T = proj.shape[0]
+    if T != B:
+        raise ValueError(f"memory_decode: {T} tokens for {B} requests; each request brings exactly one")
+    out = torch.empty(T, H * dv, dtype=F32 if gates is None else out_dtype, device=proj.device)
+    if gates is not None:
+        _chk(weight, what + " weight", F32, (H * dv,))
+        if weight is None or gate_col + H * dv > proj.shape[1]:
+            raise ValueError("memory_decode: the output norm's weight is missing or the gate's columns are out of range")
+    ci, cf, bi, bf, cap = (gates.col_i, gates.col_f, gates.bi, gates.bf, gates.cap) if gates else (0, 0, None, None, 1.0)
+    check(library().mi_memory_decode(
+        _ptr(proj), proj.shape[1], int(cols[0]), int(cols[1]), int(cols[2]), int(bool(silu)), float(q_scale), ci, cf,
+        _ptr(bi), _ptr(bf), cap, _ptr(state), state.shape[1], st.s, st.n, st.m, _ptr(decay), _ptr(q_start),
+        _ptr(state_slot), int(gate_col), _ptr(weight), float(eps), _ptr(out) if gates else None,
+        _code(out, what + " out"), None if gates else _ptr(out), B, H, d, dv, _stream()), what)
+    return out
+
+
+# --------------------------------------------------------------------------- #
+# a gated linear recurrence per channel
+# --------------------------------------------------------------------------- #
+
+def lru_segment_tokens() -> int:
+    """Tokens per segment of :func:`lru_scan` with ``segments``."""
+    return int(library().mi_lru_segment_tokens())
+
+
+def lru_gates(u: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor):
+    """``(a, x)`` float32 ``[T, W]`` of a real-gated linear recurrence: with ``u [T, W]`` float32 in ``W / n`` equal
+    parts, ``r = logistic(wr_b u_b + br)``, ``i = logistic(wi_b u_b + bi)`` (``wr``, ``wi`` ``[W/n, n, n]``),
+    ``a = exp(-8 r softplus(lam))`` and ``x = sqrt(1 - a^2) i u``.  Matrices in bfloat16: tensor cores with ``u`` as
+    three bfloat16 parts; in float32: the fixed-order products of :func:`dense_f32_heads`."""
+    _chk(u, "lru_gates u", F32)
+    T, W = u.shape
+    P, n, _ = wr.shape
+    _chk(wr, "lru_gates wr", None, (P, n, n))
+    _chk(wi, "lru_gates wi", wr.dtype, (P, n, n))
+    if P * n != W:
+        raise ValueError(f"lru_gates: {P} parts of {n} for rows of {W}")
+    for t, name in ((br, "br"), (bi, "bi"), (lam, "lam")):
+        _chk(t, "lru_gates " + name, F32, (W,))
+    if wr.dtype == BF16:
+        a, x = torch.empty_like(u), torch.empty_like(u)
+        check(library().mi_lru_gates_tc(_ptr(u), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(lam), _ptr(a), _ptr(x), T, W,
+                                        n, _stream()), "lru_gates")
+        return a, x
+    zr, zi = dense_f32_heads(u, wr), dense_f32_heads(u, wi)
+    check(library().mi_lru_prepare(_ptr(u), _ptr(zr), _ptr(zi), _ptr(br), _ptr(bi), _ptr(lam), T, W, _stream()),
+          "lru_prepare")
+    return zr, zi
+
+
+def lru_scan(a: torch.Tensor, x: torch.Tensor, y: torch.Tensor, y_col: int, y_bias: torch.Tensor, state: torch.Tensor,
+             state_offset: int, q_start: torch.Tensor, state_slot: torch.Tensor, out_dtype: torch.dtype,
+             segments: bool = False, max_q_len: int = 0) -> torch.Tensor:
+    """``S <- a S + x`` per channel over every request's portion; returns ``S * gelu_tanh(y + y_bias)`` (``y``: the
+    columns ``y_col ..``).  ``S`` lives in ``state[slot, state_offset:]``.  ``segments``: segments of
+    :func:`lru_segment_tokens` tokens side by side, their carries chained (the sums then run in another order)."""
+    _chk(a, "lru_scan a", F32)
+    T, W = a.shape
+    _chk(x, "lru_scan x", F32, (T, W))
+    _chk(y, "lru_scan y", F32, (T, None))
+    _chk(y_bias, "lru_scan y_bias", F32, (W,))
+    _chk(state, "lru_scan state", F32)
+    B = state_slot.numel()
+    _chk(q_start, "lru_scan q_start", I32, (B + 1,))
+    _chk(state_slot, "lru_scan state_slot", I32, (B,))
+    if y_col + W > y.shape[1] or state_offset + W > state.shape[1]:
+        raise ValueError("lru_scan: columns or state section out of range")
+    if DEBUG_BOUNDS:
+        _dbg_range(state_slot, 0, state.shape[0], "lru_scan state_slot")
+    out = torch.empty(T, W, dtype=out_dtype, device=a.device)
+    sa = ss = None
+    if segments:
+        n = T // lru_segment_tokens() + B
+        sa, ss = (torch.empty(n * W, dtype=F32, device=a.device) for _ in range(2))
+    check(library().mi_lru_scan(_ptr(a), _ptr(x), y.data_ptr() + 4 * y_col, y.shape[1], _ptr(y_bias), _ptr(sa), _ptr(ss),
+                                state.data_ptr() + 4 * state_offset, state.shape[1], _ptr(q_start), _ptr(state_slot),
+                                _ptr(out), _code(out, "lru_scan out"), B, max(int(max_q_len), 1), W, _stream()), "lru_scan")
+    return out
+
+
+def lru_decode(proj: torch.Tensor, x_col: int, y_col: int, x_bias: torch.Tensor, conv: torch.Tensor,
+               conv_bias: torch.Tensor, y_bias: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor,
+               bi: torch.Tensor, lam: torch.Tensor, state: torch.Tensor, s_off: int, c_off: int, q_start: torch.Tensor,
+               state_slot: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """:func:`causal_conv`, :func:`lru_gates` and :func:`lru_scan` when every request brings exactly ONE token, in one
+    launch (matrices in bfloat16; the convolution's state from ``c_off`` on, the recurrence's from ``s_off`` on)."""
+    what = "lru_decode"
+    _chk(proj, what + " proj", F32)
+    T = proj.shape[0]
+    P, n, _ = wr.shape
+    W = P * n
+    _chk(wr, what + " wr", BF16, (P, n, n))
+    _chk(wi, what + " wi", BF16, (P, n, n))
+    _chk(conv, what + " conv", F32, (W, None))
+    taps = conv.shape[1]
+    for t in (x_bias, conv_bias, y_bias, br, bi, lam):
+        _chk(t, what + " vector", F32, (W,))
+    _chk(state, what + " state", F32)
+    B = state_slot.numel()
+    _chk(q_start, what + " q_start", I32, (B + 1,))
+    _chk(state_slot, what + " state_slot", I32, (B,))
+    if T != B:
+        raise ValueError(f"lru_decode: {T} tokens for {B} requests; each request brings exactly one")
+    if max(x_col, y_col) + W > proj.shape[1] or max(s_off + W, c_off + (taps - 1) * W) > state.shape[1]:
+        raise ValueError("lru_decode: columns or state sections out of range")
+    if DEBUG_BOUNDS:
+        _dbg_range(state_slot, 0, state.shape[0], what + " state_slot")
+    out = torch.empty(T, W, dtype=out_dtype, device=proj.device)
+    check(library().mi_lru_decode(_ptr(proj), proj.shape[1], int(x_col), int(y_col), _ptr(x_bias), _ptr(conv),
+                                  _ptr(conv_bias), _ptr(y_bias), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(lam),
+                                  _ptr(state), state.shape[1], int(s_off), int(c_off), _ptr(q_start), _ptr(state_slot),
+                                  _ptr(out), _code(out, what + " out"), B, W, n, taps, _stream()), what)
+    return out
+
+
+# --------------------------------------------------------------------------- #
+# two outputs normalised by themselves; squared rectifier
+# --------------------------------------------------------------------------- #
+
+def normed_pair_add(hidden: torch.Tensor, pair, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                    out_dtype: torch.dtype = F32, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """``hidden += a y1 / rms(y1) * w1 + b y2 / rms(y2) * w2`` with ``pair = ((y1, w1, a, eps1), (y2, w2, b, eps2))``, and,
+    with ``weight``, the RMS norm of the new rows in the same launch.  ``rows`` (int32, with ``weight``) selects and
+    orders the rows to normalise; ``hidden`` is then left untouched."""
+    _chk(hidden, "normed_pair_add hidden", F32)
+    T, H = hidden.shape
+    (y1, w1, a, e1), (y2, w2, b, e2) = pair
+    for t in (y1, y2):
+        _chk(t, "normed_pair_add y", F32, (T, H))
+    for t in (w1, w2):
+        _chk(t, "normed_pair_add weight of an output", F32, (H,))
+    _chk(weight, "normed_pair_add weight", None, (H,))
+    _chk(rows, "normed_pair_add rows", I32)
+    if DEBUG_BOUNDS:
+        _dbg_range(rows, 0, T, "normed_pair_add rows")
+    n = T if rows is None else rows.numel()
+    out = None if weight is None else torch.empty(n, H, dtype=out_dtype, device=hidden.device)
+    check(library().mi_normed_pair_add(
+        _ptr(hidden), _ptr(y1), _ptr(w1), float(a), float(e1), _ptr(y2), _ptr(w2), float(b), float(e2), _ptr(rows),
+        _ptr(weight), 0 if weight is None else _code(weight, "normed_pair_add weight"), _ptr(out),
+        0 if out is None else _code(out, "normed_pair_add out"), n, H, float(eps), _stream()), "normed_pair_add")
+    return out
+
+
+def squared_relu_(x: torch.Tensor) -> torch.Tensor:
+    """``max(x, 0)^2`` in place."""
+    _chk(x, "squared_relu x")
+    check(library().mi_squared_relu(_ptr(x), _ptr(x), _code(x, "squared_relu x"), x.numel(), _stream()), "squared_relu")
+    return x
+
+
+# --------------------------------------------------------------------------- #
 # attention with capped scores mixed over the heads
 # --------------------------------------------------------------------------- #
 
@@ -1445,7 +1784,8 @@ def rope_store(qkv: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
                dk: int, dv: int, page_size: int, out_dtype: torch.dtype,
                q_gain: Optional[torch.Tensor] = None, k_gain: Optional[torch.Tensor] = None,
                eps: float = 0.0, neighbours: bool = False, v_first: Optional[torch.Tensor] = None,
-               blend: Optional[torch.Tensor] = None) -> torch.Tensor:
+               blend: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, values_are_keys: bool = False,
+               norm: Optional[str] = None, magnitude: float = 1.0) -> torch.Tensor:
     """Rotary encoding of the first ``rot_dim`` dimensions of the query and key heads of float32 rows
     ``[nh*dk | nkv*dk | nkv*dv]``, cache write of keys ``[pages, nkv, page_size, dk]`` and values
     ``[pages, nkv, page_size, dv]`` (slot -1: not written).  With ``q_gain`` and ``k_gain`` (float32
@@ -1453,7 +1793,11 @@ def rope_store(qkv: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
     multiplied by the gain.  The rotation pairs dimension ``i`` with ``i + rot_dim / 2``, or, with
     ``neighbours``, dimension ``2i`` with ``2i + 1``.  With ``v_first`` (float32 ``[T, nkv*dv]``; rows may be a
     column slice of a wider matrix) and ``blend`` (one float32 on the device) the values that are cached are
-    ``(1 - blend) v + blend v_first``.  Returns ``q [T, nh, dk]`` in ``out_dtype``."""
+    ``(1 - blend) v + blend v_first``.  The rows may go on with columns that are not read.  ``bias`` (float32, a number
+    per column of q, k and v) is added first.  ``values_are_keys``: the rows hold no values; a token's value is its key
+    as projected (with its bias), before norm and rotation (``dv = dk``).  ``norm`` says where the head norm stands,
+    ``"before"`` the rotation (default with gains) or ``"after"`` it, with or without gains.  ``magnitude`` multiplies
+    cosines and sines.  Returns ``q [T, nh, dk]`` in ``out_dtype``."""
     vf_stride = 0
     if v_first is not None:
         if (not v_first.is_cuda or v_first.dtype != F32 or v_first.dim() != 2 or v_first.stride(1) != 1
@@ -1467,7 +1811,14 @@ def rope_store(qkv: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
     _chk(k_gain, "rope_store k_gain", F32, (dk,))
     _chk(qkv, "rope_store qkv", F32)
     T = qkv.shape[0]
-    _chk(qkv, "rope_store qkv", F32, (T, (nh + nkv) * dk + nkv * dv))
+    width = (nh + nkv) * dk + (0 if values_are_keys else nkv * dv)
+    if qkv.dim() != 2 or qkv.shape[1] < width or (values_are_keys and dk != dv):
+        raise ValueError(f"rope_store: rows of {tuple(qkv.shape)} for q, k and v of {width} columns")
+    if norm not in (None, "before", "after"):
+        raise ValueError(f"rope_store: norm '{norm}' is not 'before' or 'after'")
+    form = {"before": 1, "after": 2}[norm] if norm else (1 if q_gain is not None else 0)
+    _chk(bias, "rope_store bias", F32, (width,))
+    v_col = nh * dk if values_are_keys else (nh + nkv) * dk
     _chk(positions, "rope_store positions", I32, (T,))
     _chk(inv_freq, "rope_store inv_freq", F32)
     if rot_dim and (inv_freq is None or inv_freq.numel() != rot_dim // 2):
@@ -1478,23 +1829,28 @@ def rope_store(qkv: torch.Tensor, positions: torch.Tensor, inv_freq: Optional[to
     q = torch.empty(T, nh, dk, dtype=out_dtype, device=qkv.device)
     if DEBUG_BOUNDS:
         _dbg_range(slot_mapping, -1, k_cache.shape[0] * page_size, "rope_store slot_mapping")
-    check(library().mi_rope_store(_ptr(qkv), _ptr(positions), _ptr(inv_freq), _ptr(slot_mapping), _ptr(q),
+    check(library().mi_rope_store_form(_ptr(qkv), _ptr(positions), _ptr(inv_freq), _ptr(slot_mapping), _ptr(q),
                                   _ptr(k_cache), _ptr(v_cache), _code(q, "rope_store q"), T, nh, nkv, dk, dv,
                                   int(rot_dim), page_size, _ptr(q_gain), _ptr(k_gain), float(eps),
                                   int(bool(neighbours)), _ptr(v_first), int(vf_stride),
-                                  _ptr(blend) if v_first is not None else None, _stream()),
+                                  _ptr(blend) if v_first is not None else None, qkv.shape[1], v_col, _ptr(bias), form,
+                                  float(magnitude), _stream()),
           "rope_store")
     return q
 
 
-def attention_mix_supported(nh: int, nkv: int, dk: int, dv: int, dtype: torch.dtype) -> bool:
-    return bool(library().mi_attn_mix_supported(nh, nkv, dk, dv, 4 if dtype == F32 else 2))
+def attention_mix_supported(nh: int, nkv: int, dk: int, dv: int, dtype: torch.dtype, independent: bool = False) -> bool:
+    """``independent``: heads that exchange nothing (no mix), which several blocks may share."""
+    fn = library().mi_attn_mix_independent_supported if independent else library().mi_attn_mix_supported
+    return bool(fn(nh, nkv, dk, dv, 4 if dtype == F32 else 2))
 
 
 def attention_mix(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, mix: Optional[torch.Tensor],
                   block_table: torch.Tensor, q_start: torch.Tensor, kv_len: torch.Tensor, max_q_len: int,
                   window: int, scale: float, softcap: float, keep_first: int = 0,
-                  value_dim: int = 0, sink: bool = False, head_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  value_dim: int = 0, sink: bool = False, head_bias: Optional[torch.Tensor] = None, chunk: int = 0,
+                  sink_score: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                  gate_col: int = 0) -> torch.Tensor:
     """Attention of a ragged batch over the paged cache with ``score <- softcap * tanh(score / softcap)``
     (``softcap`` 0: none) and then ``score_h <- sum_g mix[h, g] score_g`` (``mix`` None: none) before the
     softmax over the visible keys: key ``j`` is visible from position ``p`` iff ``j <= p`` and (``window`` is
@@ -1503,6 +1859,10 @@ def attention_mix(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     softmax counts one key more, of score 0 and without a value: ``p_j = exp(s_j) / (1 + sum exp(s_j))``.
     With ``head_bias`` (float32 ``[nh]``) there is no softmax: a visible key's weight is
     ``logistic(score + head_bias[h])`` by itself, not normalised over the keys.
+    With ``chunk`` (then no window) a query sees the keys of its own chunk of ``chunk`` positions only, counted from
+    the request's first token.  ``sink_score`` (float32 ``[nh]``, with ``sink``) gives the key more a score per head,
+    which is not scaled.  With ``gate`` (float32 rows, ``nh`` columns from ``gate_col`` on) head ``h``'s output is
+    multiplied by ``logistic(gate[t, gate_col + h])``.
     Returns ``[T, nh, dv]``."""
     _chk(q, "attention_mix q")
     _chk(head_bias, "attention_mix head_bias", F32, (q.shape[1],))
@@ -1524,18 +1884,13 @@ def attention_mix(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
     out = torch.empty(T, nh, dv, dtype=q.dtype, device=q.device)
     if DEBUG_BOUNDS:
         _dbg_batch("attention_mix", q_start, kv_len, block_table, T, k_cache.shape[0], page_size, int(window),
-                   int(max_q_len))
-    if head_bias is not None:
-        check(library().mi_attn_mix_form(_ptr(q), _ptr(k_cache), _ptr(v_cache), _code(q, "attention_mix q"), _ptr(mix),
-                                         _ptr(block_table), _ptr(q_start), _ptr(kv_len), _ptr(out), B, int(max_q_len),
-                                         nh, nkv, dk, dv, page_size, max_pages, int(window), float(scale),
-                                         float(softcap), int(keep_first), vrs, int(bool(sink)), _ptr(head_bias),
-                                         _stream()), "attention_mix")
-        return out
-    check(library().mi_attn_mix(_ptr(q), _ptr(k_cache), _ptr(v_cache), _code(q, "attention_mix q"), _ptr(mix),
-                                _ptr(block_table), _ptr(q_start), _ptr(kv_len), _ptr(out), B, int(max_q_len), nh, nkv,
-                                dk, dv, page_size, max_pages, int(window), float(scale), float(softcap),
-                                int(keep_first), vrs, int(bool(sink)), _stream()), "attention_mix")
+                   int(max_q_len), int(chunk))
+    check(library().mi_attn_mix_form(_ptr(q), _ptr(k_cache), _ptr(v_cache), _code(q, "attention_mix q"), _ptr(mix),
+                                     _ptr(block_table), _ptr(q_start), _ptr(kv_len), _ptr(out), B, int(max_q_len),
+                                     nh, nkv, dk, dv, page_size, max_pages, int(window), float(scale), float(softcap),
+                                     int(keep_first), vrs, int(bool(sink)), _ptr(head_bias),
+                                     *_attn_form("attention_mix", nh, T, int(window), bool(sink), int(chunk), sink_score,
+                                                 gate, gate_col), _stream()), "attention_mix")
     return out
 
 
@@ -1555,7 +1910,9 @@ def attention_mix_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      window: int, scale: float, softcap: float, splits: int = 1,
                      part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                      keep_first: int = 0, value_dim: int = 0, sink: bool = False,
-                     head_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     head_bias: Optional[torch.Tensor] = None, chunk: int = 0,
+                     sink_score: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                     gate_col: int = 0) -> torch.Tensor:
     """:func:`attention_mix` on the tensor cores (bfloat16).  ``splits > 1`` (steps of one token per request
     only): the keys of a request are cut into ``splits`` blocks whose partial results go through the float32
     scratch ``part_o`` (``B * splits * nh * dv``) and ``part_ml`` (``B * splits * nh * 2``); with
@@ -1582,18 +1939,14 @@ def attention_mix_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     out = torch.empty(T, nh, dv, dtype=BF16, device=q.device)
     if DEBUG_BOUNDS:
         _dbg_batch("attention_mix_tc", q_start, kv_len, block_table, T, k_cache.shape[0], page_size, int(window),
-                   int(max_q_len))
-    if head_bias is not None:
-        check(library().mi_attn_mix_tc_form(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(mix), _ptr(block_table),
-                                            _ptr(q_start), _ptr(kv_len), _ptr(out), _ptr(part_o), _ptr(part_ml), B,
-                                            int(max_q_len), nh, nkv, dk, dv, page_size, max_pages, int(window),
-                                            float(scale), float(softcap), int(splits), int(keep_first), vrs,
-                                            int(bool(sink)), _ptr(head_bias), _stream()), "attention_mix_tc")
-        return out
-    check(library().mi_attn_mix_tc(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(mix), _ptr(block_table), _ptr(q_start),
-                                   _ptr(kv_len), _ptr(out), _ptr(part_o), _ptr(part_ml), B, int(max_q_len), nh, nkv, dk,
-                                   dv, page_size, max_pages, int(window), float(scale), float(softcap), int(splits),
-                                   int(keep_first), vrs, int(bool(sink)), _stream()), "attention_mix_tc")
+                   int(max_q_len), int(chunk))
+    check(library().mi_attn_mix_tc_form(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(mix), _ptr(block_table),
+                                        _ptr(q_start), _ptr(kv_len), _ptr(out), _ptr(part_o), _ptr(part_ml), B,
+                                        int(max_q_len), nh, nkv, dk, dv, page_size, max_pages, int(window),
+                                        float(scale), float(softcap), int(splits), int(keep_first), vrs,
+                                        int(bool(sink)), _ptr(head_bias),
+                                        *_attn_form("attention_mix_tc", nh, T, int(window), bool(sink), int(chunk),
+                                                    sink_score, gate, gate_col), _stream()), "attention_mix_tc")
     return out
 
 

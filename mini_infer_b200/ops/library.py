@@ -29,7 +29,7 @@ _SIGNATURES = {
     "mi_attn_tiled": [P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
     "mi_attn_decode": [P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
     "mi_attn_decode_split": [P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
-    "mi_attn_decode_split_form": [P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, P],
+    "mi_attn_decode_split_form": [P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, P, P, L, P],
     "mi_moe_router": [P, I, P, P, I, P, P, P, P, P, I, I, I, I, I, P, P],
     "mi_moe_permute": [P, P, P, P, P, I, I, I, P],
     "mi_grouped_gemm_plain": [P, I, P, P, I, P, P, I, I, I, I, I, I, I, F, F, P, P],
@@ -42,7 +42,7 @@ _SIGNATURES = {
     "mi_dense_skinny": [P, P, P, P, I, I, I, I, P],
     "mi_gather_rows_bf16": [P, P, P, I, I, P],
     "mi_attn_prefill": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P],
-    "mi_attn_prefill_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, F, I, P],
+    "mi_attn_prefill_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, F, I, I, P, P, L, P],
     "mi_grouped_gemm_tc": [P, P, P, P, P, I, I, I, I, I, I, F, F, P, P],
     "mi_grouped_gemm_tc_form": [P, P, P, P, P, I, I, I, I, I, I, I, F, F, P, P],
     "mi_random_fill": [P, I, L, ctypes.c_uint, ctypes.c_uint, F, F, P],
@@ -52,7 +52,7 @@ _SIGNATURES = {
     "mi_delta_scan": [P, I, P, I, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, I, F, P],
     "mi_ssd_scan": [P, I, P, I, P, P, P, P, L, P, P, P, I, I, I, I, I, P],
     "mi_gated_group_rmsnorm": [P, P, I, P, I, I, P, I, I, I, I, I, F, P],
-    "mi_rope_store": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P, F, I, P, L, P, P],
+    "mi_rope_store_form": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P, F, I, P, L, P, L, I, P, I, F, P],
     "mi_attn_mix": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, P],
     "mi_attn_mix_tc": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, I, P],
     "mi_out_norm_add": [P, P, P, P, P, P, P, I, P, I, P, I, I, I, F, F, P],
@@ -82,11 +82,23 @@ _SIGNATURES = {
     "mi_norm_conv_decode": [P, P, I, F, P, P, L, P, P, P, I, I, I, I, P],
     "mi_delta_scan_form": [P, I, P, I, P, I, P, P, P, L, P, P, P, P, I, I, I, I, I, I, F, I, F, P],
     "mi_gla_scan_segments": [P, I, P, I, P, P, L, P, P, P, P, I, I, I, I, I, F, F, I, I, P, P, P, P],
-    "mi_attn_mix_form": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, P, P],
-    "mi_attn_mix_tc_form": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, I, P, P],
+    "mi_attn_mix_form": [P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, P, I, P, P, L, P],
+    "mi_attn_mix_tc_form": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, I, I, I, P, I, P, P, L, P],
     "mi_attn_prefill_tc_logistic": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P],
     "mi_group_rmsnorm": [P, P, P, I, P, I, I, I, I, F, P],
     "mi_out_norm_add_groups": [P, P, P, P, P, P, P, I, P, I, P, I, I, I, F, F, I, P],
+    "mi_normed_pair_add": [P, P, P, F, F, P, P, F, F, P, P, I, P, I, I, I, F, P],
+    "mi_squared_relu": [P, P, I, L, P],
+    "mi_causal_conv_plain": [P, I, P, P, P, I, P, L, P, P, P, P, I, I, I, I, I, P],
+    "mi_memory_gates": [P, I, I, I, P, P, F, P, L, L, P, P, P, P, I, I, P],
+    "mi_memory_walk": [P, I, I, I, I, I, F, P, L, L, L, P, P, P, P, P, P, I, I, I, I, P],
+    "mi_memory_chunks": [P, I, I, I, I, I, F, P, L, L, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
+    "mi_memory_finish": [P, P, P, P, I, P, P, I, I, I, I, F, P],
+    "mi_memory_decode": [P, I, I, I, I, I, F, I, I, P, P, F, P, L, L, L, L, P, P, P, I, P, F, P, I, P, I, I, I, I, P],
+    "mi_lru_gates_tc": [P, P, P, P, P, P, P, P, I, I, I, P],
+    "mi_lru_prepare": [P, P, P, P, P, P, I, I, P],
+    "mi_lru_scan": [P, P, P, I, P, P, P, P, L, P, P, P, I, I, I, I, P],
+    "mi_lru_decode": [P, I, I, I, P, P, P, P, P, P, P, P, P, P, L, L, L, P, P, P, I, I, I, I, I, P],
 }
 
 
@@ -111,6 +123,9 @@ _OTHERS = {
     "mi_attn_mix_tc_supported": ([I, I, I, I], c_int),
     "mi_attn_mix_tc_splits": ([I], c_int),
     "mi_attn_mix_supported": ([I, I, I, I, I], c_int),
+    "mi_attn_mix_independent_supported": ([I, I, I, I, I], c_int),
+    "mi_memory_chunk_tokens": ([], c_int),
+    "mi_lru_segment_tokens": ([], c_int),
     "mi_attn_prefill_tc_shared_supported": ([I, I, I, I], c_int),
     "mi_attn_prefill_tc_logistic_supported": ([I, I, I], c_int),
     "mi_attn_decode_split_size": ([], c_int),

@@ -292,6 +292,21 @@ class TensorSum(Deferred):
 
 
 @dataclass
+class NormedPair(Deferred):
+    """``a y1 / rms(y1) * w1 + b y2 / rms(y2) * w2``: the outputs of two parts that read the same input, each normalised by
+    itself; ``first`` and ``second`` are ``(y, weight, scale, eps)``."""
+
+    first: Tuple[torch.Tensor, torch.Tensor, float, float]
+    second: Tuple[torch.Tensor, torch.Tensor, float, float]
+
+    def materialize(self) -> torch.Tensor:
+        from ..ops import functional as F
+        out = torch.zeros_like(self.first[0])
+        F.normed_pair_add(out, (self.first, self.second))
+        return out
+
+
+@dataclass
 class RoundedResidual(Deferred):
     """Nothing is left to add: the residual stream is up to date, and ``x`` is its rounding to the activation
     type, which a block whose parts read the residual itself takes instead of rounding the rows again."""

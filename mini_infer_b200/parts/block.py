@@ -18,19 +18,86 @@ import torch
 from ..config.registry import part_class, register_part
 from ..ops import functional as F
 from .tuning import TUNING
-from .base import (Block, BuiltLayer, CacheBinding, Embedding, LMHead, RoundedResidual, Runtime, StepContext,
+from .base import (Block, BuiltLayer, CacheBinding, Embedding, LMHead, NormedPair, RoundedResidual, Runtime, StepContext,
                    StreamUpdate, TensorDecl, TensorSum, TokenNeed, WeightedRowSum, apply_norm, as_streams, linear,
                    read_streams, resolve, split_sum)
 
 
+def _mixer_pair(block: Block, layer: BuiltLayer, h: torch.Tensor, ctx: StepContext, caches):
+    """The outputs of ``mixer`` and ``mixer_b`` on the same input.  The two share nothing but the input they read: in
+    steps of few tokens, whose kernels are short chains that leave the device idle, the second one goes to a second
+    stream.  In a prompt step the walk of a recurrence beside the tensor-memory attention and the library's products,
+    whose blocks want whole SMs, lost 7 to 19 %, so large steps stay on one stream."""
+    if (TUNING.parallel_residual_two_streams and h.is_cuda
+            and ctx.num_tokens <= TUNING.parallel_residual_two_streams_max_tokens_full_sm_mixer):
+        main = torch.cuda.current_stream()
+        if block._side_stream is None:
+            block._side_stream = torch.cuda.Stream(device=h.device)
+        side = block._side_stream
+        side.wait_stream(main)
+        h.record_stream(side)
+        with torch.cuda.stream(side):
+            y2 = layer.mixer_b.forward(h, ctx, caches.get("mixer_b"))
+        y2.record_stream(main)
+        y = layer.mixer.forward(h, ctx, caches.get("mixer"))
+        main.wait_stream(side)
+        return y, y2
+    y = layer.mixer.forward(h, ctx, caches.get("mixer"))
+    return y, layer.mixer_b.forward(h, ctx, caches.get("mixer_b"))
+
+
 class PreNormResidual(Block):
+    """``a = x + Mixer(Norm1(x))``; ``y = a + FFN(Norm2(a))``.  params: ``feed_forward`` (default True; False: a layer of a
+    mixer alone, without the roles ``feed_forward_norm`` and ``feed_forward``); ``second_mixer`` (default False; True: two
+    mixers read ``Norm1(x)`` and what is added is ``s NormA(Mixer(h)) + t NormB(MixerB(h))``, with the roles ``mixer_b``,
+    ``mixer_out_norm`` and ``mixer_b_out_norm`` and the numbers ``mixer_scale`` and ``second_mixer_scale``, default 1;
+    the outputs' norms must be plain RMS norms).
+
+    The two normalised outputs travel on as a :class:`NormedPair`: one kernel takes both root mean squares, updates the
+    residual and runs the norm that follows."""
+
     graph_safe = True
     accepts_deferred = True
     roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
 
+    def __init__(self, params=None, prefix=""):
+        super().__init__(params or {}, prefix)
+        self.has_ff = bool(self.params.get("feed_forward", True))
+        self.second = bool(self.params.get("second_mixer", False))
+        self.scales = (float(self.params.get("mixer_scale", 1.0)), float(self.params.get("second_mixer_scale", 1.0)))
+        self._side_stream = None
+        self._weights = None
+        if self.second:
+            self.kernel_files = ("residual_forms.cu",)
+        if self.second or not self.has_ff:
+            self.roles = {"mixer_norm": "norm", "mixer": "mixer"}
+            if self.has_ff:
+                self.roles.update({"feed_forward_norm": "norm", "feed_forward": "feed_forward"})
+            if self.second:
+                self.roles.update({"mixer_b": "mixer", "mixer_out_norm": "norm", "mixer_b_out_norm": "norm"})
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        self._weights = None
+
+    def _out_norms(self, layer: BuiltLayer):
+        if self._weights is None:
+            rms = [n.rms_parameters() for n in (layer.mixer_out_norm, layer.mixer_b_out_norm)]
+            if None in rms:
+                raise ValueError("prenorm_residual: the norm of a mixer's output must be a plain RMS norm")
+            self._weights = [(w.to(torch.float32).contiguous(), eps) for w, eps in rms]
+        return self._weights
+
     def forward(self, layer: BuiltLayer, hidden: torch.Tensor, pending, ctx: StepContext, caches):
         x = apply_norm(layer.mixer_norm, hidden, pending)
-        y = layer.mixer.forward(x, ctx, caches.get("mixer"))
+        if self.second:
+            y, y2 = _mixer_pair(self, layer, x, ctx, caches)
+            (w, eps), (w2, eps2) = self._out_norms(layer)
+            y = NormedPair((y, w, self.scales[0], eps), (y2, w2, self.scales[1], eps2))
+        else:
+            y = layer.mixer.forward(x, ctx, caches.get("mixer"))
+        if not self.has_ff:
+            return y
         return layer.feed_forward.forward_from_residual(hidden, y, layer.feed_forward_norm, ctx)
 
     def prefetch_layer(self, layer: BuiltLayer, ctx: StepContext, caches) -> None:
@@ -311,29 +378,10 @@ class SandwichResidual(Block):
         if left is not None:
             hidden.add_(left)
         h = self._read(hidden, layer.mixer_norm, layer.mixer_conv if self.conv else None, ctx, caches.get("mixer_conv"))
-        y2 = None
-        if (self.second and TUNING.parallel_residual_two_streams and h.is_cuda
-                and ctx.num_tokens <= TUNING.parallel_residual_two_streams_max_tokens_full_sm_mixer):
-            # The two mixers share nothing but the input they read: in steps of few tokens, whose kernels are short
-            # chains that leave the device idle, the second one goes to a second stream (decode at batch 8: 0.538 ->
-            # 0.456 ms and 1.117 -> 1.005 ms at the two bench sizes).  In a prompt step the walk of the recurrence
-            # beside the tensor-memory attention and the library's products, whose blocks want whole SMs, lost 7 to
-            # 19 %, so large steps stay on one stream.
-            main = torch.cuda.current_stream()
-            if self._side_stream is None:
-                self._side_stream = torch.cuda.Stream(device=h.device)
-            side = self._side_stream
-            side.wait_stream(main)
-            h.record_stream(side)
-            with torch.cuda.stream(side):
-                y2 = layer.mixer_b.forward(h, ctx, caches.get("mixer_b"))
-            y2.record_stream(main)
-            y = layer.mixer.forward(h, ctx, caches.get("mixer"))
-            main.wait_stream(side)
+        if self.second:
+            y, y2 = _mixer_pair(self, layer, h, ctx, caches)
         else:
             y = layer.mixer.forward(h, ctx, caches.get("mixer"))
-            if self.second:
-                y2 = layer.mixer_b.forward(h, ctx, caches.get("mixer_b"))
         if self.second:
             # a * y + b * y2 is formed inside the output norm's kernel, as a sum of rows with weights
             wa, wb = self._weights(y.shape[0], y.device)

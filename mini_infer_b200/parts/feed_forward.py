@@ -107,6 +107,46 @@ class GatedMLP(FeedForward):
         return linear(F.geglu_tanh(linear(x, self.w_gate_up, self.rt.act)), self.w_down, torch.float32)
 
 
+class SquaredReluMLP(FeedForward):
+    """``max(x Wu^T, 0)^2 Wd^T``.  params: ``hidden_size``, ``intermediate_size``, optional ``up``, ``down`` (tensor names
+    below the prefix; default ``up_proj.weight`` and so on).
+
+    Tensors: ``<prefix><up> [I, H]``, ``<prefix><down> [H, I]``."""
+
+    graph_safe = True
+    kernel_files = ("residual_forms.cu", "moe_skinny.cu")
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        self.H = int(self.params["hidden_size"])
+        self.I = int(self.params["intermediate_size"])
+        self.names = [self.prefix + self.params.get(k, k + "_proj.weight") for k in ("up", "down")]
+
+    def tensor_decls(self) -> List[TensorDecl]:
+        u, d = self.names
+        return [TensorDecl(u, (self.I, self.H)), TensorDecl(d, (self.H, self.I))]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        self.w_up, self.w_down = (rt.precision.matrix(tensors[n], rt.device) for n in self.names)
+
+    def prefetch_first(self, ctx, cache=None) -> None:
+        F.l2_prefetch(self.w_up)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        if ctx is not None and ctx.prefetch is not None:
+            ctx.prefetch((self.w_down,))
+        if x.is_cuda and x.shape[0] <= TUNING.dense_skinny_max_tokens and F.dense_skinny_takes(x, self.w_up):
+            act = F.dense_skinny(x, self.w_up, squared_relu=True)
+        else:
+            act = F.squared_relu_(linear(x, self.w_up, self.rt.act))
+        y = linear(act, self.w_down, torch.float32)
+        if ctx is not None and ctx.prefetch is not None:
+            # while the next norm runs, the next layer's first weights arrive
+            ctx.prefetch(ctx.prefetch_upcoming)
+        return y
+
+
 class SparseMoE(FeedForward):
     """Softmax router, top-k routed SwiGLU experts, optional sigmoid-gated shared expert.
 
@@ -408,5 +448,6 @@ class SparseMoE(FeedForward):
 
 
 register_part("feed_forward", "gated_mlp", GatedMLP)
+register_part("feed_forward", "squared_relu_mlp", SquaredReluMLP)
 register_part("feed_forward", "swiglu_mlp", SwiGLUMLP)
 register_part("feed_forward", "sparse_moe", SparseMoE)

@@ -12,7 +12,7 @@ import torch
 
 from ..config.registry import register_part
 from ..ops import functional as F
-from .base import Deferred, Norm, Runtime, TensorDecl, WeightedRowSum, split_sum
+from .base import Deferred, Norm, NormedPair, Runtime, TensorDecl, WeightedRowSum, split_sum
 
 
 class RMSNorm(Norm):
@@ -53,6 +53,8 @@ class RMSNorm(Norm):
             # the sum is formed row by row inside the norm's kernel and never written out
             return F.combine_add_rmsnorm(hidden, delta.rows, delta.index, delta.weights, delta.extra, delta.scale,
                                          self.weight, self.eps, self.rt.act, rows)
+        if isinstance(delta, NormedPair):
+            return F.normed_pair_add(hidden, (delta.first, delta.second), self.weight, self.eps, self.rt.act, rows)
         if isinstance(delta, Deferred):
             delta = delta.materialize()
         return F.add_rmsnorm(hidden, delta, self.weight, self.eps, self.rt.act, rows)

@@ -23,7 +23,16 @@ state is the last ``taps - 1`` rows it read.
 ``dt = softplus(dt + dt_bias)``, ``x``, ``B``, ``C`` behind one causal convolution with bias and silu,
 ``y * silu(z)`` normalised in groups, through ``W_o``.
 
-Both keep ``S`` and the last ``taps - 1`` inputs of their convolutions in one float32 row per request
+``matrix_lstm``: matrix memory with exponential gates (mLSTM), ``S <- exp(f + m - m') S + exp(i - m') k v^T`` with a
+running maximum ``m' = max(f + m, i)``, ``n`` likewise with ``k`` alone, ``o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)``.
+
+``fixed_decay_attention``: linear attention with a constant decay per head, ``S <- decay S + k v^T``, ``o = S^T q``,
+q, k and v through silu.
+
+``gated_lru``: a linear recurrence per channel behind a short convolution, with gates that are products of the channels
+of one part, times a second branch through gelu.
+
+All keep what they carry (``S``, a running maximum, the last ``taps - 1`` inputs of their convolutions) in one float32 row per request
 (:class:`StateNeed`), are computed in float32 beyond the projections, and walk a request's tokens in order
 whatever the cut of the step.
 """
@@ -338,6 +347,225 @@ class GatedLinearAttention(Mixer):
         return linear(y, self.w_o, torch.float32)
 
 
+def _scan_in_chunks(rt: Runtime, ctx: StepContext) -> bool:
+    """Long portions of the bfloat16 path go over chunks on the tensor cores; the float32 path keeps one walk for every
+    step, so that its sums run in one order however a prompt was cut."""
+    return rt.act == torch.bfloat16 and ctx.max_q_len >= TUNING.memory_chunks_min_tokens
+
+
+class MatrixLSTM(Mixer):
+    """params: ``hidden_size``, ``num_heads``, ``head_dim`` (q, k), ``value_dim``, ``gate_cap`` (both gates' inputs ``z``
+    become ``cap tanh(z / cap)``), ``eps`` (of the output norm).
+
+    With ``q`` times ``head_dim^-1/2``, a log input gate ``i`` and a log forget gate ``f = logsigmoid(.)`` per head, the
+    memory described at the top of this file; every head's ``o`` is divided by its root mean square, the heads together
+    are multiplied by ``norm`` and ``sigmoid(W_g h)`` and go through ``W_o``.
+
+    Tensors below the prefix: ``q``, ``k`` ``[heads*head_dim, hidden]``, ``v``, ``g`` ``[heads*value_dim, hidden]``, ``i``,
+    ``f`` ``[heads, hidden]`` with ``i.b``, ``f.b`` ``[heads]``, ``norm [heads*value_dim]``,
+    ``o [hidden, heads*value_dim]``."""
+
+    graph_safe = True
+    kernel_files = ("matrix_memory.cu",)
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        p = self.params
+        self.H = int(p["hidden_size"])
+        self.nh = int(p["num_heads"])
+        self.d = int(p["head_dim"])
+        self.dv = int(p["value_dim"])
+        self.cap = float(p["gate_cap"])
+        self.eps = float(p["eps"])
+        if not self.cap > 0:
+            raise ValueError(f"matrix_lstm: gate_cap = {self.cap} must be positive")
+        if not 1 <= self.d <= 256:
+            raise ValueError(f"matrix_lstm: keys of {self.d} numbers (at most 256)")
+        self.n_qk = self.nh * self.d
+        self.n_v = self.nh * self.dv
+        self.state = F.MemoryState(self.nh, self.d, self.dv, True)
+
+    def tensor_decls(self) -> List[TensorDecl]:
+        p = self.prefix
+        return [TensorDecl(p + "q", (self.n_qk, self.H)), TensorDecl(p + "k", (self.n_qk, self.H)),
+                TensorDecl(p + "v", (self.n_v, self.H)), TensorDecl(p + "g", (self.n_v, self.H)),
+                TensorDecl(p + "o", (self.H, self.n_v)), TensorDecl(p + "norm", (self.n_v,), "norm"),
+                TensorDecl(p + "i", (self.nh, self.H)), TensorDecl(p + "i.b", (self.nh,), "bias"),
+                TensorDecl(p + "f", (self.nh, self.H)), TensorDecl(p + "f.b", (self.nh,), "bias")]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        m, dev, p = rt.precision.matrix, rt.device, self.prefix
+        # one product for everything that reads the layer's input: q | k | v | output gate | input gate | forget gate
+        self.w_in = torch.cat([m(tensors[p + n], dev) for n in ("q", "k", "v", "g", "i", "f")], dim=0)
+        self.cols = (0, self.n_qk, 2 * self.n_qk)
+        self.col_gate = 2 * self.n_qk + self.n_v
+        col_i = self.col_gate + self.n_v
+        self.gates = F.LogGates(col_i, col_i + self.nh, _f32(tensors[p + "i.b"], dev), _f32(tensors[p + "f.b"], dev), self.cap)
+        self.norm_w = _f32(tensors[p + "norm"], dev)
+        self.w_o = m(tensors[p + "o"], dev)
+
+    def prefetch_first(self, ctx: StepContext, cache: Optional[CacheBinding]) -> None:
+        F.l2_prefetch(self.w_in)
+
+    def cache_need(self):
+        return StateNeed((self.state.floats,), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
+        state = ctx.states[cache.group]
+        proj = linear(x, self.w_in, torch.float32)
+        if ctx.prefetch is not None:
+            ctx.prefetch((self.w_o,))       # arrives while the states are read and written
+        args = (proj, self.cols, self.state, state, ctx.q_start, ctx.state_slot)
+        if ctx.all_decode and self.rt.act == torch.bfloat16:
+            y = F.memory_decode(*args, gates=self.gates, q_scale=self.d ** -0.5, gate_col=self.col_gate,
+                                weight=self.norm_w, eps=self.eps, out_dtype=self.rt.act)
+        else:
+            o, den, g = F.memory_scan(*args, gates=self.gates, q_scale=self.d ** -0.5,
+                                      chunks=_scan_in_chunks(self.rt, ctx), max_q_len=ctx.max_q_len)
+            y = F.memory_finish(o, den, g, proj, self.col_gate, self.norm_w, self.eps, self.rt.act)
+        return linear(y, self.w_o, torch.float32)
+
+
+class FixedDecayAttention(Mixer):
+    """params: ``hidden_size``, ``num_heads``, ``head_dim`` (q, k), ``value_dim``, ``decay`` (a number in (0, 1] per head),
+    ``eps`` (of the output norm).
+
+    ``q = silu(W_q h)``, ``k = silu(W_k h)``, ``v = silu(W_v h)``; per head ``S <- decay S + k v^T``, ``o = S^T q``; the
+    heads together ``rmsnorm(o) * norm * sigmoid(W_g h)`` through ``W_o``.
+
+    Tensors below the prefix: ``q``, ``k`` ``[heads*head_dim, hidden]``, ``v``, ``g`` ``[heads*value_dim, hidden]``,
+    ``norm [heads*value_dim]``, ``o [hidden, heads*value_dim]``."""
+
+    graph_safe = True
+    kernel_files = ("matrix_memory.cu", "recurrent.cu")
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        p = self.params
+        self.H = int(p["hidden_size"])
+        self.nh = int(p["num_heads"])
+        self.d = int(p["head_dim"])
+        self.dv = int(p["value_dim"])
+        self.eps = float(p["eps"])
+        self.decay_values = [float(v) for v in p["decay"]]
+        if len(self.decay_values) != self.nh or not all(0.0 < v <= 1.0 for v in self.decay_values):
+            raise ValueError(f"fixed_decay_attention: decays {self.decay_values} are not {self.nh} numbers in (0, 1]")
+        if not 1 <= self.d <= 256:
+            raise ValueError(f"fixed_decay_attention: keys of {self.d} numbers (at most 256)")
+        self.n_qk = self.nh * self.d
+        self.n_v = self.nh * self.dv
+        self.state = F.MemoryState(self.nh, self.d, self.dv, False)
+
+    def tensor_decls(self) -> List[TensorDecl]:
+        p = self.prefix
+        return [TensorDecl(p + "q", (self.n_qk, self.H)), TensorDecl(p + "k", (self.n_qk, self.H)),
+                TensorDecl(p + "v", (self.n_v, self.H)), TensorDecl(p + "g", (self.n_v, self.H)),
+                TensorDecl(p + "o", (self.H, self.n_v)), TensorDecl(p + "norm", (self.n_v,), "norm")]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        m, dev, p = rt.precision.matrix, rt.device, self.prefix
+        self.w_in = torch.cat([m(tensors[p + n], dev) for n in ("q", "k", "v", "g")], dim=0)
+        self.cols = (0, self.n_qk, 2 * self.n_qk)
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=dev)
+        self.norm_w = _f32(tensors[p + "norm"], dev)
+        self.w_o = m(tensors[p + "o"], dev)
+
+    def prefetch_first(self, ctx: StepContext, cache: Optional[CacheBinding]) -> None:
+        F.l2_prefetch(self.w_in)
+
+    def cache_need(self):
+        return StateNeed((self.state.floats,), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
+        state = ctx.states[cache.group]
+        proj = linear(x, self.w_in, torch.float32)
+        args = (proj, self.cols, self.state, state, ctx.q_start, ctx.state_slot)
+        if ctx.all_decode and self.rt.act == torch.bfloat16:
+            o = F.memory_decode(*args, decay=self.decay, silu=True)
+        else:
+            o = F.memory_scan(*args, decay=self.decay, silu=True, chunks=_scan_in_chunks(self.rt, ctx),
+                              max_q_len=ctx.max_q_len)
+        y = F.gated_group_rmsnorm(o, proj, 2 * self.n_qk + self.n_v, self.norm_w, 1, False, self.eps, self.rt.act)
+        return linear(y, self.w_o, torch.float32)
+
+
+class GatedLRU(Mixer):
+    """Real-gated linear recurrent unit behind a short convolution, times a second branch.  params: ``hidden_size``,
+    ``width``, ``blocks`` (equal parts of the width whose gates read each other), ``conv`` (taps).
+
+    ``y = gelu_tanh(W_y h + b)``, ``u = conv(W_x h + b)`` (causal, per channel, with bias); per part ``r = sigmoid(ra u +
+    b)``, ``i = sigmoid(ri u + b)``; ``log a = -8 r softplus(lam)``, ``S <- a S + sqrt(1 - a^2) i u``; ``W_o (S y)``.
+
+    Tensors below the prefix: ``y``, ``x`` ``[width, hidden]`` with ``y.b``, ``x.b`` ``[width]``; ``conv [width, taps]``,
+    ``conv.b [width]``; ``ra``, ``ri`` ``[blocks, n, n]`` with ``ra.b``, ``ri.b`` ``[blocks, n]``; ``lam [width]``;
+    ``o [hidden, width]``."""
+
+    graph_safe = True
+    kernel_files = ("gated_lru.cu", "recurrent.cu")
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        p = self.params
+        self.H = int(p["hidden_size"])
+        self.W = int(p["width"])
+        self.blocks = int(p["blocks"])
+        self.taps = int(p["conv"])
+        if self.blocks < 1 or self.W % self.blocks:
+            raise ValueError(f"gated_lru: a width of {self.W} does not split into {self.blocks} blocks")
+        if not 1 <= self.taps <= F.CONV_MAX_TAPS:
+            raise ValueError(f"gated_lru: a convolution of {self.taps} taps (at most {F.CONV_MAX_TAPS})")
+        self.n = self.W // self.blocks
+        self.conv_off = -(-self.W // 4) * 4
+        self.floats = -(-(self.conv_off + (self.taps - 1) * self.W) // 4) * 4
+
+    def tensor_decls(self) -> List[TensorDecl]:
+        p, W, B, n = self.prefix, self.W, self.blocks, self.n
+        return [TensorDecl(p + "y", (W, self.H)), TensorDecl(p + "y.b", (W,), "bias"),
+                TensorDecl(p + "x", (W, self.H)), TensorDecl(p + "x.b", (W,), "bias"),
+                TensorDecl(p + "conv", (W, self.taps), "conv"), TensorDecl(p + "conv.b", (W,), "bias"),
+                TensorDecl(p + "ra", (B, n, n)), TensorDecl(p + "ra.b", (B, n), "bias"),
+                TensorDecl(p + "ri", (B, n, n)), TensorDecl(p + "ri.b", (B, n), "bias"),
+                TensorDecl(p + "lam", (W,), "bias"), TensorDecl(p + "o", (self.H, W))]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.rt = rt
+        m, dev, p = rt.precision.matrix, rt.device, self.prefix
+        vec = lambda name: _f32(tensors[p + name], dev).reshape(-1)
+        self.w_in = torch.cat([m(tensors[p + "y"], dev), m(tensors[p + "x"], dev)], dim=0)
+        self.y_bias, self.x_bias, self.conv_bias = vec("y.b"), vec("x.b"), vec("conv.b")
+        self.w_conv = _f32(tensors[p + "conv"], dev)
+        self.w_r, self.w_i = m(tensors[p + "ra"], dev), m(tensors[p + "ri"], dev)
+        self.b_r, self.b_i, self.lam = vec("ra.b"), vec("ri.b"), vec("lam")
+        self.w_o = m(tensors[p + "o"], dev)
+
+    def prefetch_first(self, ctx: StepContext, cache: Optional[CacheBinding]) -> None:
+        F.l2_prefetch(self.w_in)
+
+    def cache_need(self):
+        return StateNeed((self.floats,), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
+        state, W = ctx.states[cache.group], self.W
+        proj = linear(x, self.w_in, torch.float32)                       # y | x
+        if ctx.prefetch is not None:
+            ctx.prefetch((self.w_o,))
+        if ctx.all_decode and self.rt.act == torch.bfloat16:
+            out = F.lru_decode(proj, W, 0, self.x_bias, self.w_conv, self.conv_bias, self.y_bias, self.w_r, self.w_i,
+                               self.b_r, self.b_i, self.lam, state, 0, self.conv_off, ctx.q_start, ctx.state_slot,
+                               self.rt.act)
+        else:
+            u = F.causal_conv(proj, W, W, self.x_bias, self.w_conv, self.conv_bias, state, self.conv_off, ctx.q_start,
+                              ctx.req_of_token, ctx.state_slot)
+            a, drive = F.lru_gates(u, self.w_r, self.w_i, self.b_r, self.b_i, self.lam)
+            # the float32 path walks every portion in one piece, so that its sums run in one order
+            segments = self.rt.act == torch.bfloat16 and ctx.max_q_len >= TUNING.lru_segments_min_tokens
+            out = F.lru_scan(a, drive, proj, 0, self.y_bias, state, 0, ctx.q_start, ctx.state_slot, self.rt.act,
+                             segments, ctx.max_q_len)
+        return linear(out, self.w_o, torch.float32)
+
+
 class ResidualShortConv(Mixer):
     """``x + conv(x)``: a causal convolution over time on each channel, ``conv(x)_t = sum_j w[:, j] x_(t - taps +
     1 + j)``, zeros before a request's start, no bias and no activation.  It reads float32 rows and writes the
@@ -389,3 +617,6 @@ register_part("mixer", "gated_delta", GatedDelta)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "residual_short_conv", ResidualShortConv)
 register_part("mixer", "mamba2", Mamba2)
+register_part("mixer", "matrix_lstm", MatrixLSTM)
+register_part("mixer", "fixed_decay_attention", FixedDecayAttention)
+register_part("mixer", "gated_lru", GatedLRU)

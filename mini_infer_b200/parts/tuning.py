@@ -105,6 +105,12 @@ class Tuning:
     scan_segment_tokens: int = 128
     scan_max_segments: int = 32
 
+    # Matrix memories with one gate per head and the gated linear recurrence per channel (bfloat16 path): portions of at
+    # least so many tokens go over chunks of 64 tokens on the tensor cores, or in segments of 64 tokens side by side;
+    # shorter ones are walked token by token.
+    memory_chunks_min_tokens: int = 48
+    lru_segments_min_tokens: int = 128
+
     # Attention through a latent.  Steps of at most ``latent_small_max_tokens`` tokens run the head's key and value
     # matrices inside kernels of their own, one block per (token, head), which read the matrices once per token;
     # above, the library's batched products read them once.

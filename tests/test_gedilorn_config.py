@@ -154,9 +154,8 @@ def test_a_mixer_that_cannot_stretch_a_rotation_refuses_it():
     from mini_infer_b200.config.spec import PartSpec
     from mini_infer_b200.parts import Runtime, precision_from_name
     pos = PartSpec("rope_yarn", {"head_dim": 8, "theta": 100.0, "factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0})
-    part = part_class("mixer", "head_mix_attention")({
-        "hidden_size": 16, "num_heads": 2, "num_kv_heads": 1, "head_dim": 8, "value_dim": 8, "window": 4, "scale": 0.3,
-        "head_mix": False, "position": pos}, "m.")
+    part = part_class("mixer", "gqa_attention")({"hidden_size": 16, "num_heads": 2, "num_kv_heads": 1, "head_dim": 8,
+                                                 "position": pos}, "m.")
     t = {d.name: torch.zeros(d.shape) for d in part.tensor_decls()}
     with pytest.raises(ValueError, match="stretch"):
         part.load(t, Runtime(precision_from_name("float32"), torch.device("cpu")))
