@@ -87,9 +87,9 @@ def matrix_memory(q, k, v, i, f):
 def mlstm_mixer(h, W, p, m, eps, rnd):
     T = h.shape[0]
     H, d, e, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
-    q = (h @ W[p + "q"].T).reshape(T, H, d) * d ** -0.5
-    k = (h @ W[p + "k"].T).reshape(T, H, d)
-    v = (h @ W[p + "v"].T).reshape(T, H, e)
+    q = rnd(h @ W[p + "q"].T).reshape(T, H, d) * d ** -0.5
+    k = rnd(h @ W[p + "k"].T).reshape(T, H, d)
+    v = rnd(h @ W[p + "v"].T).reshape(T, H, e)
     i = cap * torch.tanh((h @ W[p + "i"].T + W[p + "i.b"]) / cap)
     f = log_sigmoid(cap * torch.tanh((h @ W[p + "f"].T + W[p + "f.b"]) / cap))
     o = unit_rms(matrix_memory(q, k, v, i, f), eps).reshape(T, H * e) * W[p + "norm"]
@@ -187,9 +187,9 @@ def chunk_attention(h, W, p, m, eps, rnd):
     out = torch.zeros(T, H, d, dtype=h.dtype)
     for hd in range(H):
         g = hd // (H // G)
-        out[:, hd] = sink_softmax((q[:, hd] @ k[:, g].T) * m["scale"], visible, W[p + "sink"][hd]) @ v[:, g]
+        out[:, hd] = rnd(sink_softmax((q[:, hd] @ k[:, g].T) * m["scale"], visible, W[p + "sink"][hd])) @ v[:, g]
     gate = sigmoid(h @ W[p + "g"].T)
-    return rnd(rnd(out) * gate[:, :, None]).reshape(T, H * d) @ W[p + "o"].T
+    return rnd(out * gate[:, :, None]).reshape(T, H * d) @ W[p + "o"].T
 
 
 def fixed_decay_memory(q, k, v, decay):
@@ -206,8 +206,8 @@ def fixed_decay_memory(q, k, v, decay):
 def lightning_attention(h, W, p, m, eps, rnd):
     T = h.shape[0]
     H, d, e = m["heads"], m["dim"], m["vdim"]
-    q, k = silu(h @ W[p + "q"].T).reshape(T, H, d), silu(h @ W[p + "k"].T).reshape(T, H, d)
-    v = silu(h @ W[p + "v"].T).reshape(T, H, e)
+    q, k = rnd(silu(h @ W[p + "q"].T)).reshape(T, H, d), rnd(silu(h @ W[p + "k"].T)).reshape(T, H, d)
+    v = rnd(silu(h @ W[p + "v"].T)).reshape(T, H, e)
     o = fixed_decay_memory(q, k, v, torch.tensor(m["decay"], dtype=h.dtype)).reshape(T, H * e)
     return rnd(unit_rms(o, eps) * W[p + "norm"] * sigmoid(h @ W[p + "g"].T)) @ W[p + "o"].T
 
@@ -222,7 +222,7 @@ MIXERS = {"mlstm": mlstm_mixer, "rglru": rglru_mixer, "parallel": parallel_mixer
 
 
 def feed_forward(h, W, p, rnd):
-    return rnd(torch.relu(h @ W[p + "up"].T) ** 2) @ W[p + "down"].T
+    return rnd(torch.relu(rnd(h @ W[p + "up"].T)) ** 2) @ W[p + "down"].T
 
 
 def forward(config: dict, weights: Dict[str, torch.Tensor], tokens, rnd: Optional[Callable] = None,
