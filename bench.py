@@ -1080,6 +1080,124 @@ def run_gedilorn(args):
                        _gedilorn_kernel_work, _gedilorn_twin_kernel_work, "dense_twin", graph_prompts=True)
 
 
+# --------------------------------------------------------------------------- #
+# --dedizen: the Dedizen design beside the closest built-in model (dense layers) at equal sizes
+# --------------------------------------------------------------------------- #
+DEDIZEN_SIZES = {   # width, attention heads of 128 and key/value heads; linear-attention heads, key and value size;
+                    # matrix-memory heads, key and value size; channels of the recurrence and parts; feed-forward width,
+                    # and the twin's (three matrices instead of two)
+    "0.5b": (1024, 8, 2, 8, 64, 128, 4, 128, 256, 1280, 10, 4096, 2816),
+    "2b": (2048, 16, 4, 16, 128, 128, 4, 256, 512, 2560, 10, 8192, 5632),
+    "4b": (2560, 20, 4, 20, 128, 128, 5, 256, 512, 3840, 15, 9600, 6400),
+}
+DEDIZEN_LAYERS = ("parallel", "mlstm", "rglru", "parallel", "mlstm", "rglru")
+
+
+def dedizen_config(size, window, vocab):
+    W, H, G, rh, rd, rv, mh, md, mv, C, blocks, ff, _ = DEDIZEN_SIZES[size]
+    left = {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "mask": {"size": window}, "scale": 128 ** -0.5,
+            "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": rh, "dim": rd, "vdim": rv, "decay": [1.0 - 2.0 ** (-3 - 5 * h / max(rh - 1, 1)) for h in range(rh)]}
+    mixers = {"parallel": {"left": left, "right": right},
+              "mlstm": {"heads": mh, "dim": md, "vdim": mv, "gate_cap": 15.0},
+              "rglru": {"width": C, "blocks": blocks, "conv": 4}}
+    return {"architecture": "Dedizen", "vocab": vocab, "width": W, "norm": {"eps": 1e-6},
+            "layers": [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": ff}} for t in DEDIZEN_LAYERS]}
+
+
+def dedizen_twin_config(size, window, vocab):
+    """The closest built-in model: Qwen2-MoE with every layer dense (grouped-query attention behind a window of the
+    chunks' size, SwiGLU feed-forward with as many parameters), as many layers."""
+    W, H, G = DEDIZEN_SIZES[size][:3]
+    n = len(DEDIZEN_LAYERS)
+    return dict(A27B, vocab_size=vocab, hidden_size=W, intermediate_size=DEDIZEN_SIZES[size][12], num_hidden_layers=n,
+                num_attention_heads=H, num_key_value_heads=G, head_dim=128, num_experts=4, num_experts_per_tok=2,
+                moe_intermediate_size=64, shared_expert_intermediate_size=0, mlp_only_layers=list(range(n)),
+                use_sliding_window=True, sliding_window=window, max_window_layers=0, max_position_embeddings=1 << 20)
+
+
+def _dedizen_kernel_work(cfg, T, B, ctx, decode):
+    """Algorithmic bytes and floating-point operations of the design's own kernels for one step over all layers
+    (prefill of T tokens of one request, or a decode step of B requests at context ctx)."""
+    rows, W = (B if decode else T), cfg["width"]
+    out = {}
+
+    def add(name, by, fl=0.0):
+        a = out.setdefault(name, [0.0, 0.0])
+        a[0] += by
+        a[1] += fl
+
+    def memory(H, d, e, log_gates):
+        v = H * e
+        rows_in = (2 * H * d + v) * 4
+        if decode:
+            # the state read and written, the token's row in, the finished row (or the float read-out) out
+            add("mem::memory_decode_kernel", B * (H * d * (e + (1 if log_gates else 0)) * 8 + rows_in + (v * 6 if log_gates else v * 4)),
+                B * H * d * e * 5.0)
+        else:
+            n = T // 64
+            states = n * H * d * e * 4
+            add("mem::memory_chunk_states_kernel", T * (H * d + v) * 4 + states, T * H * d * e * 2.0)
+            add("mem::memory_chunk_chain_kernel", 2 * states)
+            add("mem::memory_chunk_outputs_kernel", T * rows_in + states + T * v * 4, T * H * (2.0 * d * e + 64.0 * (d + e)))
+            if log_gates:
+                add("mem::memory_gates_kernel", T * H * (8 + 32))
+                add("mem::memory_finish_kernel", T * v * (4 + 4 + 2))
+        if not log_gates:
+            add("gated_group_rmsnorm_kernel", rows * v * (4 + 4 + 2))
+    for L in cfg["layers"]:
+        m, ff = L["mixer"], L["mlp"]["ff"]
+        if not decode:
+            add("squared_relu_bf16x8_kernel", T * ff * 4)
+        if L["type"] == "mlstm":
+            memory(m["heads"], m["dim"], m["vdim"], True)
+        elif L["type"] == "rglru":
+            C, n = m["width"], m["width"] // m["blocks"]
+            if decode:
+                add("lru::lru_decode_kernel", B * C * (8 + 2 + 8 + 8 * (m["conv"] - 1)) + 2 * C * n * 2, B * C * n * 4.0)
+            else:
+                for name in ("causal_conv_silu_kernel", "causal_conv_silu_vec4_kernel"):
+                    add(name, T * C * 8, T * C * 2.0 * m["conv"])
+                add("lru::lru_gates_tc_kernel", T * C * 12 + 2 * C * n * 2, T * C * n * 4.0)
+                add("lru::lru_segments_kernel", T * C * 8)
+                add("lru::lru_scan_kernel", T * C * (12 + 2))
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, size = a["heads"], a["kv_heads"], a["dim"], a["mask"]["size"]
+            keys = ctx % size + 1                        # of the token at position ctx
+            pairs = B * keys if decode else sum(t % size + 1 for t in range(T))
+            by = (B * keys * G * 2 * d * 2 + B * H * 2 * d * 2) if decode else T * (H + G) * 2 * d * 2
+            for name in ("attn_decode_split_kernel", "pt::attn_prefill_tc_kernel"):
+                add(name, by, pairs * H * 4.0 * d)
+            add("rope_store_vec_kernel", rows * ((H + G) * d * 4 + (H + 2 * G) * d * 2))
+            memory(r["heads"], r["dim"], r["vdim"], False)
+            add("normed_pair_add_kernel", rows * W * (8 + 8 + 2))
+    singles = sum(2 if L["type"] != "parallel" else 1 for L in cfg["layers"])
+    add("add_rmsnorm_vec_kernel", singles * rows * W * (3 * 4 + 2))
+    return out
+
+
+def _dedizen_twin_kernel_work(cfg, size, window, T, B, ctx, decode):
+    W, H, G = DEDIZEN_SIZES[size][:3]
+    rows, n, d, ff = (B if decode else T), len(DEDIZEN_LAYERS), 128, DEDIZEN_SIZES[size][12]
+    if decode:
+        keys = min(ctx, window)
+        pairs, by = B * keys, B * keys * G * 2 * d * 2 + B * H * 2 * d * 2
+        attn = "attn_decode_split_kernel"
+    else:
+        pairs, by, attn = sum(min(t + 1, window) for t in range(T)), T * (H + G) * 2 * d * 2, "pt::attn_prefill_tc_kernel"
+    return {attn: [n * by, n * pairs * H * 4.0 * d],
+            "add_rmsnorm_vec_kernel": [2 * n * rows * W * (3 * 4 + 2), 0.0],
+            "swiglu_bf16x8_kernel": [n * rows * ff * 6, 0.0],
+            "qkv_post_rows_kernel": [n * rows * (H + 2 * G) * d * 6, 0.0],
+            "embed_gather_kernel": [rows * W * 6, 0.0]}
+
+
+def run_dedizen(args):
+    return _run_design(args, "dedizen", args.dedizen, args.dedizen_chunk, dedizen_config, dedizen_twin_config,
+                       _dedizen_kernel_work, _dedizen_twin_kernel_work, "dense_twin", graph_prompts=True)
+
+
 def run_reference(args):
     """The reference arm: Deyu-Kong/mini-infer itself, unmodified, built out of tree for sm_100 by
     ``baseline/build_reference.py`` and driven by ``baseline/reference_bench.cpp`` through its stock path
@@ -1227,6 +1345,11 @@ def main():
     ap.add_argument("--gedilorn", default="", metavar="SIZES",
                     help="instead of the default workload: the Gedilorn design beside Qwen2-MoE with dense layers at "
                          "these sizes (comma-separated, of " + ", ".join(GEDILORN_SIZES) + "), see run_gedilorn")
+    ap.add_argument("--dedizen", default="", metavar="SIZES",
+                    help="instead of the default workload: the Dedizen design beside Qwen2-MoE with dense layers at "
+                         "these sizes (comma-separated, of " + ", ".join(DEDIZEN_SIZES) + "), see run_dedizen")
+    ap.add_argument("--dedizen-chunk", type=int, default=1024, help="attention chunk of the --dedizen models (and the "
+                    "twin's window)")
     ap.add_argument("--reference-timeout", type=int, default=1500, help="seconds the reference's program may take")
     ap.add_argument("--reference-prefill-batch", type=int, default=1,
                     help="prompts the reference's scheduler prefills per iteration (its cuBLAS handles, one per "
@@ -1254,6 +1377,8 @@ def main():
         return run_bogetar(args)
     if args.gedilorn:
         return run_gedilorn(args)
+    if args.dedizen:
+        return run_dedizen(args)
     return run_ours(args)
 
 
