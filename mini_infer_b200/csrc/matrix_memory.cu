@@ -82,10 +82,13 @@ __device__ __forceinline__ void log_gates(const LogGates& g, int64_t t, int h, f
 // One block per (head, request).  The gates of 256 tokens are formed side by side, one thread runs the chain of m over
 // them (an addition and a maximum per token), and the exponentials are formed side by side again.
 // gates [T][H] = (keep, write, exp(-m), f);  logs [T][H] = (i, m, m before, 0) or null.
+// SCAN: the step m -> max(f + m, i) as the pair (f, i), pairs composed by warps and then over the warps: the sums of f
+// run in another order than in the chain, which is what the chunks of long portions do with them anyway.
+template <bool SCAN>
 __global__ void __launch_bounds__(256)
 memory_gates_kernel(LogGates lg, State st, const int* __restrict__ q_start, const int* __restrict__ state_slot,
                     float4* __restrict__ gates, float4* __restrict__ logs, int H) {
-    __shared__ float si[256], sf[256], sm[257];
+    __shared__ float si[256], sf[256], sm[257], wf[8], wi[8];
     wait_for_earlier_kernels();
     const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
     const int q0 = q_start[b], n = q_start[b + 1] - q0;
@@ -93,17 +96,44 @@ memory_gates_kernel(LogGates lg, State st, const int* __restrict__ q_start, cons
     if (tid == 0) sm[0] = *m_state;
     for (int c0 = 0; c0 < n; c0 += 256) {
         const int nc = min(256, n - c0);
-        float li = 0.f, lf = 0.f;
+        float li = -INFINITY, lf = 0.f;                  // (beyond the portion: a step that changes nothing)
         if (tid < nc) log_gates(lg, q0 + c0 + tid, h, li, lf);
+        if (SCAN) {
+            const int lane = tid & 31, warp = tid >> 5;
+            float cf = lf, ci = li;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float pf = __shfl_up_sync(0xffffffffu, cf, o), pi = __shfl_up_sync(0xffffffffu, ci, o);
+                if (lane >= o) { ci = fmaxf(cf + pi, ci); cf += pf; }
+            }
+            if (lane == 31) { wf[warp] = cf; wi[warp] = ci; }
+            __syncthreads();
+            float m = sm[0];
+            for (int w = 0; w < warp; ++w) m = fmaxf(wf[w] + m, wi[w]);
+            const float mine = fmaxf(cf + m, ci);
+            __syncthreads();                             // sm[0] has been read
+            sm[tid + 1] = mine;
+            __syncthreads();
+        } else {
         si[tid] = li;
         sf[tid] = lf;
         __syncthreads();
         if (tid == 0) {
+            // eight tokens' gates are asked for before the first of them: the chain is an addition and a maximum
             float m = sm[0];
-#pragma unroll 8
-            for (int t = 0; t < nc; ++t) { m = fmaxf(sf[t] + m, si[t]); sm[t + 1] = m; }
+            for (int t = 0; t < 256; t += 8) {
+                float f8[8], i8[8];
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { f8[k] = sf[t + k]; i8[k] = si[t + k]; }
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { m = fmaxf(f8[k] + m, i8[k]); f8[k] = m; }
+#pragma unroll
+                for (int k = 0; k < 8; ++k) sm[t + k + 1] = f8[k];
+                if (t + 8 >= nc) break;
+            }
         }
         __syncthreads();
+        }
         if (tid < nc) {
             const float before = sm[tid], m = sm[tid + 1];
             const int64_t at = (int64_t)(q0 + c0 + tid) * H + h;
@@ -261,25 +291,45 @@ memory_walk_kernel(Rows in, State st, const float4* __restrict__ gates, const fl
         }
 }
 
-// y = rmsnorm_head(o / (max(|n . q|, exp(-m)) + 1e-6)) * w * logistic(gate): a block per (token, head); w has H * dv
-// entries, den is n . q and gates[..].z is exp(-m).
-template <typename AT>
+// y = rmsnorm_group(o / (max(|n . q|, exp(-m)) + 1e-6)) * w * logistic(gate): a block per (token, group of gs columns).
+// With log gates a group is a head (gs = dv; den is n . q and gates[..].z is exp(-m)); den null: nothing is divided and a
+// group is whatever the caller says.  w has an entry per column.
+template <typename AT, typename GT>
 __global__ void __launch_bounds__(128)
 memory_finish_kernel(const float* __restrict__ o, const float* __restrict__ den, const float4* __restrict__ gates,
-                     const float* __restrict__ gate, int64_t ld_gate, const float* __restrict__ w, AT* __restrict__ out,
-                     int H, int dv, float eps) {
+                     const GT* __restrict__ gate, int64_t ld_gate, const float* __restrict__ w, AT* __restrict__ out,
+                     int n, int gs, float eps, int vec) {
     __shared__ float scratch[32];
     wait_for_earlier_kernels();
     const int64_t t = blockIdx.x;
-    const int h = blockIdx.y;
-    const float* row = o + (t * H + h) * dv;
-    const float inv = 1.0f / (fmaxf(fabsf(den[t * H + h]), gates[t * H + h].z) + 1e-6f);
+    const int h = blockIdx.y, H = n / gs;
+    const float* row = o + t * n + (int64_t)h * gs;
+    const float* wr = w + h * gs;
+    const GT* gr = gate + t * ld_gate + h * gs;
+    AT* orow = out + t * n + (int64_t)h * gs;
+    const float inv = den ? 1.0f / (fmaxf(fabsf(den[t * H + h]), gates[t * H + h].z) + 1e-6f) : 1.0f;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < dv; c += blockDim.x) { const float v = row[c] * inv; ss += v * v; }
+    if (vec) {
+        for (int c = 4 * threadIdx.x; c < gs; c += 4 * blockDim.x) {
+            const float4 v = *reinterpret_cast<const float4*>(row + c);
+            const float a = v.x * inv, b = v.y * inv, d = v.z * inv, e = v.w * inv;
+            ss += (a * a + b * b) + (d * d + e * e);
+        }
+    } else {
+        for (int c = threadIdx.x; c < gs; c += blockDim.x) { const float v = row[c] * inv; ss += v * v; }
+    }
     ss = block_sum(ss, scratch);
-    const float rr = inv / sqrtf(ss / (float)dv + eps);
-    for (int c = threadIdx.x; c < dv; c += blockDim.x)
-        out[(t * H + h) * dv + c] = from_float<AT>(row[c] * rr * w[h * dv + c] * sigmoid_f(gate[t * ld_gate + h * dv + c]));
+    const float rr = inv / sqrtf(ss / (float)gs + eps);
+    if (vec) {
+        for (int c = 4 * threadIdx.x; c < gs; c += 4 * blockDim.x) {
+            const float4 v = *reinterpret_cast<const float4*>(row + c), u = *reinterpret_cast<const float4*>(wr + c);
+            store4(orow + c, make_float4(v.x * rr * u.x * sigmoid_f(to_float(gr[c])), v.y * rr * u.y * sigmoid_f(to_float(gr[c + 1])),
+                                         v.z * rr * u.z * sigmoid_f(to_float(gr[c + 2])), v.w * rr * u.w * sigmoid_f(to_float(gr[c + 3]))));
+        }
+    } else {
+        for (int c = threadIdx.x; c < gs; c += blockDim.x)
+            orow[c] = from_float<AT>(row[c] * rr * wr[c] * sigmoid_f(to_float(gr[c])));
+    }
 }
 
 }  // namespace mem
@@ -429,7 +479,7 @@ memory_decode_kernel(Rows in, LogGates lg, State st, const float* __restrict__ d
 //   outputs   the two sums above
 //
 // The projections q, k and v are the bfloat16 operands.  What the recurrence makes is float: a float factor of a
-// product on the tensor cores (a weighted key, a weighted score, the state) goes in as a sum of two bfloat16 numbers,
+// product on the tensor cores (a weighted value, a weighted score, the state) goes in as a sum of two bfloat16 numbers,
 // high part and remainder, so that it loses no more than 2^-17 of itself, and all sums are float.
 // A request's chunks count from the portion's start; chunk c of request b has the index q_start[b] / 64 + b + c.
 // ---------------------------------------------------------------------------
@@ -482,24 +532,60 @@ __device__ __forceinline__ void chunk_log_decays(const float4* gates, int64_t t0
     }
 }
 
-// four neighbouring floats of a row (zeros beyond its end)
-__device__ __forceinline__ float4 load4(const float* p, int n, bool vec) {
-    if (vec && n >= 4) return *reinterpret_cast<const float4*>(p);
-    return make_float4(n > 0 ? p[0] : 0.f, n > 1 ? p[1] : 0.f, n > 2 ? p[2] : 0.f, n > 3 ? p[3] : 0.f);
+// Projection rows in bfloat16, and what is done to them.
+struct RowsB {
+    const __nv_bfloat16* p;
+    int64_t ld;
+    int q, k, v;
+    int act;
+    float q_scale;
+    int vec;                // rows, columns and heads on 16-byte boundaries
+};
+
+__device__ __forceinline__ void copy_async_16b(void* smem_dst, const void* src) {
+    const uint32_t dst = static_cast<uint32_t>(__cvta_generic_to_shared(smem_dst));
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src));
 }
-__device__ __forceinline__ float4 act4(float4 v, int act) {
-    if (act) { v.x = silu_f(v.x); v.y = silu_f(v.y); v.z = silu_f(v.z); v.w = silu_f(v.w); }
-    return v;
+__device__ __forceinline__ void copy_async_wait_all() { asm volatile("cp.async.wait_all;\n" ::: "memory"); }
+
+// eight neighbouring numbers of a row through the activation (zeros from column n on)
+__device__ __forceinline__ uint4 load8(const __nv_bfloat16* p, int n, int act, bool vec) {
+    uint4 r = make_uint4(0u, 0u, 0u, 0u);
+    __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&r);
+    if (vec && n >= 8) r = *reinterpret_cast<const uint4*>(p);
+    else {
+#pragma unroll
+        for (int x = 0; x < 8; ++x) if (x < n) e[x] = p[x];
+    }
+    if (act) {
+#pragma unroll
+        for (int x = 0; x < 8; ++x) { const float f = __bfloat162float(e[x]); e[x] = __float2bfloat16_rn(__fdividef(f, 1.0f + __expf(-f))); }
+    }
+    return r;
 }
 
-// U [chunk][H][d][dv], Un [chunk][H][d] (log gates), keepc [chunk][H].  Block = 4 warps: a value tile of 64 columns of
-// one (chunk, head); dp = d rounded up to 16.
+// 64 rows of `width` columns (padded to wp, a multiple of 8) into shared memory; rows from nt on are zeros.  Without an
+// activation, copies that nothing has to touch are left in flight (copy_async_wait_all before the barrier).
+__device__ __forceinline__ void fill_rows(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int64_t ld, int width, int wp,
+                                          int nt, int act, bool vec) {
+    const int w8 = wp / 8;
+    for (int idx = threadIdx.x; idx < kC * w8; idx += blockDim.x) {
+        const int j = idx / w8, i = 8 * (idx - j * w8);
+        __nv_bfloat16* d = dst + j * pitch + i;
+        if (j < nt && vec && !act && i + 8 <= width) copy_async_16b(d, src + j * ld + i);
+        else *reinterpret_cast<uint4*>(d) = j < nt ? load8(src + j * ld + i, width - i, act, vec) : make_uint4(0u, 0u, 0u, 0u);
+    }
+}
+
+// U [chunk][H][d][dvp] (dvp: dv rounded up to 8, zeros beyond dv), Un [chunk][H][d] (log gates), keepc [chunk][H].  A block
+// of 4 warps takes a value tile of 64 columns of one (chunk, head).  The weights go into the values, w_j v_j, as high part
+// and remainder: a tile's values are its own, while its keys serve every tile of the head.  dp = d rounded up to 16.
 template <bool LOG>
 __global__ void __launch_bounds__(128)
-memory_chunk_states_kernel(Rows in, const float4* __restrict__ gates, const float4* __restrict__ logs,
+memory_chunk_states_kernel(RowsB in, const float4* __restrict__ gates, const float4* __restrict__ logs,
                            const float* __restrict__ decay, const int* __restrict__ q_start, float* __restrict__ U,
-                           float* __restrict__ Un, float* __restrict__ keepc, int H, int d, int dv, int dp, int tiles,
-                           int vec) {
+                           float* __restrict__ Un, float* __restrict__ keepc, int H, int d, int dv, int dvp, int dp,
+                           int tiles) {
     extern __shared__ __align__(16) unsigned char raw[];
     __shared__ float Fh[kC], Fl[kC], wj[kC];
     wait_for_earlier_kernels();
@@ -510,9 +596,11 @@ memory_chunk_states_kernel(Rows in, const float4* __restrict__ gates, const floa
     const int64_t t0 = q0 + c * kC, at = (int64_t)(q0 / kC + b + c) * H + h;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int kp = dp + 8;
-    __nv_bfloat16* Kh = reinterpret_cast<__nv_bfloat16*>(raw);      // [64][kp] weighted keys, high parts
-    __nv_bfloat16* Kl = Kh + kC * kp;                               // remainders
-    __nv_bfloat16* Vs = Kl + kC * kp;                               // [64][kVP]
+    __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(raw);      // [64][kp] keys
+    __nv_bfloat16* Vh = Ks + kC * kp;                               // [64][kVP] weighted values, high parts
+    __nv_bfloat16* Vl = Vh + kC * kVP;                              // remainders
+    const int v_lo = tile * kT, nv = min(kT, dv - v_lo);
+    fill_rows(Ks, kp, in.p + t0 * in.ld + in.k + h * d, in.ld, d, dp, nt, in.act, in.vec);
     if (LOG) {
         chunk_log_decays(gates, t0, nt, H, h, Fh, Fl);
         __syncthreads();
@@ -528,141 +616,168 @@ memory_chunk_states_kernel(Rows in, const float4* __restrict__ gates, const floa
         if (tid == 0 && tile == 0) keepc[at] = expf((float)nt * ld);
     }
     __syncthreads();
-    const int d4 = dp / 4;
-    for (int idx = tid; idx < kC * d4; idx += 128) {
-        const int j = idx / d4, i = 4 * (idx - j * d4);
-        float4 k = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (j < nt) k = act4(load4(in.p + (t0 + j) * in.ld + in.k + h * d + i, d - i, vec), in.act);
+    for (int idx = tid; idx < kC * (kT / 8); idx += 128) {
+        const int j = idx / (kT / 8), i = 8 * (idx % (kT / 8));
+        uint4 v = make_uint4(0u, 0u, 0u, 0u), lo8;
+        if (j < nt) v = load8(in.p + (t0 + j) * in.ld + in.v + (int64_t)h * dv + v_lo + i, nv - i, in.act, in.vec);
+        __nv_bfloat16* hi = reinterpret_cast<__nv_bfloat16*>(&v);
+        __nv_bfloat16* lo = reinterpret_cast<__nv_bfloat16*>(&lo8);
         const float w = wj[j];
-        const float kk[4] = {k.x, k.y, k.z, k.w};
-        __nv_bfloat16 hi[4], lo[4];
 #pragma unroll
-        for (int x = 0; x < 4; ++x) split2(w * __bfloat162float(__float2bfloat16_rn(i + x < d ? kk[x] : 0.f)), hi[x], lo[x]);
-        *reinterpret_cast<uint2*>(Kh + j * kp + i) = make_uint2(pack2(hi[0], hi[1]), pack2(hi[2], hi[3]));
-        *reinterpret_cast<uint2*>(Kl + j * kp + i) = make_uint2(pack2(lo[0], lo[1]), pack2(lo[2], lo[3]));
+        for (int x = 0; x < 8; ++x) { const float f = w * __bfloat162float(hi[x]); split2(f, hi[x], lo[x]); }
+        *reinterpret_cast<uint4*>(Vh + j * kVP + i) = v;
+        *reinterpret_cast<uint4*>(Vl + j * kVP + i) = lo8;
     }
-    const int v_lo = tile * kT, nv = min(kT, dv - v_lo);
-    for (int idx = tid; idx < kC * (kT / 4); idx += 128) {
-        const int j = idx / (kT / 4), i = 4 * (idx % (kT / 4));
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (j < nt) v = act4(load4(in.p + (t0 + j) * in.ld + in.v + (int64_t)h * dv + v_lo + i, nv - i, vec), in.act);
-        store4(Vs + j * kVP + i, v);
-    }
+    copy_async_wait_all();
     __syncthreads();
-    float* Ub = U + at * d * dv;
+    float* Ub = U + at * d * dvp + v_lo;
+    const int nvp = min(kT, dvp - v_lo);
     for (int mt = warp; mt < dp / 16; mt += 4) {
         float acc[8][4];
 #pragma unroll
         for (int x = 0; x < 8; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
 #pragma unroll
         for (int kk = 0; kk < kC / 16; ++kk) {
-            // A[i][j] = weighted k_j[i]: the keys lie token by token, so the fragments are fetched transposed
-            const int jrow = kk * 16 + (lane >> 4) * 8 + (lane & 7), icol = mt * 16 + ((lane >> 3) & 1) * 8;
-            uint32_t ah[4], al[4];
-            ldmatrix_x4_trans(ah, Kh + jrow * kp + icol);
-            ldmatrix_x4_trans(al, Kl + jrow * kp + icol);
+            // A[i][j] = k_j[i]: the keys lie token by token, so the fragments are fetched transposed
+            uint32_t a[4];
+            ldmatrix_x4_trans(a, Ks + (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * kp + mt * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
-            for (int x = 0; x < 8; ++x) {
-                uint32_t b0, b1;
-                ldmatrix_x2_trans(b0, b1, Vs + (kk * 16 + (lane & 15)) * kVP + x * 8);
-                mma_bf16_16816(acc[x], ah[0], ah[1], ah[2], ah[3], b0, b1);
-                mma_bf16_16816(acc[x], al[0], al[1], al[2], al[3], b0, b1);
+            for (int x = 0; x < 8; x += 2) {
+                uint32_t bh[4], bl[4];                    // two neighbouring tiles of 8 columns
+                const int off = (kk * 16 + (lane & 15)) * kVP + (x + (lane >> 4)) * 8;
+                ldmatrix_x4_trans(bh, Vh + off);
+                ldmatrix_x4_trans(bl, Vl + off);
+                mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], bh[0], bh[1]);
+                mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], bl[0], bl[1]);
+                mma_bf16_16816(acc[x + 1], a[0], a[1], a[2], a[3], bh[2], bh[3]);
+                mma_bf16_16816(acc[x + 1], a[0], a[1], a[2], a[3], bl[2], bl[3]);
             }
         }
         const int r0 = mt * 16 + (lane >> 2), c2 = (lane & 3) * 2;
 #pragma unroll
-        for (int x = 0; x < 8; ++x)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int i = r0 + (e >> 1) * 8, col = x * 8 + c2 + (e & 1);
-                if (i < d && col < nv) Ub[(int64_t)i * dv + v_lo + col] = acc[x][e];
+        for (int x = 0; x < 8; ++x) {
+            const int col = x * 8 + c2;
+            if (col < nvp) {
+                if (r0 < d) *reinterpret_cast<float2*>(Ub + (int64_t)r0 * dvp + col) = make_float2(acc[x][0], acc[x][1]);
+                if (r0 + 8 < d) *reinterpret_cast<float2*>(Ub + (int64_t)(r0 + 8) * dvp + col) = make_float2(acc[x][2], acc[x][3]);
             }
+        }
     }
     if (LOG && tile == 0)
         for (int i = tid; i < d; i += 128) {
             float s = 0.f;
-            for (int j = 0; j < nt; ++j) s += __bfloat162float(Kh[j * kp + i]) + __bfloat162float(Kl[j * kp + i]);
+            for (int j = 0; j < nt; ++j) s += wj[j] * __bfloat162float(Ks[j * kp + i]);
             Un[at * d + i] = s;
         }
 }
 
-// S_start[0] = the request's state, S_start[c + 1] = keepc[c] S_start[c] + U[c]; S_start[c] takes the place of U[c] once
-// that has been read, and what follows the last chunk is the request's new state.  `size` elements per head, VEC a thread.
-template <int VEC>
+// S_start[0] = the request's state, S_start[c + 1] = keepc[c] S_start[c] + U[c], a thread per eight columns of a row of S;
+// what follows the last chunk is the request's new state.  S_start[c] takes the place of U[c] once that has been read, as
+// eight high parts and eight remainders in bfloat16: what the outputs' products take.
 __global__ void __launch_bounds__(256)
 memory_chunk_chain_kernel(float* __restrict__ U, const float* __restrict__ keepc, float* __restrict__ state,
                           int64_t state_stride, int64_t off, const int* __restrict__ q_start,
-                          const int* __restrict__ state_slot, int H, int size) {
+                          const int* __restrict__ state_slot, int H, int d, int dv, int dvp) {
     wait_for_earlier_kernels();
     const int b = blockIdx.z, h = blockIdx.y;
-    const int e = VEC * (blockIdx.x * blockDim.x + threadIdx.x);
+    const int e = blockIdx.x * blockDim.x + threadIdx.x, groups = dvp / 8;
     const int q0 = q_start[b], n = q_start[b + 1] - q0;
-    if (e >= size || n <= 0) return;
+    if (e >= d * groups || n <= 0) return;
+    const int i = e / groups, c8 = 8 * (e - i * groups);
     const int chunks = (n + kC - 1) / kC;
-    const int64_t first = (int64_t)(q0 / kC + b) * H + h;
-    float* S = state + (int64_t)state_slot[b] * state_stride + off + (int64_t)h * size + e;
-    float cur[VEC];
+    const int64_t first = (int64_t)(q0 / kC + b) * H + h, size = (int64_t)d * dvp;
+    float* S = state + (int64_t)state_slot[b] * state_stride + off + (int64_t)h * d * dv + (int64_t)i * dv + c8;
+    float cur[8];
 #pragma unroll
-    for (int x = 0; x < VEC; ++x) cur[x] = S[x];
-    constexpr int AHEAD = 4;
+    for (int x = 0; x < 8; ++x) cur[x] = c8 + x < dv ? S[x] : 0.f;
+    float* base = U + first * size + (int64_t)i * dvp + c8;
+    const int64_t step = H * size;
+    constexpr int AHEAD = 2;
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float u[AHEAD][VEC], keep[AHEAD];
+        float4 u[AHEAD][2];
+        float keep[AHEAD];
 #pragma unroll
-        for (int a = 0; a < AHEAD; ++a) {
+        for (int a = 0; a < AHEAD; ++a)
             if (c0 + a < chunks) {
-                const float* p = U + (first + (int64_t)(c0 + a) * H) * size + e;
-                if (VEC == 4) {
-                    const float4 f = *reinterpret_cast<const float4*>(p);
-                    u[a][0] = f.x; u[a][1 % VEC] = f.y; u[a][2 % VEC] = f.z; u[a][3 % VEC] = f.w;
-                } else {
-                    u[a][0] = *p;
-                }
+                const float4* p = reinterpret_cast<const float4*>(base + (c0 + a) * step);
+                u[a][0] = p[0];
+                u[a][1] = p[1];
                 keep[a] = keepc[first + (int64_t)(c0 + a) * H];
             }
-        }
 #pragma unroll
-        for (int a = 0; a < AHEAD; ++a) {
+        for (int a = 0; a < AHEAD; ++a)
             if (c0 + a < chunks) {
-                float* p = U + (first + (int64_t)(c0 + a) * H) * size + e;
-                if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(cur[0], cur[1 % VEC], cur[2 % VEC], cur[3 % VEC]);
-                else *p = cur[0];
+                uint4 out[2];
+                __nv_bfloat16* hl = reinterpret_cast<__nv_bfloat16*>(out);
 #pragma unroll
-                for (int x = 0; x < VEC; ++x) cur[x] = keep[a] * cur[x] + u[a][x];
+                for (int x = 0; x < 8; ++x) split2(cur[x], hl[x], hl[8 + x]);
+                uint4* p = reinterpret_cast<uint4*>(base + (c0 + a) * step);
+                p[0] = out[0];
+                p[1] = out[1];
+                const float* uu = reinterpret_cast<const float*>(u[a]);
+#pragma unroll
+                for (int x = 0; x < 8; ++x) cur[x] = keep[a] * cur[x] + uu[x];
             }
-        }
     }
 #pragma unroll
-    for (int x = 0; x < VEC; ++x) S[x] = cur[x];
+    for (int x = 0; x < 8; ++x) if (c8 + x < dv) S[x] = cur[x];
 }
 
-}  // namespace mem
-}  // namespace mi
+// the same for n, which stays float
+__global__ void __launch_bounds__(256)
+memory_chunk_norm_chain_kernel(float* __restrict__ Un, const float* __restrict__ keepc, float* __restrict__ state,
+                               int64_t state_stride, int64_t off, const int* __restrict__ q_start,
+                               const int* __restrict__ state_slot, int H, int d) {
+    wait_for_earlier_kernels();
+    const int b = blockIdx.z, h = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
+    const int q0 = q_start[b], n = q_start[b + 1] - q0;
+    if (i >= d || n <= 0) return;
+    const int chunks = (n + kC - 1) / kC;
+    const int64_t first = (int64_t)(q0 / kC + b) * H + h;
+    float* S = state + (int64_t)state_slot[b] * state_stride + off + (int64_t)h * d + i;
+    float cur = *S;
+    for (int c0 = 0; c0 < chunks; c0 += 4) {
+        float u[4], keep[4];
+#pragma unroll
+        for (int a = 0; a < 4; ++a) {
+            const int64_t at = first + (int64_t)min(c0 + a, chunks - 1) * H;
+            u[a] = Un[at * d + i];
+            keep[a] = keepc[at];
+        }
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+            if (c0 + a < chunks) { Un[(first + (int64_t)(c0 + a) * H) * d + i] = cur; cur = keep[a] * cur + u[a]; }
+    }
+    *S = cur;
+}
 
-namespace mi {
-namespace mem {
-
-// Read-outs of a chunk: warp w owns the tokens 16 w .. 16 w + 15 of it and a value tile of 64 columns.
+// Read-outs of a chunk.  Block = 8 warps: warp w owns the tokens 16 (w % 4) .. + 15 of the chunk and half of a value tile of
+// 64 columns; the block walks over `per` tiles of its head.  The weighted scores are formed once, as high part and
+// remainder in registers; a tile then costs its start state (which takes the place of the keys in shared memory) and its
+// values.
 template <bool LOG>
-__global__ void __launch_bounds__(128)
-memory_chunk_outputs_kernel(Rows in, const float4* __restrict__ gates, const float4* __restrict__ logs,
+__global__ void __launch_bounds__(256)
+memory_chunk_outputs_kernel(RowsB in, const float4* __restrict__ gates, const float4* __restrict__ logs,
                             const float* __restrict__ decay, const int* __restrict__ q_start,
                             const float* __restrict__ S0, const float* __restrict__ N0, float* __restrict__ out,
-                            float* __restrict__ den, int H, int d, int dv, int dp, int tiles, int vec, int vec_s) {
+                            float* __restrict__ den, int H, int d, int dv, int dvp, int dp, int tiles, int per, int groups) {
     extern __shared__ __align__(16) unsigned char raw[];
     __shared__ float Fh[kC], Fl[kC], ij[kC], mj[kC], inter[kC], pw[kC + 1];
     wait_for_earlier_kernels();
-    const int b = blockIdx.z, h = blockIdx.y / tiles, tile = blockIdx.y % tiles, c = blockIdx.x;
+    const int b = blockIdx.z, h = blockIdx.y / groups, group = blockIdx.y % groups, c = blockIdx.x;
     const int q0 = q_start[b], n = q_start[b + 1] - q0;
     if (c * kC >= n) return;
     const int nt = min(kC, n - c * kC);
     const int64_t t0 = q0 + c * kC, at = (int64_t)(q0 / kC + b + c) * H + h;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = warp >> 2;
     const int kp = dp + 8;
+    constexpr int SPB = kT * 4 + 16;                                // bytes of a row of the start state's tile
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(raw);      // [64][kp]
-    __nv_bfloat16* Ks = Qs + kC * kp;                               // [64][kp]
-    __nv_bfloat16* Vs = Ks + kC * kp;                               // [64][kVP]
-    __nv_bfloat16* Sh = Vs + kC * kVP;                              // [dp][kVP] start state, high parts
-    __nv_bfloat16* Sl = Sh + dp * kVP;                              // remainders
+    __nv_bfloat16* Vs = Qs + kC * kp;                               // [64][kVP]
+    __nv_bfloat16* Ks = Vs + kC * kVP;                              // [64][kp], then [dp] rows of the start state
+    unsigned char* Ss = reinterpret_cast<unsigned char*>(Ks);
+    fill_rows(Qs, kp, in.p + t0 * in.ld + in.q + h * d, in.ld, d, dp, nt, in.act, in.vec);
+    fill_rows(Ks, kp, in.p + t0 * in.ld + in.k + h * d, in.ld, d, dp, nt, in.act, in.vec);
     if (LOG) {
         chunk_log_decays(gates, t0, nt, H, h, Fh, Fl);
         __syncthreads();
@@ -675,119 +790,129 @@ memory_chunk_outputs_kernel(Rows in, const float4* __restrict__ gates, const flo
     } else if (tid <= kC) {
         pw[tid] = expf((float)tid * fmaxf(logf(decay[h]), -1e30f));
     }
-    const int d4 = dp / 4;
-    for (int idx = tid; idx < kC * d4; idx += 128) {
-        const int j = idx / d4, i = 4 * (idx - j * d4);
-        float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
-        if (j < nt) {
-            const float* row = in.p + (t0 + j) * in.ld + h * d + i;
-            q = act4(load4(row + in.q, d - i, vec), in.act);
-            k = act4(load4(row + in.k, d - i, vec), in.act);
-        }
-        store4(Qs + j * kp + i, q);
-        store4(Ks + j * kp + i, k);
-    }
-    const int v_lo = tile * kT, nv = min(kT, dv - v_lo);
-    for (int idx = tid; idx < kC * (kT / 4); idx += 128) {
-        const int j = idx / (kT / 4), i = 4 * (idx % (kT / 4));
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (j < nt) v = act4(load4(in.p + (t0 + j) * in.ld + in.v + (int64_t)h * dv + v_lo + i, nv - i, vec), in.act);
-        store4(Vs + j * kVP + i, v);
-    }
-    const float* Sb = S0 + at * d * dv + v_lo;
-    for (int idx = tid; idx < dp * (kT / 4); idx += 128) {
-        const int i = idx / (kT / 4), col = 4 * (idx % (kT / 4));
-        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i < d) s = load4(Sb + (int64_t)i * dv + col, nv - col, vec_s);
-        __nv_bfloat16 hi[4], lo[4];
-        split2(s.x, hi[0], lo[0]); split2(s.y, hi[1], lo[1]); split2(s.z, hi[2], lo[2]); split2(s.w, hi[3], lo[3]);
-        *reinterpret_cast<uint2*>(Sh + i * kVP + col) = make_uint2(pack2(hi[0], hi[1]), pack2(hi[2], hi[3]));
-        *reinterpret_cast<uint2*>(Sl + i * kVP + col) = make_uint2(pack2(lo[0], lo[1]), pack2(lo[2], lo[3]));
-    }
+    copy_async_wait_all();
     __syncthreads();
     const int r0 = lane >> 2, c2 = (lane & 3) * 2;
-    const int ta = warp * 16 + r0, tb = ta + 8;             // this thread's two tokens
-    float acc[8][4], sc[8][4];
+    const int ta = wr * 16 + r0, tb = ta + 8;               // this thread's two tokens
+    uint32_t wh[4][4], wl[4][4];                            // weighted scores as fragments, 16 keys each
+    const float ia = (LOG ? inter[ta] : pw[ta + 1]) * in.q_scale, ib = (LOG ? inter[tb] : pw[tb + 1]) * in.q_scale;
+    {
+        float sc[8][4];
 #pragma unroll
-    for (int x = 0; x < 8; ++x)
+        for (int x = 0; x < 8; ++x) sc[x][0] = sc[x][1] = sc[x][2] = sc[x][3] = 0.f;
+        for (int ks = 0; ks < dp; ks += 16) {
+            uint32_t a[4];
+            ldmatrix_x4(a, Qs + (wr * 16 + (lane & 15)) * kp + ks + (lane >> 4) * 8);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[x][e] = sc[x][e] = 0.f;
-    // q . k of the keys up to this warp's last token, and S_start^T q
-    const int xmax = 2 * warp + 2;                          // key tiles of 8 that this warp's tokens can see
-    for (int ks = 0; ks < dp; ks += 16) {
-        uint32_t a[4];
-        ldmatrix_x4(a, Qs + (warp * 16 + (lane & 15)) * kp + ks + (lane >> 4) * 8);
+            for (int x = 0; x < 8; x += 2) {
+                if (x < 2 * wr + 2) {                       // keys up to this warp's last token
+                    uint32_t k4[4];                         // (keys 8x .. + 7, + 8 .. + 15) x (columns ks .. + 7, + 8 .. + 15)
+                    ldmatrix_x4(k4, Ks + (x * 8 + (lane >> 4) * 8 + (lane & 7)) * kp + ks + ((lane >> 3) & 1) * 8);
+                    mma_bf16_16816(sc[x], a[0], a[1], a[2], a[3], k4[0], k4[1]);
+                    mma_bf16_16816(sc[x + 1], a[0], a[1], a[2], a[3], k4[2], k4[3]);
+                }
+            }
+        }
+        float suma = 0.f, sumb = 0.f;
 #pragma unroll
         for (int x = 0; x < 8; ++x) {
-            if (x < xmax) {
-                const __nv_bfloat16* kr = Ks + (x * 8 + r0) * kp + ks + c2;
-                mma_bf16_16816(sc[x], a[0], a[1], a[2], a[3], *reinterpret_cast<const uint32_t*>(kr),
-                               *reinterpret_cast<const uint32_t*>(kr + 8));
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int j = x * 8 + c2 + (e & 1), t = e < 2 ? ta : tb;
+                float wgt = 0.f;
+                if (j <= t) wgt = LOG ? expf((Fh[t] - Fh[j]) + (Fl[t] - Fl[j]) + (ij[j] - mj[t])) : pw[t - j];
+                sc[x][e] *= wgt * in.q_scale;
             }
-            uint32_t b0, b1;
-            ldmatrix_x2_trans(b0, b1, Sh + (ks + (lane & 15)) * kVP + x * 8);
-            mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], b0, b1);
-            ldmatrix_x2_trans(b0, b1, Sl + (ks + (lane & 15)) * kVP + x * 8);
-            mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], b0, b1);
+            suma += sc[x][0] + sc[x][1];
+            sumb += sc[x][2] + sc[x][3];
         }
-    }
-    const float ia = (LOG ? inter[ta] : pw[ta + 1]) * in.q_scale, ib = (LOG ? inter[tb] : pw[tb + 1]) * in.q_scale;
-    float suma = 0.f, sumb = 0.f;
 #pragma unroll
-    for (int x = 0; x < 8; ++x) {
-        acc[x][0] *= ia; acc[x][1] *= ia; acc[x][2] *= ib; acc[x][3] *= ib;
+        for (int kk = 0; kk < 4; ++kk)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int j = x * 8 + c2 + (e & 1), t = e < 2 ? ta : tb;
-            float wgt = 0.f;
-            if (j <= t) wgt = LOG ? expf((Fh[t] - Fh[j]) + (Fl[t] - Fl[j]) + (ij[j] - mj[t])) : pw[t - j];
-            sc[x][e] *= wgt * in.q_scale;
-        }
-        suma += sc[x][0] + sc[x][1];
-        sumb += sc[x][2] + sc[x][3];
-    }
-#pragma unroll
-    for (int kk = 0; kk < kC / 16; ++kk) {
-        if (kk <= warp) {
-            __nv_bfloat16 hi[8], lo[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) split2(sc[2 * kk + (e >> 2)][e & 3], hi[e], lo[e]);
-            // fragments: rows ta (elements 0, 1) and tb (2, 3), keys 2 c2 .. and the same eight keys further
-            const uint32_t h0 = pack2(hi[0], hi[1]), h1 = pack2(hi[2], hi[3]), h2 = pack2(hi[4], hi[5]), h3 = pack2(hi[6], hi[7]);
-            const uint32_t l0 = pack2(lo[0], lo[1]), l1 = pack2(lo[2], lo[3]), l2 = pack2(lo[4], lo[5]), l3 = pack2(lo[6], lo[7]);
-#pragma unroll
-            for (int x = 0; x < 8; ++x) {
-                uint32_t b0, b1;
-                ldmatrix_x2_trans(b0, b1, Vs + (kk * 16 + (lane & 15)) * kVP + x * 8);
-                mma_bf16_16816(acc[x], h0, h1, h2, h3, b0, b1);
-                mma_bf16_16816(acc[x], l0, l1, l2, l3, b0, b1);
+            for (int f = 0; f < 4; ++f) {
+                // fragment f: rows ta (0, 2) and tb (1, 3), keys c2, c2 + 1 of the first (0, 1) and second eight (2, 3)
+                __nv_bfloat16 h0, l0, h1, l1;
+                split2(sc[2 * kk + (f >> 1)][2 * (f & 1)], h0, l0);
+                split2(sc[2 * kk + (f >> 1)][2 * (f & 1) + 1], h1, l1);
+                wh[kk][f] = pack2(h0, h1);
+                wl[kk][f] = pack2(l0, l1);
+            }
+        if (LOG && group == 0 && wc == 0) {
+            // n . q: the weights' sum and what the start of the chunk brought
+            suma += __shfl_xor_sync(0xffffffffu, suma, 1); suma += __shfl_xor_sync(0xffffffffu, suma, 2);
+            sumb += __shfl_xor_sync(0xffffffffu, sumb, 1); sumb += __shfl_xor_sync(0xffffffffu, sumb, 2);
+            const float* nb = N0 + at * d;
+            float da = 0.f, db = 0.f;
+            for (int i = lane & 3; i < d; i += 4) {
+                const float x = nb[i];
+                da += x * __bfloat162float(Qs[ta * kp + i]);
+                db += x * __bfloat162float(Qs[tb * kp + i]);
+            }
+            da += __shfl_xor_sync(0xffffffffu, da, 1); da += __shfl_xor_sync(0xffffffffu, da, 2);
+            db += __shfl_xor_sync(0xffffffffu, db, 1); db += __shfl_xor_sync(0xffffffffu, db, 2);
+            if ((lane & 3) == 0) {
+                if (ta < nt) den[(t0 + ta) * H + h] = suma + ia * da;
+                if (tb < nt) den[(t0 + tb) * H + h] = sumb + ib * db;
             }
         }
     }
-    float* ob = out + t0 * H * dv + (int64_t)h * dv + v_lo;
-#pragma unroll
-    for (int x = 0; x < 8; ++x)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int t = e < 2 ? ta : tb, col = x * 8 + c2 + (e & 1);
-            if (t < nt && col < nv) ob[(int64_t)t * H * dv + col] = acc[x][e];
+    for (int tile = group * per; tile < min(tiles, (group + 1) * per); ++tile) {
+        const int v_lo = tile * kT, nv = min(kT, dv - v_lo), nvp = min(kT, dvp - v_lo);
+        __syncthreads();                                    // the keys, or the tile before, have been read
+        const float* Sb = S0 + at * d * dvp + v_lo;
+        for (int idx = tid; idx < dp * (kT / 4); idx += 256) {
+            const int i = idx / (kT / 4), q4 = 4 * (idx % (kT / 4));
+            unsigned char* dst = Ss + i * SPB + q4 * 4;
+            if (i < d && q4 < nvp) copy_async_16b(dst, Sb + (int64_t)i * dvp + q4);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
         }
-    if (LOG && tile == 0) {
-        // n . q: the weights' sum and what the start of the chunk brought
-        suma += __shfl_xor_sync(0xffffffffu, suma, 1); suma += __shfl_xor_sync(0xffffffffu, suma, 2);
-        sumb += __shfl_xor_sync(0xffffffffu, sumb, 1); sumb += __shfl_xor_sync(0xffffffffu, sumb, 2);
-        const float* nb = N0 + at * d;
-        float da = 0.f, db = 0.f;
-        for (int i = lane & 3; i < d; i += 4) {
-            const float nv_ = nb[i];
-            da += nv_ * __bfloat162float(Qs[ta * kp + i]);
-            db += nv_ * __bfloat162float(Qs[tb * kp + i]);
+        fill_rows(Vs, kVP, in.p + t0 * in.ld + in.v + (int64_t)h * dv + v_lo, in.ld, nv, kT, nt, in.act, in.vec);
+        copy_async_wait_all();
+        __syncthreads();
+        float acc[4][4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+        for (int ks = 0; ks < dp; ks += 16) {
+            uint32_t a[4];
+            ldmatrix_x4(a, Qs + (wr * 16 + (lane & 15)) * kp + ks + (lane >> 4) * 8);
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                uint32_t s4[4];                             // eight columns: high parts, then remainders
+                ldmatrix_x4_trans(s4, Ss + (ks + (lane & 15)) * SPB + (wc * 4 + x) * 32 + (lane >> 4) * 16);
+                mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], s4[0], s4[1]);
+                mma_bf16_16816(acc[x], a[0], a[1], a[2], a[3], s4[2], s4[3]);
+            }
         }
-        da += __shfl_xor_sync(0xffffffffu, da, 1); da += __shfl_xor_sync(0xffffffffu, da, 2);
-        db += __shfl_xor_sync(0xffffffffu, db, 1); db += __shfl_xor_sync(0xffffffffu, db, 2);
-        if ((lane & 3) == 0) {
-            if (ta < nt) den[(t0 + ta) * H + h] = suma + ia * da;
-            if (tb < nt) den[(t0 + tb) * H + h] = sumb + ib * db;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) { acc[x][0] *= ia; acc[x][1] *= ia; acc[x][2] *= ib; acc[x][3] *= ib; }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            if (kk <= wr) {
+#pragma unroll
+                for (int x = 0; x < 4; x += 2) {
+                    uint32_t b4[4];
+                    ldmatrix_x4_trans(b4, Vs + (kk * 16 + (lane & 15)) * kVP + (wc * 4 + x + (lane >> 4)) * 8);
+                    mma_bf16_16816(acc[x], wh[kk][0], wh[kk][1], wh[kk][2], wh[kk][3], b4[0], b4[1]);
+                    mma_bf16_16816(acc[x], wl[kk][0], wl[kk][1], wl[kk][2], wl[kk][3], b4[0], b4[1]);
+                    mma_bf16_16816(acc[x + 1], wh[kk][0], wh[kk][1], wh[kk][2], wh[kk][3], b4[2], b4[3]);
+                    mma_bf16_16816(acc[x + 1], wl[kk][0], wl[kk][1], wl[kk][2], wl[kk][3], b4[2], b4[3]);
+                }
+            }
+        }
+        float* ob = out + t0 * H * dv + (int64_t)h * dv + v_lo;
+        const bool pair = (dv & 1) == 0;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const int col = (wc * 4 + x) * 8 + c2;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int t = e ? tb : ta;
+                if (t < nt) {
+                    float* p = ob + (int64_t)t * H * dv + col;
+                    if (pair && col + 1 < nv) *reinterpret_cast<float2*>(p) = make_float2(acc[x][2 * e], acc[x][2 * e + 1]);
+                    else { if (col < nv) p[0] = acc[x][2 * e]; if (col + 1 < nv) p[1] = acc[x][2 * e + 1]; }
+                }
+            }
         }
     }
 }
@@ -808,17 +933,21 @@ static bool bad_memory(int B, int H, int d, int dv, int64_t ld) {
 }
 
 // The log gates of a step and the chain of their running maximum (state: float rows, m [H] at m_off).  gates and logs
-// hold T * H * 4 floats (logs may be null).
+// hold T * H * 4 floats (logs may be null).  scan: the chain composed in a tree (see memory_gates_kernel).
 int mi_memory_gates(const float* proj, int ld, int col_i, int col_f, const float* bi, const float* bf, float cap,
                     float* state, int64_t stride, int64_t m_off, const int* q_start, const int* state_slot, float* gates,
-                    float* logs, int B, int H, cudaStream_t stream) {
+                    float* logs, int B, int H, int scan, cudaStream_t stream) {
     if (B <= 0) return kOk;
     if (bad_memory(B, H, 1, 1, ld)) return kBadShape;
     if (!(cap > 0.f)) { set_last_error("matrix memory: gates capped at %g", (double)cap); return kBadShape; }
     const mem::LogGates lg = {proj, ld, col_i, col_f, bi, bf, cap};
     const mem::State st = {state, stride, 0, 0, m_off};
-    launch_dependent(mem::memory_gates_kernel, dim3(H, B), dim3(256), 0, stream, lg, st, q_start, state_slot,
-                     (float4*)gates, (float4*)logs, H);
+    if (scan)
+        launch_dependent(mem::memory_gates_kernel<true>, dim3(H, B), dim3(256), 0, stream, lg, st, q_start, state_slot,
+                         (float4*)gates, (float4*)logs, H);
+    else
+        launch_dependent(mem::memory_gates_kernel<false>, dim3(H, B), dim3(256), 0, stream, lg, st, q_start, state_slot,
+                         (float4*)gates, (float4*)logs, H);
     return finish_launch("memory_gates");
 }
 
@@ -852,68 +981,72 @@ int mi_memory_walk(const float* proj, int ld, int col_q, int col_k, int col_v, i
 
 int mi_memory_chunk_tokens() { return mem::kC; }
 
-// The same over chunks of 64 tokens on the tensor cores.  U: (T / 64 + B) * H * d * dv floats of scratch, Un: the same
-// without dv (with gates), keepc: without d as well.
-int mi_memory_chunks(const float* proj, int ld, int col_q, int col_k, int col_v, int act, float q_scale, float* state,
+// floats of a row of the chunks' scratch U for a value size
+int mi_memory_chunk_value_pitch(int dv) { return (dv + 7) / 8 * 8; }
+
+// The same over chunks of 64 tokens on the tensor cores: q, k and v as columns of bfloat16 rows.  gates, logs: as
+// mi_memory_gates leaves them, or null with decay.  U: (T / 64 + B) * H * d * mi_memory_chunk_value_pitch(dv) floats of
+// scratch, Un: (..) * H * d (with gates), keepc: (..) * H.
+int mi_memory_chunks(const void* proj, int ld, int col_q, int col_k, int col_v, int act, float q_scale, float* state,
                      int64_t stride, int64_t s_off, int64_t n_off, const float* gates, const float* logs,
                      const float* decay, const int* q_start, const int* state_slot, float* out, float* den, float* U,
                      float* Un, float* keepc, int B, int max_q_len, int H, int d, int dv, cudaStream_t stream) {
     if (B <= 0 || max_q_len <= 0) return kOk;
     if (bad_memory(B, H, d, dv, ld)) return kBadShape;
     const int tiles = (dv + mem::kT - 1) / mem::kT, dp = (d + 15) / 16 * 16, chunks = (max_q_len + mem::kC - 1) / mem::kC;
+    const int dvp = mi_memory_chunk_value_pitch(dv);
     if ((gates == nullptr) == (decay == nullptr) || (gates && (!den || !logs || !Un)) || !U || !keepc ||
-        (int64_t)H * tiles > 65535) {
+        (reinterpret_cast<uintptr_t>(U) & 15) || (int64_t)H * tiles > 65535) {
         set_last_error("matrix memory in chunks: log gates or fixed decays with their scratch; %d heads x %d value tiles", H, tiles);
         return kBadShape;
     }
-    const mem::Rows in = {proj, ld, col_q, col_k, col_v, act, q_scale};
-    const int vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 && col_v % 4 == 0 &&
+    const int vec = d % 8 == 0 && dv % 8 == 0 && ld % 8 == 0 && col_q % 8 == 0 && col_k % 8 == 0 && col_v % 8 == 0 &&
                     (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
-    const int vec_s = dv % 4 == 0 && (reinterpret_cast<uintptr_t>(U) & 15) == 0;
-    const dim3 grid(chunks, H * tiles, B);
-    const size_t tile_bytes = (size_t)mem::kC * (dp + 8) * 2, v_bytes = (size_t)mem::kC * mem::kVP * 2;
-    const size_t smem_s = 2 * tile_bytes + v_bytes, smem_o = 2 * tile_bytes + v_bytes + (size_t)2 * dp * mem::kVP * 2;
+    const mem::RowsB in = {(const __nv_bfloat16*)proj, ld, col_q, col_k, col_v, act, q_scale, vec};
+    // value tiles a block of the outputs walks over: as many as leave two blocks per SM
+    const int64_t blocks = (int64_t)chunks * H * tiles * B;
+    int per = (int)(blocks / 296);
+    per = per < 1 ? 1 : (per > tiles ? tiles : per);
+    const int groups = (tiles + per - 1) / per;
+    const size_t rows_bytes = (size_t)mem::kC * (dp + 8) * 2, v_bytes = (size_t)mem::kC * mem::kVP * 2;
+    const size_t s_bytes = (size_t)dp * (mem::kT * 4 + 16);
+    const size_t smem_s = rows_bytes + 2 * v_bytes;
+    const size_t smem_o = rows_bytes + v_bytes + (rows_bytes > s_bytes ? rows_bytes : s_bytes);
 #define MI_CHUNKS(LOG)                                                                                                 \
     do {                                                                                                               \
         cudaFuncSetAttribute(mem::memory_chunk_states_kernel<LOG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_s); \
         cudaFuncSetAttribute(mem::memory_chunk_outputs_kernel<LOG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o); \
-        launch_dependent(mem::memory_chunk_states_kernel<LOG>, grid, dim3(128), smem_s, stream, in, (const float4*)gates, \
-                         (const float4*)logs, decay, q_start, U, Un, keepc, H, d, dv, dp, tiles, vec);                 \
+        launch_dependent(mem::memory_chunk_states_kernel<LOG>, dim3(chunks, H * tiles, B), dim3(128), smem_s, stream, in, \
+                         (const float4*)gates, (const float4*)logs, decay, q_start, U, Un, keepc, H, d, dv, dvp, dp, tiles); \
+        launch_dependent(mem::memory_chunk_chain_kernel, dim3((d * (dvp / 8) + 255) / 256, H, B), dim3(256), 0, stream, U, \
+                         (const float*)keepc, state, stride, s_off, q_start, state_slot, H, d, dv, dvp);               \
+        if (LOG)                                                                                                       \
+            launch_dependent(mem::memory_chunk_norm_chain_kernel, dim3((d + 255) / 256, H, B), dim3(256), 0, stream, Un, \
+                             (const float*)keepc, state, stride, n_off, q_start, state_slot, H, d);                    \
+        launch_dependent(mem::memory_chunk_outputs_kernel<LOG>, dim3(chunks, H * groups, B), dim3(256), smem_o, stream, in, \
+                         (const float4*)gates, (const float4*)logs, decay, q_start, (const float*)U, (const float*)Un, out, \
+                         den, H, d, dv, dvp, dp, tiles, per, groups);                                                  \
     } while (0)
     if (gates) MI_CHUNKS(true); else MI_CHUNKS(false);
 #undef MI_CHUNKS
-    int launched = 3;
-    const int size = d * dv;
-    if (size % 4 == 0 && s_off % 4 == 0 && stride % 4 == 0 && vec_s && (reinterpret_cast<uintptr_t>(state) & 15) == 0)
-        launch_dependent(mem::memory_chunk_chain_kernel<4>, dim3((size / 4 + 255) / 256, H, B), dim3(256), 0, stream, U,
-                         (const float*)keepc, state, stride, s_off, q_start, state_slot, H, size);
-    else
-        launch_dependent(mem::memory_chunk_chain_kernel<1>, dim3((size + 255) / 256, H, B), dim3(256), 0, stream, U,
-                         (const float*)keepc, state, stride, s_off, q_start, state_slot, H, size);
-    if (gates) {
-        launch_dependent(mem::memory_chunk_chain_kernel<1>, dim3((d + 255) / 256, H, B), dim3(256), 0, stream, Un,
-                         (const float*)keepc, state, stride, n_off, q_start, state_slot, H, d);
-        ++launched;
-        launch_dependent(mem::memory_chunk_outputs_kernel<true>, grid, dim3(128), smem_o, stream, in, (const float4*)gates,
-                         (const float4*)logs, decay, q_start, (const float*)U, (const float*)Un, out, den, H, d, dv, dp,
-                         tiles, vec, vec_s);
-    } else {
-        launch_dependent(mem::memory_chunk_outputs_kernel<false>, grid, dim3(128), smem_o, stream, in, (const float4*)gates,
-                         (const float4*)logs, decay, q_start, (const float*)U, (const float*)Un, out, den, H, d, dv, dp,
-                         tiles, vec, vec_s);
-    }
-    return finish_launch("memory_chunks", launched);
+    return finish_launch("memory_chunks", gates ? 4 : 3);
 }
 
-int mi_memory_finish(const float* o, const float* den, const float* gates, const float* gate, int ld_gate, const float* w,
-                     void* out, int adtype, int T, int H, int dv, float eps, cudaStream_t stream) {
+// out [T, n] = rmsnorm over groups of gs columns of o / (max(|den|, exp(-m)) + 1e-6), times w [n], times logistic(gate);
+// den and gates null: nothing is divided.  gate: rows of ld_gate numbers of the type gdtype.
+int mi_memory_finish(const float* o, const float* den, const float* gates, const void* gate, int gdtype, int ld_gate,
+                     const float* w, void* out, int adtype, int T, int n, int gs, float eps, cudaStream_t stream) {
     if (T <= 0) return kOk;
-    if (bad_memory(1, H, 1, dv, ld_gate)) return kBadShape;
+    if (gs < 1 || n % gs || n / gs > 65535 || (den == nullptr) != (gates == nullptr)) {
+        set_last_error("matrix memory: %d columns in groups of %d", n, gs);
+        return kBadShape;
+    }
+    const int vec = gs % 4 == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
     int threads = 32;
-    while (threads < dv && threads < 128) threads *= 2;
-    MI_DISPATCH_1(adtype, AT,
-        launch_dependent(mem::memory_finish_kernel<AT>, dim3(T, H), dim3(threads), 0, stream, o, den, (const float4*)gates,
-                         gate, ld_gate, w, (AT*)out, H, dv, eps));
+    while (threads < (vec ? gs / 4 : gs) && threads < 128) threads *= 2;
+    MI_DISPATCH_2(adtype, AT, gdtype, GT,
+        launch_dependent(mem::memory_finish_kernel<AT, GT>, dim3(T, n / gs), dim3(threads), 0, stream, o, den,
+                         (const float4*)gates, (const GT*)gate, ld_gate, w, (AT*)out, n, gs, eps, vec));
     return finish_launch("memory_finish");
 }
 

@@ -1516,8 +1516,8 @@ class MemoryState:
         self.floats = self.m + (up(heads) if log_gates else 0)
 
 
-def _chk_memory(what, proj, cols, st: MemoryState, state, q_start, state_slot):
-    _chk(proj, what + " proj", F32)
+def _chk_memory(what, proj, cols, st: MemoryState, state, q_start, state_slot, dtype=F32):
+    _chk(proj, what + " proj", dtype)
     _chk(state, what + " state", F32)
     B = state_slot.numel()
     _chk(q_start, what + " q_start", I32, (B + 1,))
@@ -1530,84 +1530,107 @@ def _chk_memory(what, proj, cols, st: MemoryState, state, q_start, state_slot):
     return B
 
 
-def _chk_gates(what, proj, gates, decay, heads):
+def _chk_gates(what, rows, gates, decay, heads):
     if (gates is None) == (decay is None):
         raise ValueError(f"{what}: either log gates or fixed decays")
     _chk(decay, what + " decay", F32, (heads,))
     if gates is not None:
         _chk(gates.bi, what + " bi", F32, (heads,))
         _chk(gates.bf, what + " bf", F32, (heads,))
-        if gates.col_i + heads > proj.shape[1] or gates.col_f + heads > proj.shape[1]:
+        _chk(rows, what + " gates' rows", F32)
+        if gates.col_i + heads > rows.shape[1] or gates.col_f + heads > rows.shape[1]:
             raise ValueError(f"{what}: the gates' columns are out of range")
 
 
+def _memory_gates(rows, gates: LogGates, st: MemoryState, state, q_start, state_slot, B, scan: bool):
+    """``(gates [T, H, 4], logs or None)`` as the walk and the chunks take them; m in the state moves on."""
+    T, H = rows.shape[0], st.heads
+    g = torch.empty(T, H, 4, dtype=F32, device=rows.device)
+    logs = torch.empty(T, H, 4, dtype=F32, device=rows.device) if scan else None
+    check(library().mi_memory_gates(_ptr(rows), rows.shape[1], gates.col_i, gates.col_f, _ptr(gates.bi), _ptr(gates.bf),
+                                    gates.cap, _ptr(state), state.shape[1], st.m, _ptr(q_start), _ptr(state_slot), _ptr(g),
+                                    _ptr(logs), B, H, int(scan), _stream()), "memory_gates")
+    return g, logs
+
+
 def memory_chunk_tokens() -> int:
-    """Tokens per chunk of :func:`memory_scan` with ``chunks``."""
+    """Tokens per chunk of :func:`memory_chunks`."""
     return int(library().mi_memory_chunk_tokens())
 
 
 def memory_scan(proj: torch.Tensor, cols: Tuple[int, int, int], st: MemoryState, state: torch.Tensor,
                 q_start: torch.Tensor, state_slot: torch.Tensor, gates: Optional[LogGates] = None,
-                decay: Optional[torch.Tensor] = None, q_scale: float = 1.0, silu: bool = False, chunks: bool = False,
-                max_q_len: int = 0):
-    """``S <- keep S + write k v^T``, ``o = S^T q`` per head over every request's portion; q, k (``heads x d``) and v
-    (``heads x dv``) are the columns ``cols`` of the float32 rows ``proj``, through silu first with ``silu``; q also
-    times ``q_scale``.
+                decay: Optional[torch.Tensor] = None, q_scale: float = 1.0, silu: bool = False):
+    """``S <- keep S + write k v^T``, ``o = S^T q`` per head over every request's portion, token by token in one order
+    whatever the cut of a step; q, k (``heads x d``) and v (``heads x dv``) are the columns ``cols`` of the float32 rows
+    ``proj``, through silu first with ``silu``; q also times ``q_scale``.
 
     ``decay`` (float32 ``[heads]``): ``keep = decay``, ``write = 1``; returns ``o`` float32 ``[T, heads*dv]``.
-    ``gates``: with a running maximum ``m <- max(f + m, i)``, ``keep = exp(f + m_before - m)``, ``write = exp(i - m)``,
-    and ``n <- keep n + write k`` beside S; returns ``(o, n . q [T, heads], gates [T, heads, 4])`` for
-    :func:`memory_finish` (``gates[..., 2] = exp(-m)``).
-
-    The walk goes token by token in one order whatever the cut of a step.  ``chunks`` (bfloat16 path): on the tensor
-    cores over chunks of :func:`memory_chunk_tokens` tokens, q, k and v rounded to bfloat16, what the recurrence makes
-    held in float (as pairs of bfloat16 where it is an operand); ``max_q_len`` is the longest portion."""
+    ``gates`` (their columns are columns of ``proj``): with a running maximum ``m <- max(f + m, i)``,
+    ``keep = exp(f + m_before - m)``, ``write = exp(i - m)``, and ``n <- keep n + write k`` beside S; returns
+    ``(o, n . q [T, heads], gates [T, heads, 4])`` for :func:`memory_finish` (``gates[..., 2] = exp(-m)``)."""
     what = "memory_scan"
     B = _chk_memory(what, proj, cols, st, state, q_start, state_slot)
-    H, d, dv = st.heads, st.d, st.dv
+    H, d, dv, T = st.heads, st.d, st.dv, proj.shape[0]
     _chk_gates(what, proj, gates, decay, H)
-    T, dev, lib = proj.shape[0], proj.device, library()
-    new = lambda *shape: torch.empty(*shape, dtype=F32, device=dev)
-    g = logs = den = None
+    g = den = None
     if gates is not None:
-        g, den = new(T, H, 4), new(T, H)
-        logs = new(T, H, 4) if chunks else None
-        check(lib.mi_memory_gates(_ptr(proj), proj.shape[1], gates.col_i, gates.col_f, _ptr(gates.bi), _ptr(gates.bf),
-                                  gates.cap, _ptr(state), state.shape[1], st.m, _ptr(q_start), _ptr(state_slot), _ptr(g),
-                                  _ptr(logs), B, H, _stream()), "memory_gates")
-    out = new(T, H * dv)
-    head = (_ptr(proj), proj.shape[1], int(cols[0]), int(cols[1]), int(cols[2]), int(bool(silu)), float(q_scale),
-            _ptr(state), state.shape[1], st.s, st.n)
-    if chunks:
-        n = T // memory_chunk_tokens() + B
-        U, keep = new(n * H * d * dv), new(n * H)
-        Un = new(n * H * d) if gates is not None else None
-        check(lib.mi_memory_chunks(*head, _ptr(g), _ptr(logs), _ptr(decay), _ptr(q_start), _ptr(state_slot), _ptr(out),
-                                   _ptr(den), _ptr(U), _ptr(Un), _ptr(keep), B, int(max_q_len), H, d, dv, _stream()),
-              "memory_chunks")
-    else:
-        check(lib.mi_memory_walk(*head, _ptr(g), _ptr(decay), _ptr(q_start), _ptr(state_slot), _ptr(out), _ptr(den), B, H,
-                                 d, dv, _stream()), "memory_walk")
+        g, _ = _memory_gates(proj, gates, st, state, q_start, state_slot, B, False)
+        den = torch.empty(T, H, dtype=F32, device=proj.device)
+    out = torch.empty(T, H * dv, dtype=F32, device=proj.device)
+    check(library().mi_memory_walk(_ptr(proj), proj.shape[1], int(cols[0]), int(cols[1]), int(cols[2]), int(bool(silu)),
+                                   float(q_scale), _ptr(state), state.shape[1], st.s, st.n, _ptr(g), _ptr(decay),
+                                   _ptr(q_start), _ptr(state_slot), _ptr(out), _ptr(den), B, H, d, dv, _stream()),
+          "memory_walk")
     return out if gates is None else (out, den, g)
 
 
-def memory_finish(o: torch.Tensor, den: torch.Tensor, gates: torch.Tensor, gate: torch.Tensor, gate_col: int,
-                  weight: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
-    """``rmsnorm_head(o / (max(|den|, gates[..., 2]) + 1e-6)) * weight * logistic(gate)`` with a weight per column."""
+def memory_chunks(proj: torch.Tensor, cols: Tuple[int, int, int], st: MemoryState, state: torch.Tensor,
+                  q_start: torch.Tensor, state_slot: torch.Tensor, max_q_len: int, gates: Optional[LogGates] = None,
+                  gate_rows: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None, q_scale: float = 1.0,
+                  silu: bool = False):
+    """:func:`memory_scan` for long portions, on the tensor cores over chunks of :func:`memory_chunk_tokens` tokens:
+    ``proj`` holds q, k and v in bfloat16 (with ``silu`` rounded to it once more), the log gates' columns are columns of
+    the float32 rows ``gate_rows``; what the recurrence makes is held in float, as a pair of bfloat16 numbers where it is
+    an operand.  ``max_q_len`` is the longest portion.  Sums run in another order than the walk's."""
+    what = "memory_chunks"
+    B = _chk_memory(what, proj, cols, st, state, q_start, state_slot, BF16)
+    H, d, dv, T, dev = st.heads, st.d, st.dv, proj.shape[0], proj.device
+    _chk_gates(what, gate_rows, gates, decay, H)
+    new = lambda *shape: torch.empty(*shape, dtype=F32, device=dev)
+    g = logs = den = Un = None
+    n = T // memory_chunk_tokens() + B
+    if gates is not None:
+        g, logs = _memory_gates(gate_rows, gates, st, state, q_start, state_slot, B, True)
+        den, Un = new(T, H), new(n * H * d)
+    out, keep = new(T, H * dv), new(n * H)
+    U = new(n * H * d * int(library().mi_memory_chunk_value_pitch(dv)))
+    check(library().mi_memory_chunks(
+        _ptr(proj), proj.shape[1], int(cols[0]), int(cols[1]), int(cols[2]), int(bool(silu)), float(q_scale), _ptr(state),
+        state.shape[1], st.s, st.n, _ptr(g), _ptr(logs), _ptr(decay), _ptr(q_start), _ptr(state_slot), _ptr(out), _ptr(den),
+        _ptr(U), _ptr(Un), _ptr(keep), B, int(max_q_len), H, d, dv, _stream()), what)
+    return out if gates is None else (out, den, g)
+
+
+def memory_finish(o: torch.Tensor, gate: torch.Tensor, gate_col: int, weight: torch.Tensor, eps: float,
+                  out_dtype: torch.dtype, groups: int = 1, den: Optional[torch.Tensor] = None,
+                  gates: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``rmsnorm(o) * weight * logistic(gate)`` over ``groups`` equal parts of every float32 row of ``o``, with a weight
+    per column and the gate in the columns ``gate_col ..`` of ``gate`` (float32 or bfloat16).  With ``den`` and ``gates``
+    (:func:`memory_scan`; a part is then a head) ``o`` is first divided by ``max(|den|, gates[..., 2]) + 1e-6``."""
     T, n = o.shape
-    H = den.shape[1]
-    dv = n // H
     _chk(o, "memory_finish o", F32)
-    _chk(den, "memory_finish den", F32, (T, H))
-    _chk(gates, "memory_finish gates", F32, (T, H, 4))
-    _chk(gate, "memory_finish gate", F32, (T, None))
+    _chk(den, "memory_finish den", F32, (T, groups))
+    _chk(gates, "memory_finish gates", F32, (T, groups, 4))
+    _chk(gate, "memory_finish gate", None, (T, None))
     _chk(weight, "memory_finish weight", F32, (n,))
-    if gate_col + n > gate.shape[1]:
-        raise ValueError("memory_finish: the gate's columns are out of range")
+    if gate_col < 0 or gate_col + n > gate.shape[1] or n % groups:
+        raise ValueError("memory_finish: the gate's columns are out of range, or the parts are not equal")
     out = torch.empty(T, n, dtype=out_dtype, device=o.device)
-    check(library().mi_memory_finish(_ptr(o), _ptr(den), _ptr(gates), gate.data_ptr() + 4 * gate_col, gate.shape[1],
-                                     _ptr(weight), _ptr(out), _code(out, "memory_finish out"), T, H, dv, float(eps),
-                                     _stream()), "memory_finish")
+    check(library().mi_memory_finish(_ptr(o), _ptr(den), _ptr(gates), gate.data_ptr() + gate.element_size() * gate_col,
+                                     _code(gate, "memory_finish gate"), gate.shape[1], _ptr(weight), _ptr(out),
+                                     _code(out, "memory_finish out"), T, n, n // groups, float(eps), _stream()),
+          "memory_finish")
     return out
 
 

@@ -90,10 +90,10 @@ _SIGNATURES = {
     "mi_normed_pair_add": [P, P, P, F, F, P, P, F, F, P, P, I, P, I, I, I, F, P],
     "mi_squared_relu": [P, P, I, L, P],
     "mi_causal_conv_plain": [P, I, P, P, P, I, P, L, P, P, P, P, I, I, I, I, I, P],
-    "mi_memory_gates": [P, I, I, I, P, P, F, P, L, L, P, P, P, P, I, I, P],
+    "mi_memory_gates": [P, I, I, I, P, P, F, P, L, L, P, P, P, P, I, I, I, P],
     "mi_memory_walk": [P, I, I, I, I, I, F, P, L, L, L, P, P, P, P, P, P, I, I, I, I, P],
     "mi_memory_chunks": [P, I, I, I, I, I, F, P, L, L, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P],
-    "mi_memory_finish": [P, P, P, P, I, P, P, I, I, I, I, F, P],
+    "mi_memory_finish": [P, P, P, P, I, I, P, P, I, I, I, I, F, P],
     "mi_memory_decode": [P, I, I, I, I, I, F, I, I, P, P, F, P, L, L, L, L, P, P, P, I, P, F, P, I, P, I, I, I, I, P],
     "mi_lru_gates_tc": [P, P, P, P, P, P, P, P, I, I, I, P],
     "mi_lru_prepare": [P, P, P, P, P, P, I, I, P],
@@ -125,6 +125,7 @@ _OTHERS = {
     "mi_attn_mix_supported": ([I, I, I, I, I], c_int),
     "mi_attn_mix_independent_supported": ([I, I, I, I, I], c_int),
     "mi_memory_chunk_tokens": ([], c_int),
+    "mi_memory_chunk_value_pitch": ([I], c_int),
     "mi_lru_segment_tokens": ([], c_int),
     "mi_attn_prefill_tc_shared_supported": ([I, I, I, I], c_int),
     "mi_attn_prefill_tc_logistic_supported": ([I, I, I], c_int),

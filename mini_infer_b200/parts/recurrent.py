@@ -397,11 +397,15 @@ class MatrixLSTM(Mixer):
         self.rt = rt
         m, dev, p = rt.precision.matrix, rt.device, self.prefix
         # one product for everything that reads the layer's input: q | k | v | output gate | input gate | forget gate
+        # (long portions: two, the first four in bfloat16 and the gates of the recurrence in float32)
         self.w_in = torch.cat([m(tensors[p + n], dev) for n in ("q", "k", "v", "g", "i", "f")], dim=0)
         self.cols = (0, self.n_qk, 2 * self.n_qk)
         self.col_gate = 2 * self.n_qk + self.n_v
         col_i = self.col_gate + self.n_v
-        self.gates = F.LogGates(col_i, col_i + self.nh, _f32(tensors[p + "i.b"], dev), _f32(tensors[p + "f.b"], dev), self.cap)
+        bi, bf = _f32(tensors[p + "i.b"], dev), _f32(tensors[p + "f.b"], dev)
+        self.gates = F.LogGates(col_i, col_i + self.nh, bi, bf, self.cap)
+        self.gates_alone = F.LogGates(0, self.nh, bi, bf, self.cap)
+        self.w_main, self.w_gates = self.w_in[:col_i], self.w_in[col_i:]
         self.norm_w = _f32(tensors[p + "norm"], dev)
         self.w_o = m(tensors[p + "o"], dev)
 
@@ -413,6 +417,13 @@ class MatrixLSTM(Mixer):
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
         state = ctx.states[cache.group]
+        if _scan_in_chunks(self.rt, ctx):
+            proj = linear(x, self.w_main, self.rt.act)
+            o, den, g = F.memory_chunks(proj, self.cols, self.state, state, ctx.q_start, ctx.state_slot, ctx.max_q_len,
+                                        gates=self.gates_alone, gate_rows=linear(x, self.w_gates, torch.float32),
+                                        q_scale=self.d ** -0.5)
+            y = F.memory_finish(o, proj, self.col_gate, self.norm_w, self.eps, self.rt.act, self.nh, den, g)
+            return linear(y, self.w_o, torch.float32)
         proj = linear(x, self.w_in, torch.float32)
         if ctx.prefetch is not None:
             ctx.prefetch((self.w_o,))       # arrives while the states are read and written
@@ -421,9 +432,8 @@ class MatrixLSTM(Mixer):
             y = F.memory_decode(*args, gates=self.gates, q_scale=self.d ** -0.5, gate_col=self.col_gate,
                                 weight=self.norm_w, eps=self.eps, out_dtype=self.rt.act)
         else:
-            o, den, g = F.memory_scan(*args, gates=self.gates, q_scale=self.d ** -0.5,
-                                      chunks=_scan_in_chunks(self.rt, ctx), max_q_len=ctx.max_q_len)
-            y = F.memory_finish(o, den, g, proj, self.col_gate, self.norm_w, self.eps, self.rt.act)
+            o, den, g = F.memory_scan(*args, gates=self.gates, q_scale=self.d ** -0.5)
+            y = F.memory_finish(o, proj, self.col_gate, self.norm_w, self.eps, self.rt.act, self.nh, den, g)
         return linear(y, self.w_o, torch.float32)
 
 
@@ -438,7 +448,7 @@ class FixedDecayAttention(Mixer):
     ``norm [heads*value_dim]``, ``o [hidden, heads*value_dim]``."""
 
     graph_safe = True
-    kernel_files = ("matrix_memory.cu", "recurrent.cu")
+    kernel_files = ("matrix_memory.cu",)
 
     def __init__(self, params, prefix):
         super().__init__(params, prefix)
@@ -480,14 +490,16 @@ class FixedDecayAttention(Mixer):
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheBinding) -> torch.Tensor:
         state = ctx.states[cache.group]
-        proj = linear(x, self.w_in, torch.float32)
+        chunks = _scan_in_chunks(self.rt, ctx)
+        proj = linear(x, self.w_in, self.rt.act if chunks else torch.float32)
         args = (proj, self.cols, self.state, state, ctx.q_start, ctx.state_slot)
-        if ctx.all_decode and self.rt.act == torch.bfloat16:
+        if chunks:
+            o = F.memory_chunks(*args, ctx.max_q_len, decay=self.decay, silu=True)
+        elif ctx.all_decode and self.rt.act == torch.bfloat16:
             o = F.memory_decode(*args, decay=self.decay, silu=True)
         else:
-            o = F.memory_scan(*args, decay=self.decay, silu=True, chunks=_scan_in_chunks(self.rt, ctx),
-                              max_q_len=ctx.max_q_len)
-        y = F.gated_group_rmsnorm(o, proj, 2 * self.n_qk + self.n_v, self.norm_w, 1, False, self.eps, self.rt.act)
+            o = F.memory_scan(*args, decay=self.decay, silu=True)
+        y = F.memory_finish(o, proj, 2 * self.n_qk + self.n_v, self.norm_w, self.eps, self.rt.act)
         return linear(y, self.w_o, torch.float32)
 
 

@@ -41,6 +41,8 @@ def memory_case(H, d, dv, lens, seed, log_gates, pad=3):
     cols = (pad, pad + n_qk, pad + 2 * n_qk)
     col_g = pad + 2 * n_qk + n_v
     width = col_g + n_v + 2 * H
+    if pad % 8 == 0:
+        width = -(-width // 8) * 8                        # rows, and with them heads of whole eights, on 16-byte boundaries
     xs = [bf(torch.randn(n, width, generator=g)) for n in lens]
     for x in xs:
         x[:, col_g + n_v:] *= 2.0
@@ -55,7 +57,7 @@ def memory_case(H, d, dv, lens, seed, log_gates, pad=3):
         if log_gates:
             c = extra["cap"]
             i = c * torch.tanh((z[:, extra["col_i"]:extra["col_i"] + H] + extra["bi"].double()) / c)
-            f = pd.log_sigmoid(c * torch.tanh((z[:, extra["col_i"] + H:] + extra["bf"].double()) / c))
+            f = pd.log_sigmoid(c * torch.tanh((z[:, extra["col_i"] + H:extra["col_i"] + 2 * H] + extra["bf"].double()) / c))
             o = pd.matrix_memory(q * d ** -0.5, k, v, i, f)
             y = pd.unit_rms(o, 1e-5).reshape(T, n_v) * extra["w"].double() * pd.sigmoid(z[:, col_g:col_g + n_v])
         else:
@@ -83,17 +85,21 @@ def run_memory(H, d, dv, xs, extra, cuts, log_gates, chunks, dtype, slots=None, 
         live = [r for r in range(len(xs)) if step < len(cuts[r])]
         rows = [xs[r][fed[r]:fed[r] + cuts[r][step]] for r in live]
         proj = torch.cat(rows).to(DEV).contiguous()
-        starts = [0]
-        for r in rows:
-            starts.append(starts[-1] + r.shape[0])
+        starts = [sum(r.shape[0] for r in rows[:n]) for n in range(len(rows) + 1)]
         args = (proj, extra["cols"], st, state, i32(starts), i32([slots[r] for r in live]))
-        longest = max(r.shape[0] for r in rows)
+        longest = max(cuts[r][step] for r in live)
         if decode and longest == 1:
             y = fn.memory_decode(*args, gate_col=extra["col_g"], weight=extra["w"].to(DEV), eps=1e-5, out_dtype=dtype, **kw)
         else:
-            y = fn.memory_scan(*args, chunks=chunks, max_q_len=longest, **kw)
+            rows = proj
+            if chunks:
+                rows = proj.to(torch.bfloat16)
+                y = fn.memory_chunks(rows, *args[1:], longest, gate_rows=proj, **kw)
+            else:
+                y = fn.memory_scan(*args, **kw)
             if log_gates:
-                y = fn.memory_finish(*y, proj, extra["col_g"], extra["w"].to(DEV), 1e-5, dtype)
+                o, den, gv = y
+                y = fn.memory_finish(o, rows, extra["col_g"], extra["w"].to(DEV), 1e-5, dtype, H, den, gv)
         for n, r in enumerate(live):
             got[r].append(y[starts[n]:starts[n + 1]].float().cpu())
             fed[r] += cuts[r][step]
@@ -122,12 +128,13 @@ def test_memory_walked_in_any_cut(H, d, dv, log_gates):
 
 @pytest.mark.parametrize("H,d,dv", SIZES)
 @pytest.mark.parametrize("log_gates", [True, False])
-def test_memory_in_chunks_and_decoded(H, d, dv, log_gates):
+@pytest.mark.parametrize("pad", [3, 8])
+def test_memory_in_chunks_and_decoded(H, d, dv, log_gates, pad):
     """Long portions over chunks of 64 tokens, portions that end inside a chunk, single tokens on the decode kernel.  The
     projections are bfloat16 numbers already, so the forms differ from the plain sums by what float and a pair of bfloat16
     lose only (silu, whose result the chunks round to bfloat16, aside)."""
     lens = [300, 1, 70, 65]
-    xs, want, extra = memory_case(H, d, dv, lens, 7 * H + d + dv, log_gates)
+    xs, want, extra = memory_case(H, d, dv, lens, 7 * H + d + dv, log_gates, pad)
     tol = 1e-3 if log_gates else 8e-3
     for cuts in ([[300], [1], [70], [65]], [[129, 64, 63] + [1] * 44, [1], [64, 6], [2, 63]],
                  [[250] + [1] * 50, [1], [20] + [1] * 50, [15] + [1] * 50]):
@@ -160,9 +167,9 @@ def test_a_write_is_read_back_after_hundreds_of_tokens(log_gates):
     if log_gates:
         x[:, extra["col_i"]:extra["col_i"] + H] = -2.0
         x[5, extra["col_i"]:extra["col_i"] + H] = 4.0
-        x[:, extra["col_i"] + H:] = 8.0                             # forget gates near one
+        x[:, extra["col_i"] + H:extra["col_i"] + 2 * H] = 8.0                             # forget gates near one
         i = extra["cap"] * torch.tanh((x[:, extra["col_i"]:extra["col_i"] + H].double() + extra["bi"].double()) / extra["cap"])
-        f = pd.log_sigmoid(extra["cap"] * torch.tanh((x[:, extra["col_i"] + H:].double() + extra["bf"].double()) / extra["cap"]))
+        f = pd.log_sigmoid(extra["cap"] * torch.tanh((x[:, extra["col_i"] + H:extra["col_i"] + 2 * H].double() + extra["bf"].double()) / extra["cap"]))
         z = x.double()
         o = pd.matrix_memory(z[:, c[0]:c[0] + H * d].reshape(T, H, d) * d ** -0.5, z[:, c[1]:c[1] + H * d].reshape(T, H, d),
                              z[:, c[2]:c[2] + H * dv].reshape(T, H, dv), i, f)
@@ -188,12 +195,12 @@ def test_gates_at_both_ends():
     extra["cap"] = 15.0
     g = torch.Generator().manual_seed(9)
     x[:, ci:ci + H] = bf(torch.randn(T, H, generator=g) * 20)
-    x[:, ci + H:] = bf(torch.randn(T, H, generator=g) * 20)
-    x[100:180, ci + H:] = -60.0                                     # forget everything at every token
+    x[:, ci + H:ci + 2 * H] = bf(torch.randn(T, H, generator=g) * 20)
+    x[100:180, ci + H:ci + 2 * H] = -60.0                                     # forget everything at every token
     x[180:, ci:ci + H] = -60.0                                      # and write next to nothing
     z = x.double()
     i = 15 * torch.tanh((z[:, ci:ci + H] + extra["bi"].double()) / 15)
-    f = pd.log_sigmoid(15 * torch.tanh((z[:, ci + H:] + extra["bf"].double()) / 15))
+    f = pd.log_sigmoid(15 * torch.tanh((z[:, ci + H:ci + 2 * H] + extra["bf"].double()) / 15))
     o = pd.matrix_memory(z[:, c[0]:c[0] + H * d].reshape(T, H, d) * d ** -0.5, z[:, c[1]:c[1] + H * d].reshape(T, H, d),
                          z[:, c[2]:c[2] + H * dv].reshape(T, H, dv), i, f)
     want = pd.unit_rms(o, 1e-5).reshape(T, H * dv) * extra["w"].double() * pd.sigmoid(z[:, extra["col_g"]:extra["col_g"] + H * dv])
@@ -582,6 +589,16 @@ def test_two_normalised_outputs_join_the_residual(T, W, dtype):
     hidden, rows = h.to(DEV), [T - 1, 0]
     x = F().normed_pair_add(hidden, pair, w.to(DEV), 1e-5, dtype, i32(rows))
     assert torch.equal(hidden.cpu(), h) and close(x.float(), want[rows], tol)
+
+
+@pytest.mark.parametrize("n,gate_dtype", [(40, torch.float32), (96, torch.bfloat16), (33, torch.bfloat16), (2048, torch.float32)])
+def test_norm_of_all_heads_together_with_its_gate(n, gate_dtype):
+    g = torch.Generator().manual_seed(n)
+    T = 7
+    o, gate, w = torch.randn(T, n, generator=g) * 3, bf(torch.randn(T, n + 3, generator=g)), 1 + 0.2 * torch.randn(n, generator=g)
+    want = pd.unit_rms(o.double(), 1e-5) * w.double() * pd.sigmoid(gate[:, 1:n + 1].double())
+    got = F().memory_finish(o.to(DEV), gate.to(gate_dtype).to(DEV), 1, w.to(DEV), 1e-5, torch.float32)
+    assert close(got, want, 3e-6)
 
 
 @pytest.mark.parametrize("T,n", [(1, 33), (5, 64), (40, 100)])
