@@ -1142,9 +1142,9 @@ def _dedizen_kernel_work(cfg, T, B, ctx, decode):
             add("mem::memory_chunk_outputs_kernel", T * rows_in + states + T * v * 4, T * H * (2.0 * d * e + 64.0 * (d + e)))
             if log_gates:
                 add("mem::memory_gates_kernel", T * H * (8 + 32))
-                add("mem::memory_finish_kernel", T * v * (4 + 4 + 2))
+                add("mem::memory_finish_vec_kernel", T * v * (4 + 4 + 2))
         if not log_gates:
-            add("gated_group_rmsnorm_kernel", rows * v * (4 + 4 + 2))
+            add("mem::memory_finish_vec_kernel", rows * v * (4 + 2 + 2))
     for L in cfg["layers"]:
         m, ff = L["mixer"], L["mlp"]["ff"]
         if not decode:

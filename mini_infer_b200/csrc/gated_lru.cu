@@ -2,7 +2,7 @@
 // unit):  with u the output of a short convolution over time, split into `blocks` equal parts of n channels,
 //
 //   r = logistic(A_b u_b + ra),  i = logistic(I_b u_b + ri)        A_b, I_b [n, n], one pair per part
-//   log a = -8 r softplus(lam),  S_t = a S_(t-1) + sqrt(1 - a^2) i u,  out = S gelu(y + bias)
+//   log a = rate r,  rate = -8 softplus(lam),  S_t = a S_(t-1) + sqrt(1 - a^2) i u,  out = S gelu(y + bias)
 //
 //   lru_gates_tc   both gates' products on the tensor cores, gates and decays in the epilogue (bfloat16 path).  u is
 //                  float: it enters as the sum of three bfloat16 numbers, which holds all 24 bits of it, the matrices
@@ -29,13 +29,12 @@ constexpr int kMaxTaps = 8;
 constexpr int kSeg = 64;                     // tokens per segment
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
-// decay and drive of a channel from its gates' inputs; 1 - a^2 = -(e^(2 log a) - 1) without cancellation
-__device__ __forceinline__ void decay_drive(float zr, float zi, float lam, float u, float& a, float& x) {
-    const float log_a = -8.0f * sigmoid_f(zr) * softplus_f(lam);
+// decay and drive of a channel from its gates' inputs and its rate (-8 softplus(lam)); 1 - a^2 = -(e^(2 log a) - 1) without cancellation
+__device__ __forceinline__ void decay_drive(float zr, float zi, float rate, float u, float& a, float& x) {
+    const float log_a = rate * sigmoid_f(zr);
     a = expf(log_a);
     x = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_f(zi) * u;
 }
@@ -46,18 +45,25 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem_r
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
-// Block = 4 warps: 64 tokens x 32 output channels of one part, both gates.  ra, ri [blocks][n][n] bfloat16 (out, in).
-constexpr int kGT = 64, kGC = 32, kGK = 64, kGP = kGK + 8;
+// Block = 8 warps: 64 tokens x 64 output channels of one part, both gates (warp w: 16 tokens, 32 channels).  ra, ri
+// [blocks][n][n] bfloat16 (out, in).  The inner dimension goes by in slices of 32: while one slice is multiplied, the next
+// one's matrices are on their way (cp.async) and its rows of u are held in registers, split when the buffer is free.
+constexpr int kGT = 64, kGC = 64, kGK = 32, kGP = kGK + 8;
+struct GateTiles {
+    __nv_bfloat16 u[3][kGT][kGP];
+    __nv_bfloat16 w[2][kGC][kGP];
+};
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 lru_gates_tc_kernel(const float* __restrict__ u, const __nv_bfloat16* __restrict__ wr, const __nv_bfloat16* __restrict__ wi,
-                    const float* __restrict__ br, const float* __restrict__ bi, const float* __restrict__ lam,
-                    float* __restrict__ a_out, float* __restrict__ x_out, int T, int W, int n, int ctiles) {
-    __shared__ __align__(16) __nv_bfloat16 Us[3][kGT][kGP];
-    __shared__ __align__(16) __nv_bfloat16 Ws[2][kGC][kGP];
+                    const float* __restrict__ br, const float* __restrict__ bi, const float* __restrict__ rate,
+                    float* __restrict__ a_out, float* __restrict__ x_out, int T, int W, int n, int ctiles, int vec) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    GateTiles* buf = reinterpret_cast<GateTiles*>(raw);             // two of them
     wait_for_earlier_kernels();
     const int t0 = blockIdx.x * kGT, part = blockIdx.y / ctiles, c0 = (blockIdx.y % ctiles) * kGC;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r0 = lane >> 2, c2 = (lane & 3) * 2;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wt = warp & 3, wc = warp >> 2;
+    const int r0 = lane >> 2, c2 = (lane & 3) * 2;
     float acc[2][4][4];
 #pragma unroll
     for (int g = 0; g < 2; ++g)
@@ -67,43 +73,78 @@ lru_gates_tc_kernel(const float* __restrict__ u, const __nv_bfloat16* __restrict
             for (int e = 0; e < 4; ++e) acc[g][x][e] = 0.f;
     const __nv_bfloat16* w0 = wr + ((int64_t)part * n + c0) * n;
     const __nv_bfloat16* w1 = wi + ((int64_t)part * n + c0) * n;
-    for (int k0 = 0; k0 < n; k0 += kGK) {
-        __syncthreads();
-        for (int idx = tid; idx < kGT * (kGK / 2); idx += 128) {
-            const int j = idx / (kGK / 2), i = 2 * (idx % (kGK / 2));
-            float v[2];
+    const float* ub = u + (int64_t)part * n;
+    auto fetch_w = [&](int k0, GateTiles& b) {
+        for (int idx = tid; idx < 2 * kGC * (kGK / 8); idx += 256) {
+            const int i = 8 * (idx % (kGK / 8)), o = (idx / (kGK / 8)) % kGC, g = idx / (kGK / 8 * kGC);
+            __nv_bfloat16* dst = &b.w[g][o][i];
+            const __nv_bfloat16* src = (g ? w1 : w0) + (int64_t)o * n + k0 + i;
+            if (vec && c0 + o < n && k0 + i + 8 <= n) {
+                const uint32_t d = static_cast<uint32_t>(__cvta_generic_to_shared(dst));
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(d), "l"(src));
+            } else {
 #pragma unroll
-            for (int x = 0; x < 2; ++x)
-                v[x] = (t0 + j < T && k0 + i + x < n) ? u[(int64_t)(t0 + j) * W + part * n + k0 + i + x] : 0.f;
-#pragma unroll
-            for (int s = 0; s < 3; ++s) {
-                __nv_bfloat162 p = __floats2bfloat162_rn(v[0], v[1]);
-                *reinterpret_cast<__nv_bfloat162*>(&Us[s][j][i]) = p;
-                v[0] -= __bfloat162float(p.x);
-                v[1] -= __bfloat162float(p.y);
+                for (int x = 0; x < 8; ++x) dst[x] = c0 + o < n && k0 + i + x < n ? src[x] : __float2bfloat16_rn(0.f);
             }
         }
-        for (int idx = tid; idx < 2 * kGC * kGK; idx += 128) {
-            const int i = idx % kGK, o = (idx / kGK) % kGC, g = idx / (kGK * kGC);
-            __nv_bfloat16 v = __float2bfloat16_rn(0.f);
-            if (c0 + o < n && k0 + i < n) v = (g ? w1 : w0)[(int64_t)o * n + k0 + i];
-            Ws[g][o][i] = v;
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+    float4 held[2];                                                 // rows tid / 8 + 32 q, columns 4 (tid % 8) .. + 3
+    auto fetch_u = [&](int k0) {
+        const int i = k0 + 4 * (tid & 7);
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+            const int t = t0 + (tid >> 3) + 32 * q;
+            const float* p = ub + (int64_t)t * W + i;
+            held[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (t < T) {
+                if (vec && i + 4 <= n) held[q] = *reinterpret_cast<const float4*>(p);
+                else { if (i < n) held[q].x = p[0]; if (i + 1 < n) held[q].y = p[1]; if (i + 2 < n) held[q].z = p[2]; if (i + 3 < n) held[q].w = p[3]; }
+            }
         }
-        __syncthreads();
+    };
+    auto store_u = [&](GateTiles& b) {
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+            float v[4] = {held[q].x, held[q].y, held[q].z, held[q].w};
+#pragma unroll
+            for (int s = 0; s < 3; ++s) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+                uint2 w;
+                w.x = *reinterpret_cast<const uint32_t*>(&lo);
+                w.y = *reinterpret_cast<const uint32_t*>(&hi);
+                *reinterpret_cast<uint2*>(&b.u[s][(tid >> 3) + 32 * q][4 * (tid & 7)]) = w;
+                v[0] -= __bfloat162float(lo.x); v[1] -= __bfloat162float(lo.y);
+                v[2] -= __bfloat162float(hi.x); v[3] -= __bfloat162float(hi.y);
+            }
+        }
+    };
+    fetch_u(0);
+    fetch_w(0, buf[0]);
+    int which = 0;
+    for (int k0 = 0; k0 < n; k0 += kGK, which ^= 1) {
+        GateTiles& b = buf[which];
+        store_u(b);
+        asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        __syncthreads();                        // this slice is complete; the other buffer has been read
+        if (k0 + kGK < n) { fetch_w(k0 + kGK, buf[which ^ 1]); fetch_u(k0 + kGK); }
 #pragma unroll
         for (int ks = 0; ks < kGK; ks += 16) {
             if (k0 + ks < n) {
                 uint32_t a[3][4];
 #pragma unroll
-                for (int s = 0; s < 3; ++s) ldmatrix_x4(a[s], &Us[s][warp * 16 + (lane & 15)][ks + (lane >> 4) * 8]);
+                for (int s = 0; s < 3; ++s) ldmatrix_x4(a[s], &b.u[s][wt * 16 + (lane & 15)][ks + (lane >> 4) * 8]);
 #pragma unroll
                 for (int g = 0; g < 2; ++g)
 #pragma unroll
-                    for (int x = 0; x < 4; ++x) {
-                        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(&Ws[g][x * 8 + r0][ks + c2]);
-                        const uint32_t b1 = *reinterpret_cast<const uint32_t*>(&Ws[g][x * 8 + r0][ks + 8 + c2]);
+                    for (int x = 0; x < 4; x += 2) {
+                        uint32_t w4[4];
+                        ldmatrix_x4(w4, &b.w[g][wc * 32 + x * 8 + (lane >> 4) * 8 + (lane & 7)][ks + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-                        for (int s = 2; s >= 0; --s) mma_bf16_16816(acc[g][x], a[s][0], a[s][1], a[s][2], a[s][3], b0, b1);
+                        for (int s = 2; s >= 0; --s) {
+                            mma_bf16_16816(acc[g][x], a[s][0], a[s][1], a[s][2], a[s][3], w4[0], w4[1]);
+                            mma_bf16_16816(acc[g][x + 1], a[s][0], a[s][1], a[s][2], a[s][3], w4[2], w4[3]);
+                        }
                     }
             }
         }
@@ -111,14 +152,22 @@ lru_gates_tc_kernel(const float* __restrict__ u, const __nv_bfloat16* __restrict
 #pragma unroll
     for (int x = 0; x < 4; ++x)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int t = t0 + warp * 16 + r0 + (e >> 1) * 8, o = c0 + x * 8 + c2 + (e & 1);
+        for (int e = 0; e < 4; e += 2) {
+            const int t = t0 + wt * 16 + r0 + (e >> 1) * 8, o = c0 + wc * 32 + x * 8 + c2;
             if (t < T && o < n) {
                 const int c = part * n + o;
-                float a, dr;
-                decay_drive(acc[0][x][e] + br[c], acc[1][x][e] + bi[c], lam[c], u[(int64_t)t * W + c], a, dr);
-                a_out[(int64_t)t * W + c] = a;
-                x_out[(int64_t)t * W + c] = dr;
+                const int64_t at = (int64_t)t * W + c;
+                const bool two = o + 1 < n;
+                float a0, x0, a1 = 0.f, x1 = 0.f;
+                decay_drive(acc[0][x][e] + br[c], acc[1][x][e] + bi[c], rate[c], u[at], a0, x0);
+                if (two) decay_drive(acc[0][x][e + 1] + br[c + 1], acc[1][x][e + 1] + bi[c + 1], rate[c + 1], u[at + 1], a1, x1);
+                if (vec) {                      // (channels in fours: two neighbours lie on an 8-byte boundary)
+                    *reinterpret_cast<float2*>(a_out + at) = make_float2(a0, a1);
+                    *reinterpret_cast<float2*>(x_out + at) = make_float2(x0, x1);
+                } else {
+                    a_out[at] = a0; x_out[at] = x0;
+                    if (two) { a_out[at + 1] = a1; x_out[at + 1] = x1; }
+                }
             }
         }
 }
@@ -126,13 +175,13 @@ lru_gates_tc_kernel(const float* __restrict__ u, const __nv_bfloat16* __restrict
 // zr, zi [T, W]: the products before their biases; a replaces zr and the drive replaces zi.
 __global__ void __launch_bounds__(256)
 lru_prepare_kernel(const float* __restrict__ u, float* __restrict__ zr, float* __restrict__ zi, const float* __restrict__ br,
-                   const float* __restrict__ bi, const float* __restrict__ lam, int64_t total, int W) {
+                   const float* __restrict__ bi, const float* __restrict__ rate, int64_t total, int W) {
     wait_for_earlier_kernels();
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
     const int c = (int)(idx % W);
     float a, x;
-    decay_drive(zr[idx] + br[c], zi[idx] + bi[c], lam[c], u[idx], a, x);
+    decay_drive(zr[idx] + br[c], zi[idx] + bi[c], rate[c], u[idx], a, x);
     zr[idx] = a;
     zi[idx] = x;
 }
@@ -242,72 +291,106 @@ struct DecodeArgs {
     const __nv_bfloat16* wi;
     const float* br;
     const float* bi;
-    const float* lam;
+    const float* rate;
     float* state;
     int64_t stride, s_off, c_off;
 };
 
-template <typename AT>
+constexpr int kDecR = 2;                // requests a cluster serves together: the part's matrices are read once for both
+constexpr int kDecCh = 4;               // channels of a warp of a block of 8 (slices of at most 32)
+
+template <typename AT, bool PRE>        // PRE: parts of up to 256 channels in eights, slices of up to 32: a lane's weights fit registers
 __global__ void __launch_bounds__(256)
 lru_decode_kernel(DecodeArgs g, const int* __restrict__ q_start, const int* __restrict__ state_slot, AT* __restrict__ out,
-                  int W, int n, int cs, int taps, int vec) {
-    extern __shared__ __align__(16) float us[];             // [n rounded up to 8] u of the part, [cs] its newest input
+                  int B, int W, int n, int cs, int taps) {
+    extern __shared__ __align__(16) float dec_sm[];         // u of the part for two requests, then the gates' products
+    const int np = (n + 7) / 8 * 8;
+    float* us = dec_sm;                                     // [2][np]
+    float* zs = us + kDecR * np;                            // [2][2][cs]
     asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
-    wait_for_earlier_kernels();
-    const int b = blockIdx.z, part = blockIdx.y, c_lo = blockIdx.x * cs, nc = min(cs, n - c_lo);
+    const int part = blockIdx.y, c_lo = blockIdx.x * cs, nc = min(cs, n - c_lo);
+    const int b0 = blockIdx.z * kDecR, nb = min(kDecR, B - b0);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int64_t t = q_start[b];
-    float* row = g.state + (int64_t)state_slot[b] * g.stride;
-    float* hist = row + g.c_off + part * n;
-    const float* pr = g.proj + t * g.ld;
-    for (int i = tid; i < n; i += 256) {
-        const int c = part * n + i;
-        float u = g.bc[c];
-        for (int j = 0; j + 1 < taps; ++j) u += g.conv[c * taps + j] * hist[(int64_t)j * W + i];
-        us[i] = u + g.conv[c * taps + taps - 1] * (pr[g.col_x + c] + g.bx[c]);
-    }
-    for (int i = n + tid; i < (n + 7) / 8 * 8; i += 256) us[i] = 0.f;
-    __syncthreads();
-    for (int o = warp; o < nc; o += 8) {
-        const int64_t wrow = ((int64_t)part * n + c_lo + o) * n;
-        float zr = 0.f, zi = 0.f;
-        if (vec) {
-            for (int k = 8 * lane; k < n; k += 256) {
-                const uint4 a = *reinterpret_cast<const uint4*>(g.wr + wrow + k), d = *reinterpret_cast<const uint4*>(g.wi + wrow + k);
-                const __nv_bfloat162* ap = reinterpret_cast<const __nv_bfloat162*>(&a);
-                const __nv_bfloat162* dp = reinterpret_cast<const __nv_bfloat162*>(&d);
+    // the weights wait for no earlier kernel: this warp's channels (warp + 8 q) are asked for first
+    uint4 pa[kDecCh], pd[kDecCh];
+    if (PRE) {
 #pragma unroll
-                for (int x = 0; x < 4; ++x) {
-                    const float2 af = __bfloat1622float2(ap[x]), df = __bfloat1622float2(dp[x]);
-                    const float u0 = us[k + 2 * x], u1 = us[k + 2 * x + 1];
-                    zr += af.x * u0; zr += af.y * u1;
-                    zi += df.x * u0; zi += df.y * u1;
-                }
-            }
-        } else {
-            for (int k = lane; k < n; k += 32) {
-                zr += to_float(g.wr[wrow + k]) * us[k];
-                zi += to_float(g.wi[wrow + k]) * us[k];
+        for (int q = 0; q < kDecCh; ++q) {
+            const int o = warp + 8 * q, k = 8 * lane;
+            pa[q] = pd[q] = make_uint4(0u, 0u, 0u, 0u);
+            if (o < nc && k < n) {
+                const int64_t at = ((int64_t)part * n + c_lo + o) * n + k;
+                pa[q] = __ldg(reinterpret_cast<const uint4*>(g.wr + at));
+                pd[q] = __ldg(reinterpret_cast<const uint4*>(g.wi + at));
             }
         }
-        zr = warp_sum(zr);
-        zi = warp_sum(zi);
-        if (lane == 0) {
-            const int c = part * n + c_lo + o;
-            float a, x;
-            decay_drive(zr + g.br[c], zi + g.bi[c], g.lam[c], us[c_lo + o], a, x);
-            float* S = row + g.s_off + c;
-            const float s = a * *S + x;
-            *S = s;
-            out[t * W + c] = from_float<AT>(s * gelu_tanh_f(pr[g.col_y + c] + g.by[c]));
+    }
+    wait_for_earlier_kernels();
+    for (int idx = tid; idx < nb * np; idx += 256) {
+        const int r = idx / np, i = idx - r * np, c = part * n + i;
+        float u = 0.f;
+        if (i < n) {
+            const float* hist = g.state + (int64_t)state_slot[b0 + r] * g.stride + g.c_off + c;
+            float h[kMaxTaps];
+#pragma unroll
+            for (int j = 0; j < kMaxTaps; ++j) h[j] = j + 1 < taps ? hist[(int64_t)j * W] : 0.f;
+            const float in = g.proj[(int64_t)q_start[b0 + r] * g.ld + g.col_x + c] + g.bx[c];
+            u = g.bc[c];
+#pragma unroll
+            for (int j = 0; j < kMaxTaps; ++j) if (j < taps) u += g.conv[c * taps + j] * (j + 1 < taps ? h[j] : in);
+        }
+        us[idx] = u;
+    }
+    __syncthreads();
+    for (int q = 0, o = warp; o < nc; ++q, o += 8) {
+        float zr[kDecR] = {0.f, 0.f}, zi[kDecR] = {0.f, 0.f};
+        if (!PRE) {
+            const int64_t wrow = ((int64_t)part * n + c_lo + o) * n;
+            for (int k = lane; k < n; k += 32) {
+                const float a = to_float(g.wr[wrow + k]), d = to_float(g.wi[wrow + k]);
+                for (int r = 0; r < nb; ++r) { zr[r] += a * us[r * np + k]; zi[r] += d * us[r * np + k]; }
+            }
+        } else if (8 * lane < n) {
+            uint4 a = pa[0], d = pd[0];
+#pragma unroll
+            for (int x = 1; x < kDecCh; ++x) if (q == x) { a = pa[x]; d = pd[x]; }
+            const __nv_bfloat162* ap = reinterpret_cast<const __nv_bfloat162*>(&a);
+            const __nv_bfloat162* dp = reinterpret_cast<const __nv_bfloat162*>(&d);
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const float2 af = __bfloat1622float2(ap[x]), df = __bfloat1622float2(dp[x]);
+#pragma unroll
+                for (int r = 0; r < kDecR; ++r) {
+                    if (r < nb) {
+                        const float2 u2 = *reinterpret_cast<const float2*>(us + r * np + 8 * lane + 2 * x);
+                        zr[r] += af.x * u2.x; zr[r] += af.y * u2.y;
+                        zi[r] += df.x * u2.x; zi[r] += df.y * u2.y;
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < kDecR; ++r) {
+            zr[r] = warp_sum(zr[r]);
+            zi[r] = warp_sum(zi[r]);
+            if (lane == 0) { zs[(2 * r) * cs + o] = zr[r]; zs[(2 * r + 1) * cs + o] = zi[r]; }
         }
     }
     cg::cluster_group cluster = cg::this_cluster();
     asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
-    cluster.sync();                                         // every block has read the convolution's state
-    for (int i = tid; i < nc; i += 256) {
-        const int c = part * n + c_lo + i;
-        float* h = hist + c_lo + i;
+    cluster.sync();                                         // the products are there; every block has read the convolution's state
+    for (int idx = tid; idx < nb * nc; idx += 256) {
+        const int r = idx / nc, o = idx - r * nc, c = part * n + c_lo + o;
+        const int64_t t = q_start[b0 + r];
+        const float* pr = g.proj + t * g.ld;
+        float* row = g.state + (int64_t)state_slot[b0 + r] * g.stride;
+        float* S = row + g.s_off + c;
+        float* h = row + g.c_off + c;
+        float a, x;
+        decay_drive(zs[(2 * r) * cs + o] + g.br[c], zs[(2 * r + 1) * cs + o] + g.bi[c], g.rate[c], us[r * np + c_lo + o], a, x);
+        const float s = a * *S + x;
+        *S = s;
+        out[t * W + c] = from_float<AT>(s * gelu_tanh_f(pr[g.col_y + c] + g.by[c]));
         for (int j = 0; j + 2 < taps; ++j) h[(int64_t)j * W] = h[(int64_t)(j + 1) * W];
         if (taps > 1) h[(int64_t)(taps - 2) * W] = pr[g.col_x + c] + g.bx[c];
     }
@@ -329,24 +412,28 @@ static bool bad_lru(int W, int n, int B) {
 }
 
 // a, x [T, W] from u [T, W] with the gates' matrices [W/n][n][n] in bfloat16
-int mi_lru_gates_tc(const float* u, const void* wr, const void* wi, const float* br, const float* bi, const float* lam,
+int mi_lru_gates_tc(const float* u, const void* wr, const void* wi, const float* br, const float* bi, const float* rate,
                     float* a, float* x, int T, int W, int n, cudaStream_t stream) {
     if (T <= 0) return kOk;
     if (bad_lru(W, n, 1)) return kBadShape;
     const int ctiles = (n + lru::kGC - 1) / lru::kGC;
     if ((int64_t)(W / n) * ctiles > 65535) { set_last_error("gated linear recurrence: %d channels", W); return kBadShape; }
-    launch_dependent(lru::lru_gates_tc_kernel, dim3((T + lru::kGT - 1) / lru::kGT, W / n * ctiles), dim3(128), 0, stream, u,
-                     (const __nv_bfloat16*)wr, (const __nv_bfloat16*)wi, br, bi, lam, a, x, T, W, n, ctiles);
+    const int vec = n % 8 == 0 && ((reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(wr) | reinterpret_cast<uintptr_t>(wi) |
+                                    reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
+    const size_t smem = 2 * sizeof(lru::GateTiles);
+    cudaFuncSetAttribute(lru::lru_gates_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_dependent(lru::lru_gates_tc_kernel, dim3((T + lru::kGT - 1) / lru::kGT, W / n * ctiles), dim3(256), smem, stream, u,
+                     (const __nv_bfloat16*)wr, (const __nv_bfloat16*)wi, br, bi, rate, a, x, T, W, n, ctiles, vec);
     return finish_launch("lru_gates_tc");
 }
 
-int mi_lru_prepare(const float* u, float* zr, float* zi, const float* br, const float* bi, const float* lam, int T, int W,
+int mi_lru_prepare(const float* u, float* zr, float* zi, const float* br, const float* bi, const float* rate, int T, int W,
                    cudaStream_t stream) {
     if (T <= 0) return kOk;
     if (bad_lru(W, W, 1)) return kBadShape;
     const int64_t total = (int64_t)T * W;
     launch_dependent(lru::lru_prepare_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, u, zr, zi, br, bi,
-                     lam, total, W);
+                     rate, total, W);
     return finish_launch("lru_prepare");
 }
 
@@ -377,7 +464,7 @@ int mi_lru_scan(const float* a, const float* x, const float* y, int ld_y, const 
 
 // One token per request (checked by the caller): convolution, gates, recurrence and output.
 int mi_lru_decode(const float* proj, int ld, int col_x, int col_y, const float* bx, const float* conv, const float* bc,
-                  const float* by, const void* wr, const void* wi, const float* br, const float* bi, const float* lam,
+                  const float* by, const void* wr, const void* wi, const float* br, const float* bi, const float* rate,
                   float* state, int64_t stride, int64_t s_off, int64_t c_off, const int* q_start, const int* state_slot,
                   void* out, int adtype, int B, int W, int n, int taps, cudaStream_t stream) {
     if (B <= 0) return kOk;
@@ -387,13 +474,13 @@ int mi_lru_decode(const float* proj, int ld, int col_x, int col_y, const float* 
     if (slices > 8) slices = 8;
     const int cs = (n + slices - 1) / slices;
     slices = (n + cs - 1) / cs;
-    const size_t smem = sizeof(float) * ((n + 7) / 8 * 8);
+    const size_t smem = sizeof(float) * (lru::kDecR * ((n + 7) / 8 * 8) + 2 * lru::kDecR * cs);
     if (smem > 200 * 1024) { set_last_error("gated linear recurrence: parts of %d channels", n); return kBadShape; }
-    const int vec = n % 8 == 0 && ((reinterpret_cast<uintptr_t>(wr) | reinterpret_cast<uintptr_t>(wi)) & 15) == 0;
+    const bool pre = n % 8 == 0 && n <= 256 && cs <= 32 && ((reinterpret_cast<uintptr_t>(wr) | reinterpret_cast<uintptr_t>(wi)) & 15) == 0;
     const lru::DecodeArgs g = {proj, ld, col_x, col_y, bx, conv, bc, by, (const __nv_bfloat16*)wr, (const __nv_bfloat16*)wi,
-                               br, bi, lam, state, stride, s_off, c_off};
+                               br, bi, rate, state, stride, s_off, c_off};
     cudaLaunchConfig_t lc = {};
-    lc.gridDim = dim3(slices, W / n, B);
+    lc.gridDim = dim3(slices, W / n, (B + lru::kDecR - 1) / lru::kDecR);
     lc.blockDim = dim3(256);
     lc.dynamicSmemBytes = smem;
     lc.stream = stream;
@@ -406,11 +493,14 @@ int mi_lru_decode(const float* proj, int ld, int col_x, int col_y, const float* 
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     lc.attrs = attr;
     lc.numAttrs = dependent_launch_enabled() ? 2 : 1;
-    MI_DISPATCH_1(adtype, AT, {
-        if (smem > 48 * 1024)
-            cudaFuncSetAttribute(lru::lru_decode_kernel<AT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        (void)cudaLaunchKernelEx(&lc, lru::lru_decode_kernel<AT>, g, q_start, state_slot, (AT*)out, W, n, cs, taps, vec);
-    });
+#define MI_LRU_DECODE(PRE)                                                                                            \
+    MI_DISPATCH_1(adtype, AT, {                                                                                       \
+        if (smem > 48 * 1024)                                                                                         \
+            cudaFuncSetAttribute(lru::lru_decode_kernel<AT, PRE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        (void)cudaLaunchKernelEx(&lc, lru::lru_decode_kernel<AT, PRE>, g, q_start, state_slot, (AT*)out, B, W, n, cs, taps); \
+    })
+    if (pre) MI_LRU_DECODE(true); else MI_LRU_DECODE(false);
+#undef MI_LRU_DECODE
     return finish_launch("lru_decode");
 }
 

@@ -291,6 +291,49 @@ memory_walk_kernel(Rows in, State st, const float4* __restrict__ gates, const fl
         }
 }
 
+// The same for groups of whole fours on 16-byte boundaries, kept in registers between the sum and the result: a warp per
+// group of up to 512 columns (ONE_WARP; eight groups a block), a block of 256 threads per group of up to 8,192.
+template <typename AT, typename GT, int VPT, bool ONE_WARP>
+__global__ void __launch_bounds__(256)
+memory_finish_vec_kernel(const float* __restrict__ o, const float* __restrict__ den, const float4* __restrict__ gates,
+                         const GT* __restrict__ gate, int64_t ld_gate, const float* __restrict__ w, AT* __restrict__ out,
+                         int n, int gs, float eps, int64_t total) {
+    __shared__ float scratch[32];
+    wait_for_earlier_kernels();
+    const int groups = n / gs;
+    const int64_t at = ONE_WARP ? (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5) : (int64_t)blockIdx.x;     // (token, group)
+    if (at >= total) return;                                       // (one warp: whole warps leave, and no block-wide barrier follows)
+    const int64_t t = at / groups;
+    const int h = (int)(at - t * groups);
+    constexpr int TH = ONE_WARP ? 32 : 256;
+    const int i0 = ONE_WARP ? threadIdx.x & 31 : threadIdx.x, nv = gs / 4;
+    const float4* row = reinterpret_cast<const float4*>(o + at * gs);
+    const float4* wr = reinterpret_cast<const float4*>(w + h * gs);
+    const GT* gr = gate + t * ld_gate + h * gs;
+    AT* orow = out + at * gs;
+    const float inv = den ? 1.0f / (fmaxf(fabsf(den[at]), gates[at].z) + 1e-6f) : 1.0f;
+    float4 v[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i = i0 + TH * j;
+        v[j] = i < nv ? row[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[j].x *= inv; v[j].y *= inv; v[j].z *= inv; v[j].w *= inv;
+        ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+    }
+    ss = ONE_WARP ? warp_sum(ss) : block_sum(ss, scratch);
+    const float rr = 1.0f / sqrtf(ss / (float)gs + eps);
+#pragma unroll
+    for (int j = 0; j < VPT; ++j) {
+        const int i = i0 + TH * j, c = 4 * i;
+        if (i < nv) {
+            const float4 u = wr[i];
+            store4(orow + c, make_float4(v[j].x * rr * u.x * sigmoid_f(to_float(gr[c])), v[j].y * rr * u.y * sigmoid_f(to_float(gr[c + 1])),
+                                         v[j].z * rr * u.z * sigmoid_f(to_float(gr[c + 2])), v[j].w * rr * u.w * sigmoid_f(to_float(gr[c + 3]))));
+        }
+    }
+}
+
 // y = rmsnorm_group(o / (max(|n . q|, exp(-m)) + 1e-6)) * w * logistic(gate): a block per (token, group of gs columns).
 // With log gates a group is a head (gs = dv; den is n . q and gates[..].z is exp(-m)); den null: nothing is divided and a
 // group is whatever the caller says.  w has an entry per column.
@@ -298,7 +341,7 @@ template <typename AT, typename GT>
 __global__ void __launch_bounds__(128)
 memory_finish_kernel(const float* __restrict__ o, const float* __restrict__ den, const float4* __restrict__ gates,
                      const GT* __restrict__ gate, int64_t ld_gate, const float* __restrict__ w, AT* __restrict__ out,
-                     int n, int gs, float eps, int vec) {
+                     int n, int gs, float eps) {
     __shared__ float scratch[32];
     wait_for_earlier_kernels();
     const int64_t t = blockIdx.x;
@@ -309,27 +352,11 @@ memory_finish_kernel(const float* __restrict__ o, const float* __restrict__ den,
     AT* orow = out + t * n + (int64_t)h * gs;
     const float inv = den ? 1.0f / (fmaxf(fabsf(den[t * H + h]), gates[t * H + h].z) + 1e-6f) : 1.0f;
     float ss = 0.f;
-    if (vec) {
-        for (int c = 4 * threadIdx.x; c < gs; c += 4 * blockDim.x) {
-            const float4 v = *reinterpret_cast<const float4*>(row + c);
-            const float a = v.x * inv, b = v.y * inv, d = v.z * inv, e = v.w * inv;
-            ss += (a * a + b * b) + (d * d + e * e);
-        }
-    } else {
-        for (int c = threadIdx.x; c < gs; c += blockDim.x) { const float v = row[c] * inv; ss += v * v; }
-    }
+    for (int c = threadIdx.x; c < gs; c += blockDim.x) { const float v = row[c] * inv; ss += v * v; }
     ss = block_sum(ss, scratch);
     const float rr = inv / sqrtf(ss / (float)gs + eps);
-    if (vec) {
-        for (int c = 4 * threadIdx.x; c < gs; c += 4 * blockDim.x) {
-            const float4 v = *reinterpret_cast<const float4*>(row + c), u = *reinterpret_cast<const float4*>(wr + c);
-            store4(orow + c, make_float4(v.x * rr * u.x * sigmoid_f(to_float(gr[c])), v.y * rr * u.y * sigmoid_f(to_float(gr[c + 1])),
-                                         v.z * rr * u.z * sigmoid_f(to_float(gr[c + 2])), v.w * rr * u.w * sigmoid_f(to_float(gr[c + 3]))));
-        }
-    } else {
-        for (int c = threadIdx.x; c < gs; c += blockDim.x)
-            orow[c] = from_float<AT>(row[c] * rr * wr[c] * sigmoid_f(to_float(gr[c])));
-    }
+    for (int c = threadIdx.x; c < gs; c += blockDim.x)
+        orow[c] = from_float<AT>(row[c] * rr * wr[c] * sigmoid_f(to_float(gr[c])));
 }
 
 }  // namespace mem
@@ -673,13 +700,36 @@ memory_chunk_states_kernel(RowsB in, const float4* __restrict__ gates, const flo
 
 // S_start[0] = the request's state, S_start[c + 1] = keepc[c] S_start[c] + U[c], a thread per eight columns of a row of S;
 // what follows the last chunk is the request's new state.  S_start[c] takes the place of U[c] once that has been read, as
-// eight high parts and eight remainders in bfloat16: what the outputs' products take.
+// eight high parts and eight remainders in bfloat16: what the outputs' products take.  With Un the last block of every
+// head chains n in the same way (it stays float).
 __global__ void __launch_bounds__(256)
-memory_chunk_chain_kernel(float* __restrict__ U, const float* __restrict__ keepc, float* __restrict__ state,
-                          int64_t state_stride, int64_t off, const int* __restrict__ q_start,
-                          const int* __restrict__ state_slot, int H, int d, int dv, int dvp) {
+memory_chunk_chain_kernel(float* __restrict__ U, float* __restrict__ Un, const float* __restrict__ keepc,
+                          float* __restrict__ state, int64_t state_stride, int64_t off, int64_t n_off,
+                          const int* __restrict__ q_start, const int* __restrict__ state_slot, int H, int d, int dv, int dvp) {
     wait_for_earlier_kernels();
     const int b = blockIdx.z, h = blockIdx.y;
+    if (Un && blockIdx.x == gridDim.x - 1) {
+        const int i = threadIdx.x, q0 = q_start[b], n = q_start[b + 1] - q0;        // (keys of at most 256 numbers)
+        if (i >= d || n <= 0) return;
+        const int chunks = (n + kC - 1) / kC;
+        const int64_t first = (int64_t)(q0 / kC + b) * H + h;
+        float* S = state + (int64_t)state_slot[b] * state_stride + n_off + (int64_t)h * d + i;
+        float cur = *S;
+        for (int c0 = 0; c0 < chunks; c0 += 8) {
+            float u[8], keep[8];
+#pragma unroll
+            for (int a = 0; a < 8; ++a) {
+                const int64_t at = first + (int64_t)min(c0 + a, chunks - 1) * H;
+                u[a] = Un[at * d + i];
+                keep[a] = keepc[at];
+            }
+#pragma unroll
+            for (int a = 0; a < 8; ++a)
+                if (c0 + a < chunks) { Un[(first + (int64_t)(c0 + a) * H) * d + i] = cur; cur = keep[a] * cur + u[a]; }
+        }
+        *S = cur;
+        return;
+    }
     const int e = blockIdx.x * blockDim.x + threadIdx.x, groups = dvp / 8;
     const int q0 = q_start[b], n = q_start[b + 1] - q0;
     if (e >= d * groups || n <= 0) return;
@@ -721,34 +771,6 @@ memory_chunk_chain_kernel(float* __restrict__ U, const float* __restrict__ keepc
     }
 #pragma unroll
     for (int x = 0; x < 8; ++x) if (c8 + x < dv) S[x] = cur[x];
-}
-
-// the same for n, which stays float
-__global__ void __launch_bounds__(256)
-memory_chunk_norm_chain_kernel(float* __restrict__ Un, const float* __restrict__ keepc, float* __restrict__ state,
-                               int64_t state_stride, int64_t off, const int* __restrict__ q_start,
-                               const int* __restrict__ state_slot, int H, int d) {
-    wait_for_earlier_kernels();
-    const int b = blockIdx.z, h = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x;
-    const int q0 = q_start[b], n = q_start[b + 1] - q0;
-    if (i >= d || n <= 0) return;
-    const int chunks = (n + kC - 1) / kC;
-    const int64_t first = (int64_t)(q0 / kC + b) * H + h;
-    float* S = state + (int64_t)state_slot[b] * state_stride + off + (int64_t)h * d + i;
-    float cur = *S;
-    for (int c0 = 0; c0 < chunks; c0 += 4) {
-        float u[4], keep[4];
-#pragma unroll
-        for (int a = 0; a < 4; ++a) {
-            const int64_t at = first + (int64_t)min(c0 + a, chunks - 1) * H;
-            u[a] = Un[at * d + i];
-            keep[a] = keepc[at];
-        }
-#pragma unroll
-        for (int a = 0; a < 4; ++a)
-            if (c0 + a < chunks) { Un[(first + (int64_t)(c0 + a) * H) * d + i] = cur; cur = keep[a] * cur + u[a]; }
-    }
-    *S = cur;
 }
 
 // Read-outs of a chunk.  Block = 8 warps: warp w owns the tokens 16 (w % 4) .. + 15 of the chunk and half of a value tile of
@@ -1018,18 +1040,16 @@ int mi_memory_chunks(const void* proj, int ld, int col_q, int col_k, int col_v, 
         cudaFuncSetAttribute(mem::memory_chunk_outputs_kernel<LOG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_o); \
         launch_dependent(mem::memory_chunk_states_kernel<LOG>, dim3(chunks, H * tiles, B), dim3(128), smem_s, stream, in, \
                          (const float4*)gates, (const float4*)logs, decay, q_start, U, Un, keepc, H, d, dv, dvp, dp, tiles); \
-        launch_dependent(mem::memory_chunk_chain_kernel, dim3((d * (dvp / 8) + 255) / 256, H, B), dim3(256), 0, stream, U, \
-                         (const float*)keepc, state, stride, s_off, q_start, state_slot, H, d, dv, dvp);               \
-        if (LOG)                                                                                                       \
-            launch_dependent(mem::memory_chunk_norm_chain_kernel, dim3((d + 255) / 256, H, B), dim3(256), 0, stream, Un, \
-                             (const float*)keepc, state, stride, n_off, q_start, state_slot, H, d);                    \
+        launch_dependent(mem::memory_chunk_chain_kernel, dim3((d * (dvp / 8) + 255) / 256 + (LOG ? 1 : 0), H, B), dim3(256), \
+                         0, stream, U, LOG ? Un : nullptr, (const float*)keepc, state, stride, s_off, n_off, q_start,  \
+                         state_slot, H, d, dv, dvp);                                                                   \
         launch_dependent(mem::memory_chunk_outputs_kernel<LOG>, dim3(chunks, H * groups, B), dim3(256), smem_o, stream, in, \
                          (const float4*)gates, (const float4*)logs, decay, q_start, (const float*)U, (const float*)Un, out, \
                          den, H, d, dv, dvp, dp, tiles, per, groups);                                                  \
     } while (0)
     if (gates) MI_CHUNKS(true); else MI_CHUNKS(false);
 #undef MI_CHUNKS
-    return finish_launch("memory_chunks", gates ? 4 : 3);
+    return finish_launch("memory_chunks", 3);
 }
 
 // out [T, n] = rmsnorm over groups of gs columns of o / (max(|den|, exp(-m)) + 1e-6), times w [n], times logistic(gate);
@@ -1041,12 +1061,29 @@ int mi_memory_finish(const float* o, const float* den, const float* gates, const
         set_last_error("matrix memory: %d columns in groups of %d", n, gs);
         return kBadShape;
     }
-    const int vec = gs % 4 == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const bool vec = gs % 4 == 0 && gs <= 8192 &&
+                     ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const int64_t total = (int64_t)T * (n / gs);
+#define MI_FINISH_VEC(VPT, ONE)                                                                                       \
+    MI_DISPATCH_2(adtype, AT, gdtype, GT,                                                                             \
+        launch_dependent(mem::memory_finish_vec_kernel<AT, GT, VPT, ONE>, dim3((unsigned)(ONE ? (total + 7) / 8 : total)), \
+                         dim3(256), 0, stream, o, den, (const float4*)gates, (const GT*)gate, ld_gate, w, (AT*)out, n, gs, \
+                         eps, total))
+    if (vec) {
+        if (gs <= 128) MI_FINISH_VEC(1, true);
+        else if (gs <= 256) MI_FINISH_VEC(2, true);
+        else if (gs <= 512) MI_FINISH_VEC(4, true);
+        else if (gs <= 2048) MI_FINISH_VEC(2, false);
+        else if (gs <= 4096) MI_FINISH_VEC(4, false);
+        else MI_FINISH_VEC(8, false);
+#undef MI_FINISH_VEC
+        return finish_launch("memory_finish");
+    }
     int threads = 32;
-    while (threads < (vec ? gs / 4 : gs) && threads < 128) threads *= 2;
+    while (threads < gs && threads < 128) threads *= 2;
     MI_DISPATCH_2(adtype, AT, gdtype, GT,
         launch_dependent(mem::memory_finish_kernel<AT, GT>, dim3(T, n / gs), dim3(threads), 0, stream, o, den,
-                         (const float4*)gates, (const GT*)gate, ld_gate, w, (AT*)out, n, gs, eps, vec));
+                         (const float4*)gates, (const GT*)gate, ld_gate, w, (AT*)out, n, gs, eps));
     return finish_launch("memory_finish");
 }
 

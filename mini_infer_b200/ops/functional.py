@@ -1672,10 +1672,10 @@ def lru_segment_tokens() -> int:
     return int(library().mi_lru_segment_tokens())
 
 
-def lru_gates(u: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, lam: torch.Tensor):
+def lru_gates(u: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor, bi: torch.Tensor, rate: torch.Tensor):
     """``(a, x)`` float32 ``[T, W]`` of a real-gated linear recurrence: with ``u [T, W]`` float32 in ``W / n`` equal
     parts, ``r = logistic(wr_b u_b + br)``, ``i = logistic(wi_b u_b + bi)`` (``wr``, ``wi`` ``[W/n, n, n]``),
-    ``a = exp(-8 r softplus(lam))`` and ``x = sqrt(1 - a^2) i u``.  Matrices in bfloat16: tensor cores with ``u`` as
+    ``a = exp(rate r)`` (``rate``: a negative number per channel) and ``x = sqrt(1 - a^2) i u``.  Matrices in bfloat16: tensor cores with ``u`` as
     three bfloat16 parts; in float32: the fixed-order products of :func:`dense_f32_heads`."""
     _chk(u, "lru_gates u", F32)
     T, W = u.shape
@@ -1684,15 +1684,15 @@ def lru_gates(u: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Ten
     _chk(wi, "lru_gates wi", wr.dtype, (P, n, n))
     if P * n != W:
         raise ValueError(f"lru_gates: {P} parts of {n} for rows of {W}")
-    for t, name in ((br, "br"), (bi, "bi"), (lam, "lam")):
+    for t, name in ((br, "br"), (bi, "bi"), (rate, "rate")):
         _chk(t, "lru_gates " + name, F32, (W,))
     if wr.dtype == BF16:
         a, x = torch.empty_like(u), torch.empty_like(u)
-        check(library().mi_lru_gates_tc(_ptr(u), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(lam), _ptr(a), _ptr(x), T, W,
+        check(library().mi_lru_gates_tc(_ptr(u), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(rate), _ptr(a), _ptr(x), T, W,
                                         n, _stream()), "lru_gates")
         return a, x
     zr, zi = dense_f32_heads(u, wr), dense_f32_heads(u, wi)
-    check(library().mi_lru_prepare(_ptr(u), _ptr(zr), _ptr(zi), _ptr(br), _ptr(bi), _ptr(lam), T, W, _stream()),
+    check(library().mi_lru_prepare(_ptr(u), _ptr(zr), _ptr(zi), _ptr(br), _ptr(bi), _ptr(rate), T, W, _stream()),
           "lru_prepare")
     return zr, zi
 
@@ -1729,7 +1729,7 @@ def lru_scan(a: torch.Tensor, x: torch.Tensor, y: torch.Tensor, y_col: int, y_bi
 
 def lru_decode(proj: torch.Tensor, x_col: int, y_col: int, x_bias: torch.Tensor, conv: torch.Tensor,
                conv_bias: torch.Tensor, y_bias: torch.Tensor, wr: torch.Tensor, wi: torch.Tensor, br: torch.Tensor,
-               bi: torch.Tensor, lam: torch.Tensor, state: torch.Tensor, s_off: int, c_off: int, q_start: torch.Tensor,
+               bi: torch.Tensor, rate: torch.Tensor, state: torch.Tensor, s_off: int, c_off: int, q_start: torch.Tensor,
                state_slot: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
     """:func:`causal_conv`, :func:`lru_gates` and :func:`lru_scan` when every request brings exactly ONE token, in one
     launch (matrices in bfloat16; the convolution's state from ``c_off`` on, the recurrence's from ``s_off`` on)."""
@@ -1742,7 +1742,7 @@ def lru_decode(proj: torch.Tensor, x_col: int, y_col: int, x_bias: torch.Tensor,
     _chk(wi, what + " wi", BF16, (P, n, n))
     _chk(conv, what + " conv", F32, (W, None))
     taps = conv.shape[1]
-    for t in (x_bias, conv_bias, y_bias, br, bi, lam):
+    for t in (x_bias, conv_bias, y_bias, br, bi, rate):
         _chk(t, what + " vector", F32, (W,))
     _chk(state, what + " state", F32)
     B = state_slot.numel()
@@ -1756,7 +1756,7 @@ def lru_decode(proj: torch.Tensor, x_col: int, y_col: int, x_bias: torch.Tensor,
         _dbg_range(state_slot, 0, state.shape[0], what + " state_slot")
     out = torch.empty(T, W, dtype=out_dtype, device=proj.device)
     check(library().mi_lru_decode(_ptr(proj), proj.shape[1], int(x_col), int(y_col), _ptr(x_bias), _ptr(conv),
-                                  _ptr(conv_bias), _ptr(y_bias), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(lam),
+                                  _ptr(conv_bias), _ptr(y_bias), _ptr(wr), _ptr(wi), _ptr(br), _ptr(bi), _ptr(rate),
                                   _ptr(state), state.shape[1], int(s_off), int(c_off), _ptr(q_start), _ptr(state_slot),
                                   _ptr(out), _code(out, what + " out"), B, W, n, taps, _stream()), what)
     return out

@@ -549,7 +549,10 @@ class GatedLRU(Mixer):
         self.y_bias, self.x_bias, self.conv_bias = vec("y.b"), vec("x.b"), vec("conv.b")
         self.w_conv = _f32(tensors[p + "conv"], dev)
         self.w_r, self.w_i = m(tensors[p + "ra"], dev), m(tensors[p + "ri"], dev)
-        self.b_r, self.b_i, self.lam = vec("ra.b"), vec("ri.b"), vec("lam")
+        self.b_r, self.b_i = vec("ra.b"), vec("ri.b")
+        # log a = -8 softplus(lam) r: the factor on r, formed once
+        self.rate = (-8.0 * torch.nn.functional.softplus(tensors[p + "lam"].to(torch.float64), threshold=40.0)).to(
+            device=dev, dtype=torch.float32).contiguous()
         self.w_o = m(tensors[p + "o"], dev)
 
     def prefetch_first(self, ctx: StepContext, cache: Optional[CacheBinding]) -> None:
@@ -565,12 +568,12 @@ class GatedLRU(Mixer):
             ctx.prefetch((self.w_o,))
         if ctx.all_decode and self.rt.act == torch.bfloat16:
             out = F.lru_decode(proj, W, 0, self.x_bias, self.w_conv, self.conv_bias, self.y_bias, self.w_r, self.w_i,
-                               self.b_r, self.b_i, self.lam, state, 0, self.conv_off, ctx.q_start, ctx.state_slot,
+                               self.b_r, self.b_i, self.rate, state, 0, self.conv_off, ctx.q_start, ctx.state_slot,
                                self.rt.act)
         else:
             u = F.causal_conv(proj, W, W, self.x_bias, self.w_conv, self.conv_bias, state, self.conv_off, ctx.q_start,
                               ctx.req_of_token, ctx.state_slot)
-            a, drive = F.lru_gates(u, self.w_r, self.w_i, self.b_r, self.b_i, self.lam)
+            a, drive = F.lru_gates(u, self.w_r, self.w_i, self.b_r, self.b_i, self.rate)
             # the float32 path walks every portion in one piece, so that its sums run in one order
             segments = self.rt.act == torch.bfloat16 and ctx.max_q_len >= TUNING.lru_segments_min_tokens
             out = F.lru_scan(a, drive, proj, 0, self.y_bias, state, 0, ctx.q_start, ctx.state_slot, self.rt.act,

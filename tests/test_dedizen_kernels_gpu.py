@@ -237,6 +237,7 @@ def lru_case(W, blocks, taps, lens, seed):
 def run_lru(W, blocks, taps, p, xs, cuts, dtype, segments, slots, decode=True, out_dtype=torch.float32):
     fn = F()
     d = {k: v.to(DEV) for k, v in p.items()}
+    d["rate"] = (-8 * pd.softplus(p["lam"].double())).float().to(DEV)
     wr, wi = d["ra"].to(dtype).contiguous(), d["ri"].to(dtype).contiguous()
     c_off = -(-W // 4) * 4
     state = torch.randn(max(slots) + 2, c_off + taps * W, generator=torch.Generator().manual_seed(1)).to(DEV)
@@ -255,11 +256,11 @@ def run_lru(W, blocks, taps, p, xs, cuts, dtype, segments, slots, decode=True, o
         longest = max(r.shape[0] for r in rows)
         if decode and longest == 1 and dtype == torch.bfloat16:
             out = fn.lru_decode(proj, W + 3, 2, d["x.b"], d["conv"], d["conv.b"], d["y.b"], wr, wi, d["ra.b"], d["ri.b"],
-                                d["lam"], state, 0, c_off, qs, sl, out_dtype)
+                                d["rate"], state, 0, c_off, qs, sl, out_dtype)
         else:
             req = i32([n for n, r in enumerate(rows) for _ in range(r.shape[0])])
             u = fn.causal_conv(proj, W + 3, W, d["x.b"], d["conv"], d["conv.b"], state, c_off, qs, req, sl)
-            a, x = fn.lru_gates(u, wr, wi, d["ra.b"], d["ri.b"], d["lam"])
+            a, x = fn.lru_gates(u, wr, wi, d["ra.b"], d["ri.b"], d["rate"])
             out = fn.lru_scan(a, x, proj, 2, d["y.b"], state, 0, qs, sl, out_dtype, segments, longest)
         for n, r in enumerate(live):
             got[r].append(out[starts[n]:starts[n + 1]].float().cpu())
@@ -300,7 +301,7 @@ def test_gate_products_on_the_tensor_cores_keep_all_bits_of_their_input():
     i = pd.sigmoid(pd.block_product(z, wi.double(), bi.double().reshape(blocks, n)))
     log_a = -8 * r * pd.softplus(lam.double())
     want = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * z
-    args = [t.to(DEV) for t in (br, bi, lam)]
+    args = [t.to(DEV) for t in (br, bi, (-8 * pd.softplus(lam.double())).float())]
     got = F().lru_gates(u.to(DEV), wr.to(torch.bfloat16).to(DEV), wi.to(torch.bfloat16).to(DEV), *args)
     assert close(got[0], want[0], 3e-6) and close(got[1], want[1], 3e-6)
 
