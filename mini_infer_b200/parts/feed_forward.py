@@ -134,8 +134,6 @@ class SquaredReluMLP(FeedForward):
         F.l2_prefetch(self.w_up)
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        if ctx is not None and ctx.prefetch is not None:
-            ctx.prefetch((self.w_down,))
         if x.is_cuda and x.shape[0] <= TUNING.dense_skinny_max_tokens and F.dense_skinny_takes(x, self.w_up):
             act = F.dense_skinny(x, self.w_up, squared_relu=True)
         else:
