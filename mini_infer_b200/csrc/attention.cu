@@ -10,7 +10,8 @@
 // the 32-bit path and as the fallback of the bfloat16 path) and a split-KV
 // decode kernel with a merge step.  Masking is positional in all cases:
 // key j is visible from the query at absolute position p iff j <= p and
-// (window == 0 or j > p - window)  (same rule as :228-236).
+// (window == 0 or j > p - window)  (same rule as :228-236); the decode kernel
+// also knows chunks, an added key with a score per head and a gate per head (AttnForm).
 //
 // Cache layout per layer: [page, kv_head, page_size, d]; block_table[b, i] is
 // the page of keys [i*page_size, (i+1)*page_size) of request b, or -1 once a

@@ -10,7 +10,8 @@
 //      second buffer
 //   4. running softmax in the layout of the A fragments (a row's maximum and sum live in a quad of lanes),
 //      O_h += P_h V_g with V fragments fetched by ldmatrix.trans from the row-major tile
-// Behind a window the first keep_first keys of a request stay visible; a value row may be the leading part of
+// Behind a window or a chunk's start (AttnForm: which also holds an added key's scores and a gate per head) the first
+// keep_first keys of a request stay visible; a value row may be the leading part of
 // a longer row (`vrs` elements from one token's values to the next one's).
 // Steps of one token per request are split over the keys (blocks of 64 keys write a partial maximum, sum
 // and unnormalised output; a merge kernel finishes), since one block per request cannot pull a window of

@@ -18,7 +18,9 @@
 //   warp 1    allocates tensor memory, issues the MMAs
 //   warps 2-5 softmax and epilogue, one lane quarter of tensor memory each
 // S is double-buffered, so the next tile's S = Q K^T runs beside this tile's softmax.  Masking is positional: key j is visible from the
-// query at position p iff j <= p and (window == 0 or j > p - window or j < keep_first) and j < kv_len.
+// query at position p iff j <= p and (window == 0 or j > p - window or j < keep_first) and j < kv_len; with chunks
+// instead of a window iff j <= p and j lies in p's chunk (or j < keep_first): see AttnForm, which also gives the added
+// key of `sink` a score per head and the output a gate per head.
 //
 // Every wait on an mbarrier is bounded: a wait that runs out sets an error status that the host
 // reads, lets all roles fall through to the common exit, and the tensor memory is freed there.

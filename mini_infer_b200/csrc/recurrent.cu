@@ -2,7 +2,8 @@
 //
 //   causal_conv_silu   short causal convolution over time per channel (+ bias) and silu, with the last
 //                      taps-1 inputs of a request kept in its state slot between steps; the residual form
-//                      (causal_conv_residual) puts out x_t + conv(x)_t instead, without an activation
+//                      (causal_conv_residual) puts out x_t + conv(x)_t instead, without an activation, the plain
+//                      form (causal_conv_plain) conv(x)_t, with an optional bias on its inputs
 //   delta_scan         gated delta rule with one decay per head and key channel (or one per head):
 //                        S <- diag(g_t) S ;  u = beta_t (v_t - S^T k_t) ;  S <- S + k_t u^T ;  o_t = S^T q_t
 //                      and, without the correction, gated linear attention:
